@@ -27,9 +27,12 @@
 //                   mean square over the value size and multiplied by diff_scale;
 //   values_in_keys  the value of a key is the first v_dim elements of its key row (a latent that is
 //                   both key and value; there are no value pages);
-//   gate            head h of token t is multiplied by sigmoid(gate[t, gate_off + h]);
+//   gate            head h of token t is multiplied by sigmoid(gate[t, gate_off + h]), or (gate_dims) its
+//                   element d by sigmoid(gate[t, gate_off + h * v_dim + d]);
 //   chunk           instead of a window: the positions are cut into blocks of `chunk` counted from
-//                   position 0 of the sequence, and a query sees the keys j <= p of its own block.
+//                   position 0 of the sequence, and a query sees the keys j <= p of its own block;
+//   slopes          a number per head: the (capped) score of the query at p and the key at j loses
+//                   slopes[h] * (p - j).
 //
 // attention_mix_kernel: one block per token (and, in steps of few tokens, per run of
 // SPLIT_TILES key tiles of that token: the runs' partial results -- maximum, sum and
@@ -104,6 +107,8 @@ struct MixExtras {
     int gate_off;
     int chunk;                 // > 0: blocks of this many positions bound what a query sees (no window then)
     float softcap;             // > 0: a scaled score s becomes softcap * tanh(s / softcap) (before mix, mask and softmax)
+    int gate_dims;             // 1: the gate is a number per element of every head instead of one per head
+    const float* slopes;       // [n_q] or null
 };
 
 __device__ __forceinline__ float sigmoid_(float x) { return 1.0f / (1.0f + expf(-x)); }
@@ -131,7 +136,8 @@ __device__ __forceinline__ void finish_heads(T* __restrict__ out, const float* _
         for (int e = threadIdx.x; e < nh * v_dim; e += threads) {
             const int h = h_first + e / v_dim;
             float y = heads[e] * out_scale;
-            if (gate != nullptr) y *= sigmoid_(to_f32(gate[(size_t)t * ex.ld_gate + ex.gate_off + h]));
+            if (gate != nullptr)
+                y *= sigmoid_(to_f32(gate[(size_t)t * ex.ld_gate + ex.gate_off + (ex.gate_dims ? h_first * v_dim + e : h)]));
             out[((size_t)t * n_q + h_first) * v_dim + e] = from_f32<T>(y);
         }
         return;
@@ -266,8 +272,10 @@ attention_mix_kernel(T* __restrict__ out, const T* __restrict__ q, const T* __re
             __syncthreads();
             for (int idx = tid; idx < ng * group * KT; idx += THREADS) {
                 const int hl = idx / KT, jj = idx % KT, h = g0 * group + hl;
-                sraw[h * KT + jj] = capped(dot_row(qs + h * head_dim, ktile + ((size_t)(hl / group) * KT + jj) * ldk + (h % maps) * head_dim,
-                                            head_dim, kdot) * scale, ex.softcap);
+                float sc = capped(dot_row(qs + h * head_dim, ktile + ((size_t)(hl / group) * KT + jj) * ldk + (h % maps) * head_dim,
+                                          head_dim, kdot) * scale, ex.softcap);
+                if (ex.slopes != nullptr) sc = fmaf(-ex.slopes[h], (float)(pos - j0 - jj), sc);
+                sraw[h * KT + jj] = sc;
             }
         }
         __syncthreads();
@@ -606,13 +614,15 @@ attention_mix_mma_kernel(bf16* __restrict__ out, const bf16* __restrict__ q, con
                 }
             }
             float* sh = sraw + (size_t)h * QB * lds;
+            const float slope = ex.slopes != nullptr ? ex.slopes[h_first + h] : 0.f;
+            const int apart = pos0 + tig * 2 - j0;                      // distance of query tig * 2 from the tile's first key
 #pragma unroll
             for (int mb = 0; mb < 2; ++mb) {
                 const int key = mb * 16 + gid;
-                sh[(tig * 2) * lds + key] = capped(c[mb][0] * scale, ex.softcap);
-                sh[(tig * 2 + 1) * lds + key] = capped(c[mb][1] * scale, ex.softcap);
-                sh[(tig * 2) * lds + key + 8] = capped(c[mb][2] * scale, ex.softcap);
-                sh[(tig * 2 + 1) * lds + key + 8] = capped(c[mb][3] * scale, ex.softcap);
+                sh[(tig * 2) * lds + key] = fmaf(-slope, (float)(apart - key), capped(c[mb][0] * scale, ex.softcap));
+                sh[(tig * 2 + 1) * lds + key] = fmaf(-slope, (float)(apart + 1 - key), capped(c[mb][1] * scale, ex.softcap));
+                sh[(tig * 2) * lds + key + 8] = fmaf(-slope, (float)(apart - key - 8), capped(c[mb][2] * scale, ex.softcap));
+                sh[(tig * 2 + 1) * lds + key + 8] = fmaf(-slope, (float)(apart - key - 7), capped(c[mb][3] * scale, ex.softcap));
             }
         }
         __syncthreads();                                            // all scores are there; K is no longer needed
@@ -790,7 +800,7 @@ attention_mix_mma_kernel(bf16* __restrict__ out, const bf16* __restrict__ q, con
         const int hm = h_first + h;                                     // the head's index in the model
         float i0 = softmax_factor(m_run[h * QB + tig * 2], l_run[h * QB + tig * 2], ex.sink, hm) * out_scale;
         float i1 = softmax_factor(m_run[h * QB + tig * 2 + 1], l_run[h * QB + tig * 2 + 1], ex.sink, hm) * out_scale;
-        if (gate != nullptr) {
+        if (gate != nullptr && !ex.gate_dims) {
             if (tig * 2 < n_tok) i0 *= sigmoid_(to_f32(gate[(size_t)(row0 + tig * 2) * ex.ld_gate + ex.gate_off + hm]));
             if (tig * 2 + 1 < n_tok) i1 *= sigmoid_(to_f32(gate[(size_t)(row0 + tig * 2 + 1) * ex.ld_gate + ex.gate_off + hm]));
         }
@@ -798,15 +808,19 @@ attention_mix_mma_kernel(bf16* __restrict__ out, const bf16* __restrict__ q, con
         for (int vb = 0; vb < VB; ++vb) {
             if (vb * 16 >= v_dim) break;
             const int vd = vb * 16 + gid;
-            if (tig * 2 < n_tok) {
-                bf16* dst = out + ((size_t)(row0 + tig * 2) * n_q_all + hm) * v_dim;
-                dst[vd] = __float2bfloat16_rn(o[hh][vb][0] * i0);
-                dst[vd + 8] = __float2bfloat16_rn(o[hh][vb][2] * i0);
-            }
-            if (tig * 2 + 1 < n_tok) {
-                bf16* dst = out + ((size_t)(row0 + tig * 2 + 1) * n_q_all + hm) * v_dim;
-                dst[vd] = __float2bfloat16_rn(o[hh][vb][1] * i1);
-                dst[vd + 8] = __float2bfloat16_rn(o[hh][vb][3] * i1);
+#pragma unroll
+            for (int c = 0; c < 2; ++c) {
+                if (tig * 2 + c >= n_tok) continue;
+                const size_t row = row0 + tig * 2 + c;
+                bf16* dst = out + (row * n_q_all + hm) * v_dim;
+                float y0 = o[hh][vb][c] * (c ? i1 : i0), y1 = o[hh][vb][2 + c] * (c ? i1 : i0);
+                if (gate != nullptr && ex.gate_dims) {
+                    const bf16* gr = gate + row * ex.ld_gate + ex.gate_off + hm * v_dim;
+                    y0 *= sigmoid_(to_f32(gr[vd]));
+                    y1 *= sigmoid_(to_f32(gr[vd + 8]));
+                }
+                dst[vd] = __float2bfloat16_rn(y0);
+                dst[vd + 8] = __float2bfloat16_rn(y1);
             }
         }
     }
@@ -1103,7 +1117,7 @@ extern "C" int kipp_attention_shared_key(void* out, const void* q, const void* k
     MixExtras ex = {};
     ex.key_maps = 1;
     if (extras != nullptr) ex = *static_cast<const MixExtras*>(extras);
-    if (ex.key_maps != 1 || ex.diff) return KIPP_ERR_ARG;
+    if (ex.key_maps != 1 || ex.diff || ex.slopes || ex.gate_dims) return KIPP_ERR_ARG;
     cudaStream_t s = (cudaStream_t)stream;
     const int vb = (v_dim + 31) / 32;
 #define KIPP_SHARED_KEY(V)                                                                                            \
@@ -1149,6 +1163,7 @@ extern "C" int kipp_attention_mix_mma_ex(void* out, const void* q, const void* k
     ex.key_maps = 1;
     if (extras != nullptr) ex = *static_cast<const MixExtras*>(extras);
     if (ex.values_in_keys || (ex.diff && ex.key_maps != 2) || (ex.key_maps > 1 && head_mix != nullptr)) return KIPP_ERR_ARG;
+    if ((ex.slopes && head_mix) || (ex.gate_dims && ex.diff)) return KIPP_ERR_ARG;
     const int kvs = kipp_attention_mix_mma_kv_per_block(n_q, n_kv, head_dim, v_dim, ex.key_maps, head_mix != nullptr);
     if (kvs <= 0 || page_size <= 0 || window < 0 || keep_first < 0) return KIPP_ERR_ARG;
     if ((((uintptr_t)q | (uintptr_t)k_pages | (uintptr_t)v_pages) & 15) != 0) return -3;
@@ -1208,7 +1223,8 @@ extern "C" int kipp_attention_mix_ex(void* out, const void* q, const void* k_pag
     ex.key_maps = 1;
     if (extras != nullptr) ex = *static_cast<const MixExtras*>(extras);
     if (ex.key_maps < 1 || (n_q / n_kv) % ex.key_maps || (ex.diff && ex.key_maps != 2) ||
-        (ex.values_in_keys && v_dim > ex.key_maps * head_dim) || ex.chunk < 0 || (ex.chunk > 0 && window > 0))
+        (ex.values_in_keys && v_dim > ex.key_maps * head_dim) || ex.chunk < 0 || (ex.chunk > 0 && window > 0) ||
+        (ex.slopes && head_mix) || (ex.gate_dims && ex.diff))
         return KIPP_ERR_ARG;
     cudaStream_t s = (cudaStream_t)stream;
     if (dtype == KIPP_DT_F32)

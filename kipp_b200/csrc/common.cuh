@@ -55,6 +55,11 @@ __device__ __forceinline__ float kipp_activation(float z, int kind) {
     }
 }
 
+// gelu in its tanh form as a gate, 0.5 z (1 + tanh(y)) = z / (1 + e^(-2 y)): nothing cancels for z far below 0.
+__device__ __forceinline__ float gelu_tanh_exponent(float z) {
+    return -1.5957691216057308f * fmaf(0.044715f * z * z, z, z);           // -2 sqrt(2/pi) (z + 0.044715 z^3)
+}
+
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);

@@ -6,10 +6,10 @@
 #include "common.cuh"
 #include <algorithm>
 
-// out[t, :] = float(table[ids[t], :]).  The residual stream is float32.
+// out[t, :] = float(table[ids[t], :]) * scale.  The residual stream is float32.
 template <typename TW>
 __global__ void embed_gather_kernel(float* __restrict__ out, const TW* __restrict__ table,
-                                    const int* __restrict__ ids, int hidden, int vocab,
+                                    const int* __restrict__ ids, int hidden, int vocab, float scale,
                                     int* __restrict__ status) {
     pdl_launch_dependents();
     pdl_wait();
@@ -22,22 +22,26 @@ __global__ void embed_gather_kernel(float* __restrict__ out, const TW* __restric
     }
     const TW* row = table + (size_t)id * hidden;
     float* dst = out + (size_t)t * hidden;
-    for (int i = threadIdx.x; i < hidden; i += blockDim.x) dst[i] = to_f32(row[i]);
+    for (int i = threadIdx.x; i < hidden; i += blockDim.x) dst[i] = to_f32(row[i]) * scale;
 }
 
-extern "C" int kipp_embed_gather(float* out, const void* table, int table_dtype, const int* ids,
-                                 int tokens, int hidden, int vocab, int* status, void* stream) {
+extern "C" int kipp_embed_gather_scaled(float* out, const void* table, int table_dtype, const int* ids,
+                                        int tokens, int hidden, int vocab, float scale, int* status, void* stream) {
     if (tokens <= 0) return 0;
     if (hidden <= 0 || vocab <= 0) return KIPP_ERR_ARG;
     cudaStream_t s = (cudaStream_t)stream;
     const int threads = hidden >= 1024 ? 256 : 128;
     if (table_dtype == KIPP_DT_F32)
         return kipp_launch(embed_gather_kernel<float>, dim3(tokens), dim3(threads), 0, s, 1, out,
-                           (const float*)table, ids, hidden, vocab, status);
+                           (const float*)table, ids, hidden, vocab, scale, status);
     if (table_dtype == KIPP_DT_BF16)
         return kipp_launch(embed_gather_kernel<bf16>, dim3(tokens), dim3(threads), 0, s, 1, out,
-                           (const bf16*)table, ids, hidden, vocab, status);
+                           (const bf16*)table, ids, hidden, vocab, scale, status);
     return KIPP_ERR_DTYPE;
+}
+extern "C" int kipp_embed_gather(float* out, const void* table, int table_dtype, const int* ids,
+                                 int tokens, int hidden, int vocab, int* status, void* stream) {
+    return kipp_embed_gather_scaled(out, table, table_dtype, ids, tokens, hidden, vocab, 1.0f, status, stream);
 }
 
 // y[r, i] = x[src(r), i] * rsqrt(mean(x[src(r), :]^2) + eps) * w[i]
@@ -432,6 +436,122 @@ extern "C" int kipp_rmsnorm_scaled_add(float* x, const float* y, const void* w, 
                        1, x, y, w, w_dtype, size, eps, mult, (bf16*)copy_bf16, vec);
 }
 
+// x[r, :] += mult * y[r, :] * rsqrt(mean(y^2) + eps_y) * w_y, and of the new x h[r, :] = x * rsqrt(mean(x^2) + eps_h) * w_h:
+// the norm of a sublayer's OUTPUT joins the stream and the norm of the next sublayer's INPUT leaves the same pass
+// (blocks with a norm on either side of every sublayer).  All float32, h in the compute type; w keeps its storage
+// type.  clear: y is left zeroed for the sublayer that adds its output into it next.  A block per row; a thread keeps
+// its first 4 KEPT values in registers between the three passes over a row, what lies beyond them is read again.
+namespace {
+constexpr int NORM_KEPT = 4;
+__device__ __forceinline__ float4 weights4(const void* w, int w_dtype, int i) {
+    if (w_dtype == KIPP_DT_F32) return *reinterpret_cast<const float4*>(static_cast<const float*>(w) + i);
+    const uint2 v = *reinterpret_cast<const uint2*>(static_cast<const bf16*>(w) + i);
+    return make_float4(__uint_as_float(v.x << 16), __uint_as_float(v.x & 0xffff0000u), __uint_as_float(v.y << 16),
+                       __uint_as_float(v.y & 0xffff0000u));
+}
+__device__ __forceinline__ float squares4(float4 v, float ss) {
+    ss = fmaf(v.x, v.x, ss); ss = fmaf(v.y, v.y, ss); ss = fmaf(v.z, v.z, ss);
+    return fmaf(v.w, v.w, ss);
+}
+__device__ __forceinline__ void store4(float* dst, float4 v) { *reinterpret_cast<float4*>(dst) = v; }
+__device__ __forceinline__ void store4(bf16* dst, float4 v) {
+    const __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+    uint2 pk;
+    pk.x = *reinterpret_cast<const uint32_t*>(&lo);
+    pk.y = *reinterpret_cast<const uint32_t*>(&hi);
+    *reinterpret_cast<uint2*>(dst) = pk;
+}
+
+template <typename TO>
+__global__ void __launch_bounds__(512)
+norm_add_norm_kernel(float* __restrict__ x, float* __restrict__ y, int clear, const void* __restrict__ w_y, int w_y_dtype,
+                     float eps_y, float mult, const void* __restrict__ w_h, int w_h_dtype, float eps_h, TO* __restrict__ h,
+                     int size, int vec) {
+    __shared__ float scratch[32];
+    pdl_launch_dependents();
+    pdl_wait();
+    float* yr = y + (size_t)blockIdx.x * size;
+    float* xr = x + (size_t)blockIdx.x * size;
+    TO* hr = h + (size_t)blockIdx.x * size;
+    const int tid = threadIdx.x, step = blockDim.x;
+    if (!vec) {
+        float ss = 0.f;
+        for (int i = tid; i < size; i += step) ss = fmaf(yr[i], yr[i], ss);
+        const float inv = mult / sqrtf(block_sum(ss, scratch) / (float)size + eps_y);
+        ss = 0.f;
+        for (int i = tid; i < size; i += step) {
+            const float o = fmaf(yr[i] * inv, load_w(w_y, w_y_dtype, i), xr[i]);
+            xr[i] = o;
+            if (clear) yr[i] = 0.f;
+            ss = fmaf(o, o, ss);
+        }
+        const float inv_h = 1.0f / sqrtf(block_sum(ss, scratch) / (float)size + eps_h);
+        for (int i = tid; i < size; i += step) hr[i] = from_f32<TO>(xr[i] * inv_h * load_w(w_h, w_h_dtype, i));
+        return;
+    }
+    float4 keep[NORM_KEPT], stream[NORM_KEPT];
+    float ss = 0.f;
+#pragma unroll
+    for (int j = 0; j < NORM_KEPT; ++j) {
+        const int i = 4 * (tid + j * step);
+        keep[j] = i < size ? *reinterpret_cast<const float4*>(yr + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+        stream[j] = i < size ? *reinterpret_cast<const float4*>(xr + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+        ss = squares4(keep[j], ss);
+    }
+    for (int i = 4 * (tid + NORM_KEPT * step); i < size; i += 4 * step) ss = squares4(*reinterpret_cast<const float4*>(yr + i), ss);
+    const float inv = mult / sqrtf(block_sum(ss, scratch) / (float)size + eps_y);
+    auto joined = [&](float4 v, float4 o, int i) {
+        const float4 w = weights4(w_y, w_y_dtype, i);
+        o.x = fmaf(v.x * inv, w.x, o.x); o.y = fmaf(v.y * inv, w.y, o.y);
+        o.z = fmaf(v.z * inv, w.z, o.z); o.w = fmaf(v.w * inv, w.w, o.w);
+        *reinterpret_cast<float4*>(xr + i) = o;
+        if (clear) *reinterpret_cast<float4*>(yr + i) = make_float4(0.f, 0.f, 0.f, 0.f);
+        return o;
+    };
+    ss = 0.f;
+#pragma unroll
+    for (int j = 0; j < NORM_KEPT; ++j) {
+        const int i = 4 * (tid + j * step);
+        if (i < size) {
+            keep[j] = joined(keep[j], stream[j], i);
+            ss = squares4(keep[j], ss);
+        }
+    }
+    for (int i = 4 * (tid + NORM_KEPT * step); i < size; i += 4 * step)
+        ss = squares4(joined(*reinterpret_cast<const float4*>(yr + i), *reinterpret_cast<const float4*>(xr + i), i), ss);
+    const float inv_h = 1.0f / sqrtf(block_sum(ss, scratch) / (float)size + eps_h);
+    auto normed = [&](float4 o, int i) {
+        const float4 w = weights4(w_h, w_h_dtype, i);
+        store4(hr + i, make_float4(o.x * inv_h * w.x, o.y * inv_h * w.y, o.z * inv_h * w.z, o.w * inv_h * w.w));
+    };
+#pragma unroll
+    for (int j = 0; j < NORM_KEPT; ++j) {
+        const int i = 4 * (tid + j * step);
+        if (i < size) normed(keep[j], i);
+    }
+    for (int i = 4 * (tid + NORM_KEPT * step); i < size; i += 4 * step) normed(*reinterpret_cast<const float4*>(xr + i), i);
+}
+}  // namespace
+
+extern "C" int kipp_norm_add_norm(float* x, float* y, int clear, const void* w_y, int w_y_dtype, float eps_y, float mult,
+                                  const void* w_h, int w_h_dtype, float eps_h, void* h, int h_dtype, int rows, int size,
+                                  void* stream) {
+    if (rows <= 0) return 0;
+    if (size <= 0 || !(eps_y > 0.f) || !(eps_h > 0.f) || (w_y_dtype != KIPP_DT_F32 && w_y_dtype != KIPP_DT_BF16) ||
+        (w_h_dtype != KIPP_DT_F32 && w_h_dtype != KIPP_DT_BF16))
+        return KIPP_ERR_ARG;
+    const int vec = size % 4 == 0 && (((uintptr_t)x | (uintptr_t)y | (uintptr_t)h | (uintptr_t)w_y | (uintptr_t)w_h) & 15) == 0;
+    const dim3 grid((unsigned)rows), block(size >= 4096 ? 512 : size >= 1024 ? 256 : 128);
+    cudaStream_t s = (cudaStream_t)stream;
+    if (h_dtype == KIPP_DT_F32)
+        return kipp_launch(norm_add_norm_kernel<float>, grid, block, 0, s, 1, x, y, clear, w_y, w_y_dtype, eps_y, mult, w_h, w_h_dtype,
+                           eps_h, (float*)h, size, vec);
+    if (h_dtype == KIPP_DT_BF16)
+        return kipp_launch(norm_add_norm_kernel<bf16>, grid, block, 0, s, 1, x, y, clear, w_y, w_y_dtype, eps_y, mult, w_h, w_h_dtype,
+                           eps_h, (bf16*)h, size, vec);
+    return KIPP_ERR_DTYPE;
+}
+
 // x *= scale over n float32 values (logits of a head with a scale).
 __global__ void scale_f32_kernel(float* __restrict__ x, long long n, float scale) {
     pdl_launch_dependents();
@@ -608,8 +728,9 @@ extern "C" int kipp_sum_streams(float* out, const float* x, long long stride, in
 }
 
 // ---------------------------------------------------------------------------------------------
-// A gated feed-forward's activation with limits: g = min(gate + bg, limit), u = clamp(up + bu, -limit, limit),
-// out = g * sigmoid(alpha * g) * (u + 1), in float32 from the projection's stored values.  gate of element i
+// A gated feed-forward's activation: g = min(gate + bg, limit), u = clamp(up + bu, -limit, limit),
+// out = act(g) (u + up_add) with act(g) = g sigmoid(alpha g) (act -1), or gelu in its tanh form (act 2), in
+// float32 from the projection's stored values.  gate of element i
 // is proj[r, gate_off + i * step], up proj[r, up_off + i * step].  limit <= 0: no limits.  row_gate given:
 // the whole row is also multiplied by sigmoid(row_gate[r]) (a gate per token on the part's output:
 // applied here, before the linear down projection).
@@ -617,8 +738,8 @@ namespace {
 template <typename T>
 __global__ void glu_limited_kernel(T* __restrict__ out, long long ld_out, const T* __restrict__ proj, long long ld_proj,
                                    int rows, int n, int gate_off, int up_off, int step, const float* __restrict__ bias_gate,
-                                   const float* __restrict__ bias_up, int bias_step, float limit, float alpha,
-                                   const float* __restrict__ row_gate) {
+                                   const float* __restrict__ bias_up, int bias_step, int act, float limit, float alpha,
+                                   float up_add, const float* __restrict__ row_gate) {
     pdl_launch_dependents();
     pdl_wait();
     const long long idx = (long long)blockIdx.x * blockDim.x + threadIdx.x;
@@ -633,7 +754,7 @@ __global__ void glu_limited_kernel(T* __restrict__ out, long long ld_out, const 
         g = fminf(g, limit);
         u = fminf(fmaxf(u, -limit), limit);
     }
-    float v = g / (1.0f + expf(-alpha * g)) * (u + 1.0f);
+    float v = g / (1.0f + expf(act == 2 ? gelu_tanh_exponent(g) : -alpha * g)) * (u + up_add);
     if (row_gate != nullptr) v *= 1.0f / (1.0f + expf(-row_gate[r]));
     out[r * ld_out + i] = from_f32<T>(v);
 }
@@ -655,19 +776,20 @@ __global__ void softcap_f32_kernel(float* __restrict__ x, long long n, float cap
 
 extern "C" int kipp_glu_limited(void* out, long long ld_out, const void* proj, long long ld_proj, int dtype, int rows, int n,
                                 int gate_off, int up_off, int step, const float* bias_gate, const float* bias_up,
-                                int bias_step, float limit, float alpha, const float* row_gate, void* stream) {
+                                int bias_step, int act, float limit, float alpha, float up_add, const float* row_gate,
+                                void* stream) {
     if (rows <= 0 || n <= 0) return 0;
-    if (step <= 0 || gate_off < 0 || up_off < 0) return KIPP_ERR_ARG;
+    if (step <= 0 || gate_off < 0 || up_off < 0 || (act != -1 && act != 2)) return KIPP_ERR_ARG;
     const long long total = (long long)rows * n, blocks = (total + 255) / 256;
     if (blocks > 0x7fffffffLL) return KIPP_ERR_ARG;
     if (dtype == KIPP_DT_F32)
         return kipp_launch(glu_limited_kernel<float>, dim3((unsigned)blocks), dim3(256), 0, (cudaStream_t)stream, 1, (float*)out,
                            ld_out, (const float*)proj, ld_proj, rows, n, gate_off, up_off, step, bias_gate, bias_up, bias_step,
-                           limit, alpha, row_gate);
+                           act, limit, alpha, up_add, row_gate);
     if (dtype == KIPP_DT_BF16)
         return kipp_launch(glu_limited_kernel<bf16>, dim3((unsigned)blocks), dim3(256), 0, (cudaStream_t)stream, 1, (bf16*)out,
                            ld_out, (const bf16*)proj, ld_proj, rows, n, gate_off, up_off, step, bias_gate, bias_up, bias_step,
-                           limit, alpha, row_gate);
+                           act, limit, alpha, up_add, row_gate);
     return KIPP_ERR_DTYPE;
 }
 

@@ -300,12 +300,16 @@ struct Params {
     const int* group_tiles;
     // The gated epilogue (EPI_SWIGLU) in its general form; glu_alpha 0 is the plain silu(gate) * up.
     // Else: g = min(gate + b, limit), u = clamp(up + b', -limit, limit) (limit 0: none; the biases lie
-    // interleaved like the weight rows, or are null), g sigmoid(alpha g) (u + 1), times
-    // sigmoid(glu_row_gate[token]) where that is given.
-    float glu_alpha, glu_limit;
+    // interleaved like the weight rows, or are null), act(g) (u + glu_up_add) with act(g) = g sigmoid(alpha g),
+    // or gelu in its tanh form where glu_act is GLU_GELU_TANH, times sigmoid(glu_row_gate[token]) where
+    // that is given.
+    int glu_act;
+    float glu_alpha, glu_limit, glu_up_add;
     const float* glu_bias;
     const float* glu_row_gate;
 };
+
+constexpr int GLU_GELU_TANH = 2;      // the code of kipp_activation
 
 // gate and up of one hidden element (f: the gate's feature index, even) of token t
 __device__ __forceinline__ float glu_of(const Params& p, float g, float u, int f, int t) {
@@ -318,7 +322,8 @@ __device__ __forceinline__ float glu_of(const Params& p, float g, float u, int f
         g = fminf(g, p.glu_limit);
         u = fminf(fmaxf(u, -p.glu_limit), p.glu_limit);
     }
-    float r = g / (1.0f + expf(-p.glu_alpha * g)) * (u + 1.0f);
+    float r = (p.glu_act == GLU_GELU_TANH ? __fdividef(g, 1.0f + __expf(gelu_tanh_exponent(g)))
+                                          : g / (1.0f + expf(-p.glu_alpha * g))) * (u + p.glu_up_add);
     if (p.glu_row_gate != nullptr) r *= 1.0f / (1.0f + expf(-p.glu_row_gate[t]));
     return r;
 }
@@ -1606,7 +1611,8 @@ extern "C" int kipp_gemm_tc_fold(void* C, int out_dtype, const void* X, const vo
 
 // The general form of the gated epilogue (see Params::glu_alpha): alpha 0 leaves the plain SwiGLU.
 struct kipp_gemm_glu {
-    float alpha, limit;
+    int act;                    // -1: g sigmoid(alpha g); GLU_GELU_TANH: gelu in its tanh form
+    float alpha, limit, up_add;
     const float* bias;          // [features] float32, interleaved like the weight rows, or null
     const float* row_gate;      // [tokens] float32: the row is also multiplied by sigmoid of it, or null
 };
@@ -1617,6 +1623,7 @@ namespace {
 thread_local const kipp_gemm_glu* glu_in_flight = nullptr;
 void apply_glu(Params& p) {
     if (glu_in_flight == nullptr || p.epilogue != EPI_SWIGLU) return;
+    p.glu_act = glu_in_flight->act; p.glu_up_add = glu_in_flight->up_add;
     p.glu_alpha = glu_in_flight->alpha; p.glu_limit = glu_in_flight->limit;
     p.glu_bias = glu_in_flight->bias; p.glu_row_gate = glu_in_flight->row_gate;
 }
@@ -1820,7 +1827,8 @@ extern "C" int kipp_gemm_tc_grouped(void* C, int out_dtype, const void* X, const
 extern "C" int kipp_gemm_tc_glu(void* C, int out_dtype, const void* X, const void* W, int tokens, int features, int K,
                                 long long ldx, long long ldw, long long ldc, const kipp_gemm_norm_fold* fold,
                                 const kipp_gemm_glu* glu, int* status, void* stream) {
-    if (glu == nullptr || !(glu->alpha > 0.f) || glu->limit < 0.f) return KIPP_ERR_ARG;
+    if (glu == nullptr || !(glu->alpha > 0.f) || glu->limit < 0.f || (glu->act != -1 && glu->act != GLU_GELU_TANH))
+        return KIPP_ERR_ARG;
     GluScope scope(glu);
     return gemm_tc_run(C, out_dtype, X, W, tokens, features, K, ldx, ldw, ldc, EPI_SWIGLU, 0, 0, 0, fold, nullptr, status, stream);
 }
@@ -1829,7 +1837,8 @@ extern "C" int kipp_gemm_tc_grouped_glu(void* C, int out_dtype, const void* X, c
                                         long long ldx, long long ldc, int groups, const int* group_of_tile,
                                         const int* group_tiles, int tile_rows, const kipp_gemm_glu* glu, int* status,
                                         void* stream) {
-    if (glu == nullptr || !(glu->alpha > 0.f) || glu->limit < 0.f || glu->bias != nullptr || glu->row_gate != nullptr)
+    if (glu == nullptr || !(glu->alpha > 0.f) || glu->limit < 0.f || (glu->act != -1 && glu->act != GLU_GELU_TANH) ||
+        glu->bias != nullptr || glu->row_gate != nullptr)
         return KIPP_ERR_ARG;
     GluScope scope(glu);
     return kipp_gemm_tc_grouped(C, out_dtype, X, W, rows, features, K, ldx, ldc, groups, EPI_SWIGLU, group_of_tile, group_tiles,

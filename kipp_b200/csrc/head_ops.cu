@@ -7,6 +7,7 @@
 //   norm       division of the head by its root mean square (eps inside the root), times a
 //              weight of the head's size; or (norm_all) division of ALL heads of the segment by the
 //              root mean square of the whole run of heads x dim columns, times a weight of that size;
+//              or (unit_norm) the division alone, without a weight;
 //   rotation   of the dims [rot_off, rot_off + rot) of the head: pair (i, i + rot/2) turns by the
 //              angle of the step's (cos, sin) table for the token; or (interleaved) pair (2i, 2i + 1);
 //   target     a row of an activation buffer (queries), or the token's slot in the key or value
@@ -34,6 +35,7 @@ struct HeadSegment {
     int heads_per_row;                       // pages: this many heads side by side in one page row
     int norm_all;                            // 1: one mean square over all heads of the segment, norm_w [heads * dim]
     int interleaved;                         // 1: the rotation pairs dim 2i with dim 2i + 1
+    int unit_norm;                           // 1: the norm's division without a weight (norm_w null)
     const float* bias;                       // [heads * dim] or null
     const float* norm_w;                     // [dim] ([heads * dim] with norm_all) or null
     const float* cos_sin;                    // [tokens, rot / 2, 2] or null
@@ -90,7 +92,8 @@ head_segments_kernel(const SegmentArgs a, int* __restrict__ status) {
 
     float inv = 1.f;
     const float* norm_w = g.norm_w;
-    if (g.norm_w != nullptr && g.norm_all) {
+    const bool divided = g.norm_w != nullptr || g.unit_norm;
+    if (divided && g.norm_all) {
         // every warp of the token sums the whole run of heads in the same order
         const T* all = static_cast<const T*>(a.src) + (size_t)t * a.ld_src + g.src_off;
         const int n = g.heads * D;
@@ -114,8 +117,8 @@ head_segments_kernel(const SegmentArgs a, int* __restrict__ status) {
             }
         }
         inv = 1.0f / sqrtf(warp_sum(ss) / (float)n + a.eps);
-        norm_w = g.norm_w + (size_t)hh * D;
-    } else if (g.norm_w != nullptr) {
+        if (norm_w != nullptr) norm_w += (size_t)hh * D;
+    } else if (divided) {
         float ss = 0.f;
         for (int i = lane; i < D; i += 32) {
             const float v = to_f32(src[i]) + (bias ? bias[i] : 0.f);
@@ -128,7 +131,8 @@ head_segments_kernel(const SegmentArgs a, int* __restrict__ status) {
                                                            : nullptr;
     auto value = [&](int i) {
         float v = to_f32(src[i]) + (bias ? bias[i] : 0.f);
-        if (norm_w != nullptr) v = v * inv * norm_w[i];
+        if (divided) v = v * inv;
+        if (norm_w != nullptr) v *= norm_w[i];
         return v;
     };
     for (int i = lane; i < D; i += 32) {

@@ -21,6 +21,7 @@
 #include "expert_parts.hpp"
 #include "zasudra.hpp"
 #include "zunilorn.hpp"
+#include "panolorn.hpp"
 
 namespace kipp {
 
@@ -353,17 +354,17 @@ inline void AttentionMixer::forward(StepContext& ctx, const LayerRun& run, int m
                 fail(KIPP_E_CONFIG, "attention: a mixer with shared_kv runs with writes_cache false, any other with true");
             HeadSegment seg[3];
             int n = 0;
-            const float* qw = qk_norm_ ? static_cast<const float*>(q_norm_) : nullptr;
+            const float* qw = qk_norm_ ? static_cast<const float*>(q_norm_) : nullptr;      // (null with unit_norm)
             const float* kw = qk_norm_ ? static_cast<const float*>(k_norm_) : nullptr;
             HeadSegment& sq = seg[n++];
             sq.src_off = 0; sq.heads = heads_; sq.dim = head_dim_; sq.src_stride = head_dim_;
-            sq.norm_w = qw; sq.norm_all = opt_.norm_whole ? 1 : 0;
+            sq.norm_w = qw; sq.norm_all = opt_.norm_whole ? 1 : 0; sq.unit_norm = opt_.unit_norm ? 1 : 0;
             sq.rot = rot; sq.cos_sin = cos_sin; sq.interleaved = opt_.interleaved ? 1 : 0;
             sq.target = 0; sq.dst = q; sq.ld_dst = q_dim_; sq.dst_stride = head_dim_;
             if (k_cols_) {
                 HeadSegment& sk = seg[n++];
                 sk.src_off = q_dim_; sk.heads = kv_heads_; sk.dim = head_dim_; sk.src_stride = head_dim_;
-                sk.norm_w = kw; sk.norm_all = opt_.norm_whole ? 1 : 0;
+                sk.norm_w = kw; sk.norm_all = opt_.norm_whole ? 1 : 0; sk.unit_norm = opt_.unit_norm ? 1 : 0;
                 sk.rot = rot; sk.cos_sin = cos_sin; sk.interleaved = opt_.interleaved ? 1 : 0;
                 sk.target = 1; sk.heads_per_row = 1;
                 HeadSegment& sv = seg[n++];                              // the values: W_v's rows, or the keys as projected
@@ -375,7 +376,9 @@ inline void AttentionMixer::forward(StepContext& ctx, const LayerRun& run, int m
                               m.entry_of_token, T, write, eps_);
             extras.sink = sink_;
             extras.chunk = opt_.chunk;
-            if (opt_.head_gate) {
+            extras.slopes = slopes_;
+            extras.gate_dims = opt_.element_gate ? 1 : 0;
+            if (g_cols_) {
                 extras.gate = static_cast<const char*>(qkv) + (size_t)(q_dim_ + k_cols_ + v_cols_) * es;
                 extras.ld_gate = qkv_cols;
                 extras.gate_off = 0;
@@ -1196,6 +1199,7 @@ inline void Engine::debug_part(const StepEntryView* entries, int n, int run_inde
     ParallelBlock* shared_norm = dynamic_cast<ParallelBlock*>(block);
     OutputNormBlock* out_norm = dynamic_cast<OutputNormBlock*>(block);
     HyperConnectionBlock* hyper = dynamic_cast<HyperConnectionBlock*>(block);
+    SandwichNormBlock* sandwich = dynamic_cast<SandwichNormBlock*>(block);
     if (which == "embedding") {
         for (auto& e : plan_->embedding) e.second->forward(ctx, residual);
     } else if (which == "feed_forward" && out_norm != nullptr) {
@@ -1204,6 +1208,9 @@ inline void Engine::debug_part(const StepEntryView* entries, int n, int run_inde
     } else if (which == "feed_forward" && hyper != nullptr) {
         if (hyper->feed_forward() == nullptr) fail(KIPP_E_ARGUMENT, "the block has no feed-forward");
         hyper->feed_forward()->forward(ctx, input, residual);
+    } else if (which == "feed_forward" && sandwich != nullptr) {
+        if (sandwich->feed_forward() == nullptr) fail(KIPP_E_ARGUMENT, "the block has no feed-forward");
+        sandwich->feed_forward()->forward(ctx, input, residual);
     } else if (which == "input_norm" && shared_norm != nullptr) {
         shared_norm->norm()->forward(ctx, residual, output, nullptr, T);
     } else if (which == "feed_forward" && shared_norm != nullptr) {

@@ -4,12 +4,12 @@
 //                    weights are the softmax over the chosen logits only; the output is the weighted
 //                    sum of the chosen experts' W_down act(W_up h)
 //
-//
-// Options: routing by scores (routing "scores": s = softmax(z) over all outputs of the router, the choice
-// by s + a learned correction per output, the weights s of the chosen divided by their sum and times
-// weight_scale); identity experts (identity n: the router has n more outputs whose expert hands the
-// token's input on, without tensors); gated experts (gated: W_down (g sigmoid(alpha g) (u + 1)) with
-// g = min(W_gate h, limit), u = clamp(W_up h, -limit, limit)); a shared feed-forward (shared: any
+// Options: routing by scores (routing "scores": s = softmax(z) over all outputs of the router; "sigmoid_scores":
+// s = sigmoid(z); the choice by s + a learned correction per output, the weights s of the chosen divided by
+// their sum (renormalize false: as they are) and times weight_scale); the weight on the expert's INPUT (weight_on_input:
+// the output is the sum of expert(w h)); identity experts (identity n: the router has n more outputs whose expert hands the
+// token's input on, without tensors); gated experts (gated: W_down (act(g) (u + up_add)) with
+// g = min(W_gate h, limit), u = clamp(W_up h, -limit, limit), act(g) = g sigmoid(alpha g) or gelu (gate_activation)); a shared feed-forward (shared: any
 // feed-forward part, under shared_prefix) that runs for every token and is added.
 //
 // Sizes, the number of experts and of choices, the activation and every tensor name are parameters
@@ -24,16 +24,22 @@ class ExpertMixture : public FeedForward {
 public:
     ExpertMixture(const Json& j, const BuildContext& ctx) {
         const std::string routing = j.get_string("routing", "chosen_softmax");
-        if (routing != "chosen_softmax" && routing != "scores")
-            fail(KIPP_E_CONFIG, "expert_mixture: routing must be chosen_softmax or scores, not '" + routing + "'");
-        by_scores_ = routing == "scores";
+        if (routing != "chosen_softmax" && routing != "scores" && routing != "sigmoid_scores")
+            fail(KIPP_E_CONFIG, "expert_mixture: routing must be chosen_softmax, scores or sigmoid_scores, not '" + routing + "'");
+        by_scores_ = routing != "chosen_softmax";
+        sigmoid_ = routing == "sigmoid_scores";
+        renormalize_ = j.get_bool("renormalize", true);
+        weight_on_input_ = j.get_bool("weight_on_input", false);
+        if (!renormalize_ && !by_scores_) fail(KIPP_E_CONFIG, "expert_mixture: renormalize false goes with routing by scores");
         identity_ = (int)j.get_int("identity", 0);
         weight_scale_ = (float)j.get_double("weight_scale", 1.0);
         correction_ = j.get_bool("correction", false);
         gated_ = j.get_bool("gated", false);
-        limit_ = (float)j.get_double("limit", 0.0);
-        alpha_ = (float)j.get_double("alpha", 1.0);
-        if (identity_ < 0 || limit_ < 0.f) fail(KIPP_E_CONFIG, "expert_mixture: identity and limit must not be negative");
+        glu_.limit = (float)j.get_double("limit", 0.0);
+        glu_.alpha = (float)j.get_double("alpha", 1.0);
+        glu_.up_add = (float)j.get_double("up_add", 1.0);
+        glu_.act = gate_activation(j, "gate_activation");
+        if (identity_ < 0 || glu_.limit < 0.f) fail(KIPP_E_CONFIG, "expert_mixture: identity and limit must not be negative");
         if ((identity_ > 0 || correction_) && !by_scores_)
             fail(KIPP_E_CONFIG, "expert_mixture: identity experts and a correction go with routing by scores");
         if (const Json* sh = j.find("shared"); sh && !sh->is_null()) {
@@ -110,16 +116,17 @@ public:
     void route(StepContext& ctx, int* expert_of, float* weight_of, const void* h, int T) {
         if (by_scores_)
             ctx.ops->moe_route_scores(expert_of, weight_of, h, hidden_, ctx.dtype, router_, bias_, T, hidden_, outputs_, experts_,
-                                      top_, weight_scale_);
+                                      top_, sigmoid_, renormalize_, weight_scale_);
         else
             ctx.ops->moe_route(expert_of, weight_of, h, hidden_, ctx.dtype, router_, bias_, T, hidden_, experts_, top_);
     }
     void combine(StepContext& ctx, float* residual, const float* rows, const float* weight_of, const int* expert_of,
                  const void* h, int T, const int* place) {
         if (identity_ > 0)
-            ctx.ops->moe_combine_identity(residual, rows, weight_of, expert_of, h, hidden_, ctx.dtype, T, hidden_, top_, place);
+            ctx.ops->moe_combine_identity(residual, rows, weight_of, expert_of, h, hidden_, ctx.dtype, T, hidden_, top_, place,
+                                          weight_on_input_);
         else
-            ctx.ops->moe_combine(residual, rows, weight_of, T, hidden_, top_, place);
+            ctx.ops->moe_combine(residual, rows, weight_on_input_ ? nullptr : weight_of, T, hidden_, top_, place);
     }
     void forward(StepContext& ctx, const void* h, float* residual) override {
         const int T = ctx.tokens(), pairs = T * top_;
@@ -150,12 +157,9 @@ public:
             float* rows = ctx.workspace->get<float>("moe_output_rows", (size_t)rows_cap * hidden_);
             route(ctx, expert_of, weight_of, h, T);
             ops.moe_padded_lists(place, tile_expert, n_tiles, expert_of, pairs, experts_, tile);
-            ops.moe_gather_rows(in, h, hidden_, place, pairs, top_, hidden_);
+            ops.moe_gather_rows(in, h, hidden_, place, pairs, top_, hidden_, weight_on_input_ ? weight_of : nullptr);
             if (gated_) {                           // the gated activation in the grouped product's epilogue
-                Ops::Glu glu;
-                glu.alpha = alpha_;
-                glu.limit = limit_;
-                ops.gemm_grouped_glu(act, ctx.dtype, inter_, in, hidden_, w_up_, rows_cap, up_rows_, hidden_, experts_, glu,
+                ops.gemm_grouped_glu(act, ctx.dtype, inter_, in, hidden_, w_up_, rows_cap, up_rows_, hidden_, experts_, glu_,
                                      tile_expert, n_tiles, tile);
             } else {
                 ops.gemm_grouped(act, ctx.dtype, inter_, in, hidden_, w_up_, rows_cap, inter_, hidden_, experts_, act_, tile_expert,
@@ -177,18 +181,17 @@ public:
         route(ctx, expert_of, weight_of, h, T);
         ops.moe_lists(sorted, tiles, n_tiles, expert_of, pairs, experts_);
         const long long one = (long long)inter_ * hidden_;
+        const float* in_weight = weight_on_input_ ? weight_of : nullptr;
         // up: the rows of a tile are gathered from their tokens; the hidden rows lie in sorted order
         if (gated_) {
             void* both = ctx.workspace->buffer("moe_gate_up", (size_t)pairs * up_rows_ * ctx.element());
             ops.moe_gemm(both, ctx.dtype, up_rows_, h, hidden_, w_up_, (long long)up_rows_ * hidden_, dtype_, up_rows_, hidden_, top_,
-                         true, false, -1, sorted, tiles, n_tiles, pairs, experts_);
-            Ops::Glu glu;
-            glu.alpha = alpha_;
-            glu.limit = limit_;
-            ops.glu_limited(act, inter_, both, up_rows_, ctx.dtype, pairs, inter_, glu);
-        } else
-        ops.moe_gemm(act, ctx.dtype, inter_, h, hidden_, w_up_, one, dtype_, inter_, hidden_, top_, true, false, act_, sorted,
-                     tiles, n_tiles, pairs, experts_);
+                         true, false, -1, sorted, tiles, n_tiles, pairs, experts_, in_weight);
+            ops.glu_limited(act, inter_, both, up_rows_, ctx.dtype, pairs, inter_, glu_);
+        } else {
+            ops.moe_gemm(act, ctx.dtype, inter_, h, hidden_, w_up_, one, dtype_, inter_, hidden_, top_, true, false, act_, sorted,
+                         tiles, n_tiles, pairs, experts_, in_weight);
+        }
         // down: one float32 row per (token, choice) pair, at the pair's own place
         ops.moe_gemm(rows, F32, hidden_, act, inter_, w_down_, one, dtype_, hidden_, inter_, top_, false, true, -1, sorted,
                      tiles, n_tiles, pairs, experts_);
@@ -204,7 +207,9 @@ private:
     int hidden_ = 0, inter_ = 0, experts_ = 0, top_ = 0, act_ = 0, dtype_ = BF16;
     int identity_ = 0, outputs_ = 0, up_rows_ = 0;
     bool router_bias_ = true, by_scores_ = false, correction_ = false, gated_ = false;
-    float weight_scale_ = 1.f, limit_ = 0.f, alpha_ = 1.f;
+    bool sigmoid_ = false, renormalize_ = true, weight_on_input_ = false;
+    float weight_scale_ = 1.f;
+    Ops::Glu glu_;
     std::unique_ptr<FeedForward> shared_;
     std::string shared_prefix_;
     std::string expert_prefix_;

@@ -90,7 +90,9 @@ struct AttentionExtras {
     int gate_off = 0;
     int chunk = 0;                         // > 0: a query sees the keys j <= p of its own block of `chunk` positions
     float softcap = 0.f;                   // > 0: a scaled score s becomes softcap * tanh(s / softcap)
-    bool any() const { return sink || key_maps != 1 || values_in_keys || diff || gate || chunk || softcap > 0.f; }
+    int gate_dims = 0;                     // 1: the gate is a number per element of every head
+    const float* slopes = nullptr;         // [n_q]: the score of keys at distance d loses slopes[h] * d
+    bool any() const { return sink || key_maps != 1 || values_in_keys || diff || gate || chunk || softcap > 0.f || slopes; }
 };
 
 // A run of heads in a projection row and what becomes of them (the layout is the kernel
@@ -103,6 +105,7 @@ struct HeadSegment {
     int heads_per_row = 1;
     int norm_all = 0;                      // 1: one mean square over all heads of the segment, norm_w [heads * dim]
     int interleaved = 0;                   // 1: the rotation pairs dim 2i with dim 2i + 1
+    int unit_norm = 0;                     // 1: the norm's division without a weight
     const float* bias = nullptr;
     const float* norm_w = nullptr;
     const float* cos_sin = nullptr;
@@ -126,10 +129,10 @@ public:
     static constexpr int PREFILL_TC_MIN_TOKENS = 64;   // shorter portions waste a 128-row tile
 
     void embed_gather(float* out, const void* table, int table_dtype, const int* ids, int tokens, int hidden,
-                      int vocab) {
-        using Fn = int (*)(float*, const void*, int, const int*, int, int, int, int*, void*);
-        static Fn f = kernel_symbol<Fn>("elementwise", "kipp_embed_gather");
-        run(f(out, table, table_dtype, ids, tokens, hidden, vocab, status, stream), "embed_gather");
+                      int vocab, float scale = 1.f) {
+        using Fn = int (*)(float*, const void*, int, const int*, int, int, int, float, int*, void*);
+        static Fn f = kernel_symbol<Fn>("elementwise", "kipp_embed_gather_scaled");
+        run(f(out, table, table_dtype, ids, tokens, hidden, vocab, scale, status, stream), "embed_gather");
     }
 
     // out[r] = x[rows[r] or r] * rsqrt(mean(x^2) + eps) * weight, float32 arithmetic.
@@ -502,6 +505,15 @@ public:
         static Fn f = kernel_symbol<Fn>("elementwise", "kipp_rmsnorm_scaled_add");
         run(f(x, y, w, w_dtype, rows, size, eps, mult, copy_bf16, stream), "rmsnorm_scaled_add");
     }
+    // x += mult * rmsnorm_y(y), and h = rmsnorm_h(the new x) in the same pass; clear: y is left zeroed
+    void norm_add_norm(float* x, float* y, bool clear, const void* w_y, int w_y_dtype, float eps_y, float mult, const void* w_h,
+                       int w_h_dtype, float eps_h, void* h, int h_dtype, int rows, int size) {
+        using Fn = int (*)(float*, float*, int, const void*, int, float, float, const void*, int, float, void*, int, int, int,
+                           void*);
+        static Fn f = kernel_symbol<Fn>("elementwise", "kipp_norm_add_norm");
+        run(f(x, y, clear ? 1 : 0, w_y, w_y_dtype, eps_y, mult, w_h, w_h_dtype, eps_h, h, h_dtype, rows, size, stream),
+            "norm_add_norm");
+    }
     // Hyper-connections (elementwise.cu): the residual stream as `streams` copies, `stride` floats apart.
     // y given: x_t <- sum_s mix[s, t] x_s + mult out_w[t] y; h given: h = rmsnorm(sum_s in_w[s] x_s).
     static int hyper_connection_max_streams() {
@@ -525,22 +537,28 @@ public:
         static Fn f = kernel_symbol<Fn>("elementwise", "kipp_sum_streams");
         run(f(out, x, stride, streams, n, stream), "sum_streams");
     }
-    // The gated activation with limits, g sigmoid(alpha g) (u + 1) with g = min(gate + b, limit) and
-    // u = clamp(up + b', -limit, limit): `bias` [2 n] float32 interleaved (gate_0, up_0, ...) or null;
-    // row_gate [rows] float32 or null: the row is also multiplied by sigmoid of it.
+    // The gated activation act(g) (u + up_add) with g = min(gate + b, limit) and u = clamp(up + b', -limit, limit)
+    // (limit 0: none): act -1 is g sigmoid(alpha g), ACT_GELU_TANH gelu in its tanh form; `bias` [2 n] float32
+    // interleaved (gate_0, up_0, ...) or null; row_gate [rows] float32 or null: the row is also multiplied by
+    // sigmoid of it.
     struct Glu {
-        float alpha = 1.f, limit = 0.f;
+        int act = -1;
+        float alpha = 1.f, limit = 0.f, up_add = 1.f;
         const float* bias = nullptr;
         const float* row_gate = nullptr;
+        // silu(gate) * up, what the products' plain gated epilogue does
+        bool plain() const {
+            return act == -1 && alpha == 1.f && limit == 0.f && up_add == 0.f && bias == nullptr && row_gate == nullptr;
+        }
     };
     // out[r, i] = glu(proj[r, 2 i], proj[r, 2 i + 1]): the stored product's neighbouring columns
     void glu_limited(void* out, long long ld_out, const void* proj, long long ld_proj, int dtype, int rows, int n,
                      const Glu& glu) {
         using Fn = int (*)(void*, long long, const void*, long long, int, int, int, int, int, int, const float*, const float*,
-                           int, float, float, const float*, void*);
+                           int, int, float, float, float, const float*, void*);
         static Fn f = kernel_symbol<Fn>("elementwise", "kipp_glu_limited");
-        run(f(out, ld_out, proj, ld_proj, dtype, rows, n, 0, 1, 2, glu.bias, glu.bias ? glu.bias + 1 : nullptr, 2, glu.limit,
-              glu.alpha, glu.row_gate, stream),
+        run(f(out, ld_out, proj, ld_proj, dtype, rows, n, 0, 1, 2, glu.bias, glu.bias ? glu.bias + 1 : nullptr, 2, glu.act,
+              glu.limit, glu.alpha, glu.up_add, glu.row_gate, stream),
             "glu_limited");
     }
     // out [M, N / 2] = glu of a [M, K] x w [N, K]^T whose rows are interleaved (gate_0, up_0, gate_1, ...):
@@ -549,6 +567,11 @@ public:
     void gemm_glu(void* out, int out_dtype, long long ldc, const void* a, long long lda, const void* w, long long ldw, int dtype,
                   int M, int N, int K, const Glu& glu, const NormFold* fold, void* scratch, long long ld_scratch) {
         if (M <= 0 || N <= 0) return;
+        if (gemm_tc_ok(dtype, a, lda, w, ldw) && out_dtype == dtype && glu.plain()) {
+            gemm(out, out_dtype, ldc, a, lda, w, ldw, dtype, M, N, K, EPI_SWIGLU, fold);
+            ++glu_epilogues;
+            return;
+        }
         if (gemm_tc_ok(dtype, a, lda, w, ldw) && out_dtype == dtype) {
             using Fn = int (*)(void*, int, const void*, const void*, int, int, int, long long, long long, long long,
                                const NormFold*, const Glu*, int*, void*);
@@ -565,6 +588,16 @@ public:
     // The grouped product (gemm_grouped) with the gated epilogue: every group's rows interleaved.
     void gemm_grouped_glu(void* out, int out_dtype, long long ldc, const void* a, long long lda, const void* w, int rows, int N,
                           int K, int groups, const Glu& glu, const int* expert_of_tile, const int* n_tiles, int tile_rows) {
+        if (glu.plain()) {
+            using Fp = int (*)(void*, int, const void*, const void*, int, int, int, long long, long long, int, int, const int*,
+                               const int*, int, int*, void*);
+            static Fp plain = kernel_symbol<Fp>("gemm_tc", "kipp_gemm_tc_grouped");
+            run(plain(out, out_dtype, a, w, rows, N, K, lda, ldc, groups, (int)EPI_SWIGLU, expert_of_tile, n_tiles, tile_rows, status,
+                      stream),
+                "gemm_tc_grouped", 1, profiling ? format("gemm_tc_grouped %d x %d glu", N, K).c_str() : nullptr);
+            ++glu_epilogues;
+            return;
+        }
         using Fn = int (*)(void*, int, const void*, const void*, int, int, int, long long, long long, int, const int*, const int*,
                            int, const Glu*, int*, void*);
         static Fn f = kernel_symbol<Fn>("gemm_tc", "kipp_gemm_tc_grouped_glu");
@@ -666,25 +699,29 @@ public:
             "ssd_scan", taps > 1 ? 5 : 4);
     }
 
-    // Routing by scores (moe.cu): softmax over all `outputs`, the choice by score + correction, weights
-    // score / sum of the chosen x weight_scale; outputs from `experts` on are identity experts (negative ids).
+    // Routing by scores (moe.cu): softmax over all `outputs` (sigmoid: of each), the choice by score + correction,
+    // weights score / sum of the chosen (renormalize; else the score) x weight_scale; outputs from `experts` on are
+    // identity experts (negative ids).
     void moe_route_scores(int* expert_of, float* weight_of, const void* h, long long ldh, int dtype, const float* router,
                           const float* correction, int tokens, int hidden, int outputs, int experts, int top,
-                          float weight_scale) {
-        using Fn = int (*)(int*, float*, const void*, long long, int, const float*, const float*, int, int, int, int, int, float,
-                           void*);
+                          bool sigmoid, bool renormalize, float weight_scale) {
+        using Fn = int (*)(int*, float*, const void*, long long, int, const float*, const float*, int, int, int, int, int, int, int,
+                           float, void*);
         static Fn f = kernel_symbol<Fn>("moe", "kipp_moe_route_scores");
-        run(f(expert_of, weight_of, h, ldh, dtype, router, correction, tokens, hidden, outputs, experts, top, weight_scale,
-              stream),
+        run(f(expert_of, weight_of, h, ldh, dtype, router, correction, tokens, hidden, outputs, experts, top, sigmoid ? 1 : 0,
+              renormalize ? 1 : 0, weight_scale, stream),
             "moe_route");
     }
-    // The combine where pairs with a negative expert id stand for the token's own input h.
+    // The combine where pairs with a negative expert id stand for the token's own input h (weighted: the
+    // other pairs' rows carry their weight already).
     void moe_combine_identity(float* y, const float* rows, const float* weight_of, const int* expert_of, const void* h,
-                              long long ldh, int dtype, int tokens, int hidden, int top, const int* place_of_pair = nullptr) {
+                              long long ldh, int dtype, int tokens, int hidden, int top, const int* place_of_pair = nullptr,
+                              bool weighted = false) {
         using Fn = int (*)(float*, const float*, const float*, const int*, const void*, long long, int, int, int, int,
-                           const int*, void*);
+                           const int*, int, void*);
         static Fn f = kernel_symbol<Fn>("moe", "kipp_moe_combine_identity");
-        run(f(y, rows, weight_of, expert_of, h, ldh, dtype, tokens, hidden, top, place_of_pair, stream), "moe_combine");
+        run(f(y, rows, weight_of, expert_of, h, ldh, dtype, tokens, hidden, top, place_of_pair, weighted ? 1 : 0, stream),
+            "moe_combine");
     }
 
     // Routed experts (moe.cu).  route: the `top` largest of z = W_r h + b per token (float32) and the
@@ -708,12 +745,12 @@ public:
     }
     void moe_gemm(void* out, int out_dtype, long long ldo, const void* a, long long lda, const void* w, long long w_expert,
                   int dtype, int N, int K, int top, bool gather, bool scatter, int activation, const int* sorted_pair,
-                  const int* tile_info, const int* n_tiles, int pairs, int experts) {
+                  const int* tile_info, const int* n_tiles, int pairs, int experts, const float* a_weight = nullptr) {
         using Fn = int (*)(void*, int, long long, const void*, long long, const void*, long long, int, int, int, int, int,
-                           int, int, const int*, const int*, const int*, int, int, void*);
+                           int, int, const int*, const int*, const int*, int, int, const float*, void*);
         static Fn f = kernel_symbol<Fn>("moe", "kipp_moe_gemm");
         run(f(out, out_dtype, ldo, a, lda, w, w_expert, dtype, N, K, top, gather ? 1 : 0, scatter ? 1 : 0, activation,
-              sorted_pair, tile_info, n_tiles, pairs, experts, stream),
+              sorted_pair, tile_info, n_tiles, pairs, experts, a_weight, stream),
             "moe_gemm", 1, profiling ? format("moe_gemm %d x %d", N, K).c_str() : nullptr);
     }
     void moe_combine(float* y, const float* rows, const float* weight_of, int tokens, int hidden, int top,
@@ -746,11 +783,12 @@ public:
         static Fn f = kernel_symbol<Fn>("moe", "kipp_moe_padded_lists");
         run(f(place_of_pair, expert_of_tile, n_tiles, expert_of, pairs, experts, tile_rows, stream), "moe_lists");
     }
+    // weight_of (or null): the row times its pair's weight
     void moe_gather_rows(void* dst, const void* src, long long ld_src, const int* place_of_pair, int pairs, int top,
-                         int hidden) {
-        using Fn = int (*)(void*, const void*, long long, const int*, int, int, int, void*);
+                         int hidden, const float* weight_of = nullptr) {
+        using Fn = int (*)(void*, const void*, long long, const int*, int, const float*, int, int, void*);
         static Fn f = kernel_symbol<Fn>("moe", "kipp_moe_gather_rows");
-        run(f(dst, src, ld_src, place_of_pair, pairs, top, hidden, stream), "moe_gather_rows");
+        run(f(dst, src, ld_src, place_of_pair, pairs, weight_of, top, hidden, stream), "moe_gather_rows");
     }
     // out[r, :] = act(a[r, :] x w[expert_of_tile[r / tile]]^T) for the rows of the tiles in use
     void gemm_grouped(void* out, int out_dtype, long long ldc, const void* a, long long lda, const void* w, int rows, int N,

@@ -368,7 +368,7 @@ private:
 };
 
 void register_builtin_parts();           // parts.hpp, recurrent_parts.hpp, latent_parts.hpp, expert_parts.hpp
-void register_builtin_architectures();   // qwen3.hpp, venizen.hpp, varunex.hpp, zasudra.hpp, zunilorn.hpp
+void register_builtin_architectures();   // qwen3.hpp, venizen.hpp, varunex.hpp, zasudra.hpp, zunilorn.hpp, panolorn.hpp
 
 inline void ensure_registered() {
     static std::once_flag once;

@@ -10,11 +10,11 @@
 namespace kipp {
 
 // ---------------------------------------------------------------------------------------------
-// x_t = float(E[id_t, :]) with no scale (src/kipp.c:2940-2942).
+// x_t = float(E[id_t, :]), with no scale by default (src/kipp.c:2940-2942).
 class TokenEmbedding : public EmbeddingStage {
 public:
-    TokenEmbedding(int vocab, int hidden, std::string weight_name = "weight")
-        : vocab_(vocab), hidden_(hidden), name_(std::move(weight_name)) {
+    TokenEmbedding(int vocab, int hidden, std::string weight_name = "weight", double scale = 1.0)
+        : vocab_(vocab), hidden_(hidden), name_(std::move(weight_name)), scale_((float)scale) {
         if (vocab <= 0 || hidden <= 0) fail(KIPP_E_CONFIG, "token_embedding: sizes must be positive");
     }
     void tensor_specs(const std::string& prefix, std::vector<TensorSpec>& out) const override {
@@ -28,12 +28,13 @@ public:
         weight_ = b.shared(prefix + name_, dtype_, vocab_, hidden_);
     }
     void forward(StepContext& ctx, float* x) override {
-        ctx.ops->embed_gather(x, weight_, dtype_, ctx.meta->token_ids, ctx.tokens(), hidden_, vocab_);
+        ctx.ops->embed_gather(x, weight_, dtype_, ctx.meta->token_ids, ctx.tokens(), hidden_, vocab_, scale_);
     }
 
 private:
     int vocab_, hidden_, dtype_ = BF16;
     std::string name_;
+    float scale_ = 1.f;
     void* weight_ = nullptr;
 };
 
@@ -552,6 +553,12 @@ inline std::map<std::string, std::string> tensor_names(const Json& j, std::map<s
 // and a mixer without keys and values of its own that reads what another run wrote (shared_kv:
 // the run order gives it that run's cache id and writes_cache false).  A cap on the scaled scores
 // (softcap c: s <- c tanh(s / c)) goes with every option of this path.
+//
+// And: the q/k norm as the bare division (unit_norm: no weights); a number per head that a (capped)
+// score loses per position of distance between query and key (distance_slopes); a sigmoid gate per
+// element of the concatenated heads (element_gate: W_g [heads x value_dim, hidden]); and, for a mixer
+// whose blocks no other run looks past, a cache that gives a block's pages back once the sequence has
+// left it (forget_blocks).
 struct AttentionOptions {
     int value_dim = 0, keep_first = 0;
     bool head_mix = false;
@@ -568,6 +575,10 @@ struct AttentionOptions {
     bool values_are_keys = false;       // no W_v: the value of a key is the key as projected (before norm and rotation)
     bool shared_kv = false;             // no keys and values of its own: the run reads the cache another run wrote
     double softcap = 0.0;               // > 0: a scaled score s becomes softcap * tanh(s / softcap) before mask and softmax
+    bool unit_norm = false;             // the q/k norm divides by the root mean square and has no weights
+    std::vector<double> distance_slopes;    // per head: a score at distance d loses slope * d (after the cap)
+    bool element_gate = false;          // the concatenated heads times sigmoid(W_g h), W_g [heads * value_dim, hidden]
+    bool forget_blocks = false;         // with chunk: pages of blocks the sequence has left go back to the pool
     std::map<std::string, std::string> names = {{"q", "q_proj.weight"}, {"k", "k_proj.weight"}, {"v", "v_proj.weight"},
                                                 {"o", "o_proj.weight"}, {"q_norm", "q_norm.weight"},
                                                 {"k_norm", "k_norm.weight"}, {"head_mix", "head_mix.weight"},
@@ -600,12 +611,19 @@ public:
         if (opt_.combine_maps && !(opt_.combine_eps > 0)) fail(KIPP_E_CONFIG, "attention: combine_eps must be positive");
         if (opt_.head_mix && maps_ != 1) fail(KIPP_E_CONFIG, "attention: head_mix and score_maps do not go together");
         const bool more = opt_.norm_whole || opt_.interleaved || opt_.chunk != 0 || opt_.sink != 0 || opt_.head_gate ||
-                          opt_.values_are_keys || opt_.shared_kv;
+                          opt_.values_are_keys || opt_.shared_kv || opt_.unit_norm || !opt_.distance_slopes.empty() ||
+                          opt_.element_gate;
         segments_ = opt_.bias || maps_ > 1 || more;
         if ((opt_.bias || maps_ > 1) && qk_norm_) fail(KIPP_E_CONFIG, "attention: q/k norm with biases or score maps is not supported");
         if (more && (opt_.bias || maps_ > 1 || opt_.head_mix))
-            fail(KIPP_E_CONFIG, "attention: norm_whole, interleaved, chunk, sink, head_gate, values_are_keys and shared_kv "
-                                "do not go with biases, score maps or head_mix");
+            fail(KIPP_E_CONFIG, "attention: norm_whole, interleaved, chunk, sink, head_gate, values_are_keys, shared_kv, unit_norm, "
+                                "distance_slopes and element_gate do not go with biases, score maps or head_mix");
+        if (opt_.unit_norm && !qk_norm_) fail(KIPP_E_CONFIG, "attention: unit_norm needs qk_norm_eps");
+        if (opt_.element_gate && opt_.head_gate) fail(KIPP_E_CONFIG, "attention: head_gate and element_gate exclude each other");
+        if (!opt_.distance_slopes.empty() && (int)opt_.distance_slopes.size() != heads)
+            fail(KIPP_E_CONFIG, "attention: distance_slopes must hold one number per head");
+        if (opt_.forget_blocks && (opt_.chunk <= 0 || opt_.shared_kv))
+            fail(KIPP_E_CONFIG, "attention: forget_blocks needs chunk and keys of the mixer's own");
         if (opt_.norm_whole && !qk_norm_) fail(KIPP_E_CONFIG, "attention: norm_whole needs qk_norm_eps");
         if (opt_.chunk < 0 || (opt_.chunk > 0 && window_ > 0)) fail(KIPP_E_CONFIG, "attention: chunk must not be negative and excludes a window");
         if (opt_.sink < 0 || opt_.sink > 2) fail(KIPP_E_CONFIG, "attention: sink must be none, learned or unit");
@@ -617,7 +635,7 @@ public:
         // columns of the fused projection: q, then k and v where the mixer has its own, then the gate
         k_cols_ = opt_.shared_kv ? 0 : kv_dim_;
         v_cols_ = opt_.shared_kv || opt_.values_are_keys ? 0 : vv_dim_;
-        g_cols_ = opt_.head_gate ? heads : 0;
+        g_cols_ = opt_.element_gate ? o_dim_ : opt_.head_gate ? heads : 0;
         proj_cols_ = q_dim_ + k_cols_ + v_cols_ + g_cols_;
         proj_ld_ = more ? (proj_cols_ + 7) / 8 * 8 : proj_cols_;
         if (opt_.softcap < 0) fail(KIPP_E_CONFIG, "attention: softcap must not be negative");
@@ -636,12 +654,12 @@ public:
         if (k_cols_) add("k", {kv_dim_, hidden_});
         if (v_cols_) add("v", {vv_dim_, hidden_});
         add("o", {hidden_, o_dim_});
-        if (qk_norm_) {
+        if (qk_norm_ && !opt_.unit_norm) {
             add("q_norm", {opt_.norm_whole ? q_dim_ : head_dim_}, "near_one");
             if (k_cols_) add("k_norm", {opt_.norm_whole ? kv_dim_ : head_dim_}, "near_one");
         }
         if (opt_.sink == 1) add("sink", {heads_});
-        if (opt_.head_gate) add("gate", {heads_, hidden_});
+        if (g_cols_) add("gate", {g_cols_, hidden_});
         if (opt_.head_mix) add("head_mix", {heads_, heads_}, "near_identity");
         if (opt_.bias) {
             add("q_bias", {q_dim_});
@@ -652,9 +670,11 @@ public:
             for (const char* r : {"lq1", "lk1", "lq2", "lk2"}) add(r, {head_dim_});
         position_->tensor_specs(p, out);
     }
-    // (the maps of a key head lie side by side in one row of the key pages)
+    // (the maps of a key head lie side by side in one row of the key pages; a query sees at most the last
+    // `chunk` positions, so a window of that size keeps what blocks need)
     std::optional<PagedKVSpec> cache_spec() const override {
-        return PagedKVSpec{kv_heads_, maps_ * head_dim_, window_, v_dim_, window_ > 0 ? opt_.keep_first : 0};
+        return PagedKVSpec{kv_heads_, maps_ * head_dim_, opt_.forget_blocks ? opt_.chunk : window_, v_dim_,
+                           window_ > 0 ? opt_.keep_first : 0};
     }
     std::shared_ptr<WorkPlanner> planner(const DeviceInfo& dev, bool own_length) override {
         if (mix_path_) {                          // (entry, first token) per tile of its tensor-core prompt kernel
@@ -679,10 +699,11 @@ public:
         if (v_cols_) b.load(nv, base + (size_t)(q_dim_ + k_cols_) * hidden_ * es, dtype_, hidden_, vv_dim_, hidden_);
         if (g_cols_)
             b.load(p + opt_.names.at("gate"), base + (size_t)(q_dim_ + k_cols_ + v_cols_) * hidden_ * es, dtype_, hidden_,
-                   heads_, hidden_);
+                   g_cols_, hidden_);
         w_o_ = b.allocate((size_t)hidden_ * o_dim_ * es, no);
         b.load(no, w_o_, dtype_, o_dim_, hidden_, o_dim_);
-        if (qk_norm_ && segments_) {              // the head segments take their norm weights in float32
+        if (qk_norm_ && opt_.unit_norm) {
+        } else if (qk_norm_ && segments_) {       // the head segments take their norm weights in float32
             const int64_t nqw = opt_.norm_whole ? q_dim_ : head_dim_, nkw = opt_.norm_whole ? kv_dim_ : head_dim_;
             norm_dtype_ = F32;
             q_norm_ = b.allocate((size_t)nqw * sizeof(float), p + opt_.names.at("q_norm"));
@@ -721,6 +742,11 @@ public:
             sink_ = static_cast<float*>(b.allocate((size_t)heads_ * sizeof(float), p + "unit sink"));
             cuda_check(cudaMemset(sink_, 0, (size_t)heads_ * sizeof(float)), "clearing the unit sink");
         }
+        if (!opt_.distance_slopes.empty()) {
+            std::vector<float> s(opt_.distance_slopes.begin(), opt_.distance_slopes.end());
+            slopes_ = static_cast<float*>(b.allocate(s.size() * sizeof(float), p + "distance slopes"));
+            cuda_check(cudaMemcpy(slopes_, s.data(), s.size() * sizeof(float), cudaMemcpyHostToDevice), "upload of the distance slopes");
+        }
         if (opt_.combine_maps) {
             // lambda is one number for the layer: formed once, in double precision
             double dot[2] = {0.0, 0.0};
@@ -740,7 +766,7 @@ public:
     }
     size_t weight_bytes() const override {
         size_t n = ((size_t)proj_cols_ * hidden_ + (size_t)hidden_ * o_dim_) * dtype_size(dtype_);
-        if (qk_norm_) n += (opt_.norm_whole ? (size_t)q_dim_ + k_cols_ : 2 * (size_t)head_dim_) * dtype_size(norm_dtype_);
+        if (qk_norm_ && !opt_.unit_norm) n += (opt_.norm_whole ? (size_t)q_dim_ + k_cols_ : 2 * (size_t)head_dim_) * dtype_size(norm_dtype_);
         if (opt_.head_mix) n += (size_t)heads_ * heads_ * sizeof(float);
         if (opt_.bias) n += (size_t)(q_dim_ + kv_dim_ + vv_dim_) * sizeof(float);
         return n;
@@ -762,6 +788,7 @@ private:
     float lambda_ = 0.f;
     void *w_qkv_ = nullptr, *w_o_ = nullptr, *q_norm_ = nullptr, *k_norm_ = nullptr;
     float *head_mix_ = nullptr, *q_bias_ = nullptr, *k_bias_ = nullptr, *v_bias_ = nullptr, *sink_ = nullptr;
+    float* slopes_ = nullptr;
     int k_cols_ = 0, v_cols_ = 0, g_cols_ = 0, proj_cols_ = 0, proj_ld_ = 0;
     std::shared_ptr<AttentionPlanner> planner_;
     std::shared_ptr<MixTilePlanner> mix_planner_;
@@ -870,8 +897,17 @@ private:
     void *w_up_ = nullptr, *w_down_ = nullptr;
 };
 
-// Gated dense feed-forward with limits: g = min(W_gate n + b_g, limit), u = clamp(W_up n + b_u, -limit, limit),
-// x += W_down (g sigmoid(alpha g) (u + 1)) + b_d.  Biases are optional (bias), limit 0 means none.  With
+// The activation of a gated feed-forward's gate (Ops::Glu::act).
+inline int gate_activation(const Json& j, const char* key) {
+    const std::string a = j.get_string(key, "swish");
+    if (a == "swish") return -1;
+    if (a == "gelu_tanh") return ACT_GELU_TANH;
+    fail(KIPP_E_CONFIG, std::string(key) + " of a gated feed-forward must be swish or gelu_tanh, not '" + a + "'");
+}
+
+// Gated dense feed-forward: g = min(W_gate n + b_g, limit), u = clamp(W_up n + b_u, -limit, limit),
+// x += W_down (act(g) (u + up_add)) + b_d, act(g) = g sigmoid(alpha g) (activation "swish") or gelu in its tanh
+// form ("gelu_tanh"); up_add is 1 unless given.  Biases are optional (bias), limit 0 means none.  With
 // row_gate the part's output is also multiplied by sigmoid(w_r . n), one number per token (a tensor
 // [1, hidden], kept in float32): the factor is applied to the hidden row before the (linear) down
 // projection.  Gate and up rows lie interleaved in one matrix, so one product makes both and the
@@ -884,6 +920,8 @@ public:
         inter_ = (int)j.get("intermediate_size").as_int();
         limit_ = (float)j.get_double("limit", 0.0);
         alpha_ = (float)j.get_double("alpha", 1.0);
+        act_ = gate_activation(j, "activation");
+        up_add_ = (float)j.get_double("up_add", 1.0);
         bias_ = j.get_bool("bias", false);
         row_gate_ = j.get_bool("row_gate", false);
         names_ = tensor_names(j, {{"gate", "gate"}, {"up", "up"}, {"down", "down"}, {"gate_bias", "gate.b"},
@@ -941,8 +979,10 @@ public:
         const int T = ctx.tokens();
         NormFold in, out;
         Ops::Glu glu;
+        glu.act = act_;
         glu.alpha = alpha_;
         glu.limit = limit_;
+        glu.up_add = up_add_;
         glu.bias = b_in_;
         if (row_gate_) {
             if (ctx.input_scale.valid()) fail(KIPP_E_STATE, "gated_mlp: a gate per token does not read an input in deferred form");
@@ -964,7 +1004,8 @@ public:
 
 private:
     int hidden_ = 0, inter_ = 0, inter_ld_ = 0, dtype_ = BF16;
-    float limit_ = 0.f, alpha_ = 1.f;
+    int act_ = -1;
+    float limit_ = 0.f, alpha_ = 1.f, up_add_ = 1.f;
     bool bias_ = false, row_gate_ = false;
     std::map<std::string, std::string> names_;
     void *w_in_ = nullptr, *w_down_ = nullptr;
@@ -1098,6 +1139,105 @@ private:
     std::unique_ptr<Mixer> mixer_;
     std::unique_ptr<Norm> n2_;
     std::unique_ptr<FeedForward> ffn_;
+    float mult_;
+    std::vector<std::string> names_;
+};
+
+// x += mult * norm1b(mixer(norm1(x))); x += mult * norm2b(ffn(norm2(x))): a norm on either side of every
+// sublayer.  A sublayer adds its output into a cleared float32 buffer; one kernel then norms that buffer,
+// adds it to the stream and norms the new stream for the sublayer that reads it next, also across blocks
+// of this kind.  The norms must be plain RMS norms.  A block without a feed-forward (ffn null, its two
+// norms too) has the first sublayer only.
+class SandwichNormBlock : public Block {
+public:
+    SandwichNormBlock(std::unique_ptr<Norm> n1, std::unique_ptr<Mixer> mixer, std::unique_ptr<Norm> n1b, std::unique_ptr<Norm> n2,
+                      std::unique_ptr<FeedForward> ffn, std::unique_ptr<Norm> n2b, double mult, std::vector<std::string> names)
+        : n1_(std::move(n1)), mixer_(std::move(mixer)), n1b_(std::move(n1b)), n2_(std::move(n2)), ffn_(std::move(ffn)),
+          n2b_(std::move(n2b)), mult_((float)mult), names_(std::move(names)) {
+        if (names_.size() != 6) fail(KIPP_E_CONFIG, "sandwich_norm_block: six name prefixes are needed");
+        if ((n2_ == nullptr) != (ffn_ == nullptr) || (n2b_ == nullptr) != (ffn_ == nullptr))
+            fail(KIPP_E_CONFIG, "sandwich_norm_block: post_norm, ffn and ffn_out_norm come together or not at all");
+        for (const Norm* n : {n1b_.get(), n2_.get(), n2b_.get()})
+            if (n != nullptr && n->size() != n1_->size()) fail(KIPP_E_CONFIG, "sandwich_norm_block: the norms differ in size");
+    }
+    void tensor_specs(const std::string& p, std::vector<TensorSpec>& out) const override {
+        each([&](const Part& part, const std::string& name) { part.tensor_specs(p + name, out); });
+    }
+    void bind(Binder& b, const std::string& p) override {
+        each([&](Part& part, const std::string& name) { part.bind(b, p + name); });
+        for (const Norm* n : {n1_.get(), n1b_.get(), n2_.get(), n2b_.get()})
+            if (n != nullptr && !n->rms_spec()) fail(KIPP_E_CONFIG, "sandwich_norm_block: the norms must be RMS norms");
+    }
+    size_t weight_bytes() const override {
+        size_t n = 0;
+        each([&](const Part& part, const std::string&) { n += part.weight_bytes(); });
+        return n;
+    }
+    bool graph_safe() const override {
+        bool ok = true;
+        each([&](const Part& part, const std::string&) { ok = ok && part.graph_safe(); });
+        return ok;
+    }
+    std::vector<Mixer*> mixers() override { return mixer_->parts(); }
+    void forward(StepContext& ctx, const LayerRun& run, float* x) override {
+        const int T = ctx.tokens(), W = n1_->size();
+        Ops& ops = *ctx.ops;
+        // the norms run between the sublayers: nothing to fold into the products, nothing pending
+        ctx.input_scale = RowScale{};
+        ctx.pending_norm = nullptr;
+        ctx.emit_for = nullptr;
+        ctx.emitted = false;
+        void* h = ctx.workspace->buffer("normed", (size_t)T * W * ctx.element());
+        float* y = ctx.workspace->get<float>("sublayer_output", (size_t)T * W);
+        const bool ready = ctx.input_ready_for == this;
+        ctx.input_ready_for = nullptr;
+        // as in HyperConnectionBlock: in steps of few tokens the kernel that reads y leaves it zeroed, else a memset does
+        const bool kernel_clears = T < 1024;
+        auto clear = [&] { cuda_check(cudaMemsetAsync(y, 0, (size_t)T * W * sizeof(float), ctx.stream), "clearing a sublayer's output"); };
+        // y joins the stream through its norm; `next` (or null) is the norm whose output h the next sublayer reads
+        auto join = [&](const Norm& out_norm, const Norm* next) {
+            const RmsNormSpec b = *out_norm.rms_spec();
+            if (next == nullptr) {
+                ops.rmsnorm_scaled_add(x, y, b.weight, b.weight_dtype, T, W, b.eps, mult_);
+                return;
+            }
+            const RmsNormSpec n = *next->rms_spec();
+            ops.norm_add_norm(x, y, kernel_clears, b.weight, b.weight_dtype, b.eps, mult_, n.weight, n.weight_dtype, n.eps, h,
+                              ctx.dtype, T, W);
+        };
+        if (!ready) n1_->forward(ctx, x, h, nullptr, T);
+        if (!ready || !kernel_clears) clear();
+        mixer_->forward(ctx, run, 0, h, y);
+        const SandwichNormBlock* next = dynamic_cast<const SandwichNormBlock*>(ctx.following_block);
+        if (next != nullptr && next->n1_->size() != W) next = nullptr;
+        const Norm* next_norm = next != nullptr ? next->n1_.get() : nullptr;
+        if (ffn_) {
+            join(*n1b_, n2_.get());
+            if (!kernel_clears) clear();
+            ffn_->forward(ctx, h, y);
+            join(*n2b_, next_norm);
+        } else {
+            join(*n1b_, next_norm);
+        }
+        ctx.input_ready_for = next;
+        ctx.emitted = false;
+    }
+    Norm* input_norm() { return n1_.get(); }
+    Norm* post_norm() { return n2_.get(); }
+    FeedForward* feed_forward() { return ffn_.get(); }
+
+private:
+    // every part with its name prefix, in the order of names_
+    template <typename F> void each(F&& f) const {
+        Part* parts[6] = {n1_.get(), mixer_.get(), n1b_.get(), n2_.get(), ffn_.get(), n2b_.get()};
+        for (size_t i = 0; i < 6; ++i)
+            if (parts[i] != nullptr) f(*parts[i], names_[i]);
+    }
+    std::unique_ptr<Norm> n1_;
+    std::unique_ptr<Mixer> mixer_;
+    std::unique_ptr<Norm> n1b_, n2_;
+    std::unique_ptr<FeedForward> ffn_;
+    std::unique_ptr<Norm> n2b_;
     float mult_;
     std::vector<std::string> names_;
 };
@@ -1518,7 +1658,7 @@ inline void register_builtin_parts() {
     Registry& r = Registry::get();
     r.add_part_kind("token_embedding", [](const Json& j, const BuildContext&) -> std::unique_ptr<Part> {
         return std::make_unique<TokenEmbedding>((int)j.get("vocab_size").as_int(), (int)j.get("hidden_size").as_int(),
-                                                j.get_string("weight_name", "weight"));
+                                                j.get_string("weight_name", "weight"), j.get_double("scale", 1.0));
     });
     r.add_part_kind("output_head", [](const Json& j, const BuildContext&) -> std::unique_ptr<Part> {
         return std::make_unique<OutputHead>((int)j.get("vocab_size").as_int(), (int)j.get("hidden_size").as_int(),
@@ -1637,6 +1777,11 @@ inline void register_builtin_parts() {
         options.values_are_keys = j.get_bool("values_are_keys", false);
         options.shared_kv = j.get_bool("shared_kv", false);
         options.softcap = j.get_double("softcap", 0.0);
+        options.unit_norm = j.get_bool("unit_norm", false);
+        if (const Json* sl = j.find("distance_slopes"); sl && !sl->is_null())
+            for (auto& v : sl->items()) options.distance_slopes.push_back(v.as_double());
+        options.element_gate = j.get_bool("element_gate", false);
+        options.forget_blocks = j.get_bool("forget_blocks", false);
         options.names = tensor_names(j, options.names);
         return std::make_unique<AttentionMixer>(
             (int)j.get("hidden_size").as_int(), (int)j.get("num_heads").as_int(), (int)j.get("num_kv_heads").as_int(),
@@ -1659,6 +1804,21 @@ inline void register_builtin_parts() {
             reg.make_as<Norm>(j.get("input_norm"), ctx, "a norm"), reg.make_as<Mixer>(j.get("mixer"), ctx, "a mixer"),
             has_ffn ? reg.make_as<Norm>(*n2, ctx, "a norm") : nullptr,
             has_ffn ? reg.make_as<FeedForward>(*ff, ctx, "a feed-forward") : nullptr, names);
+    });
+    r.add_part_kind("sandwich_norm_block", [](const Json& j, const BuildContext& ctx) -> std::unique_ptr<Part> {
+        const Registry& reg = Registry::get();
+        std::vector<std::string> names;
+        for (auto& n : j.get("names").items()) names.push_back(n.as_string());
+        auto norm = [&](const char* key) -> std::unique_ptr<Norm> {
+            const Json* n = j.find(key);
+            return n && !n->is_null() ? reg.make_as<Norm>(*n, ctx, "a norm") : nullptr;
+        };
+        const Json* ff = j.find("ffn");
+        return std::make_unique<SandwichNormBlock>(
+            reg.make_as<Norm>(j.get("input_norm"), ctx, "a norm"), reg.make_as<Mixer>(j.get("mixer"), ctx, "a mixer"),
+            reg.make_as<Norm>(j.get("mixer_out_norm"), ctx, "a norm"), norm("post_norm"),
+            ff && !ff->is_null() ? reg.make_as<FeedForward>(*ff, ctx, "a feed-forward") : nullptr, norm("ffn_out_norm"),
+            j.get_double("residual_mult", 1.0), names);
     });
     r.add_part_kind("output_norm_block", [](const Json& j, const BuildContext& ctx) -> std::unique_ptr<Part> {
         const Registry& reg = Registry::get();

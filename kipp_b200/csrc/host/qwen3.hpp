@@ -230,6 +230,7 @@ void register_venizen();                 // venizen.hpp
 void register_varunex();                 // varunex.hpp
 void register_zasudra();                 // zasudra.hpp
 void register_zunilorn();                // zunilorn.hpp
+void register_panolorn();                // panolorn.hpp
 
 inline void register_builtin_architectures() {
     Registry::get().add_architecture("Qwen3ForCausalLM", Architecture{qwen3::normalize, qwen3::plan});
@@ -237,6 +238,7 @@ inline void register_builtin_architectures() {
     register_varunex();
     register_zasudra();
     register_zunilorn();
+    register_panolorn();
 }
 
 }  // namespace kipp

@@ -11,8 +11,10 @@
 //   combine   y[t] += sum over the token's choices, in the order of their rank, of weight x row.
 //
 // A second way of routing (kipp_moe_route_scores): scores s = softmax(z) over ALL outputs of the
-// router; the choice by s + correction (a learned number per output that steers the choice only); the
-// weights are the chosen scores divided by their sum, times a scale.  The last outputs of the router
+// router, or s = sigmoid(z) output by output; the choice by s + correction (a learned number per output that
+// steers the choice only); the weights are the chosen scores divided by their sum (or as they are), times a
+// scale.  The weight may sit on the expert's INPUT instead of its output: the rows handed to the experts are
+// then weight x token and the combine adds the experts' rows as they are.  The last outputs of the router
 // may be identity experts, which hand the token's input on: their pairs carry a negative expert id,
 // the lists and products leave them out, and the combine adds weight x input for them.
 //
@@ -52,7 +54,8 @@ template <typename T, int TOK>
 __global__ void __launch_bounds__(512)
 moe_route_kernel(int* __restrict__ expert_of, float* __restrict__ weight_of, const T* __restrict__ h, long long ldh,
                  const float* __restrict__ router, const float* __restrict__ bias, int tokens, int hidden, int experts,
-                 int top, int vec, int by_scores, int real_experts, float weight_scale) {
+                 int top, int vec, int by_scores, int renormalize, int real_experts, float weight_scale) {
+    // by_scores: 0 the logits choose, 1 softmax scores, 2 sigmoid scores
     extern __shared__ float z_all[];                      // [TOK][experts], and [TOK][experts] scores when by_scores
     pdl_launch_dependents();
     pdl_wait();
@@ -99,7 +102,16 @@ moe_route_kernel(int* __restrict__ expert_of, float* __restrict__ weight_of, con
         if (t >= tokens) continue;
         float* z = z_all + (size_t)j * experts;
         float* score = z_all + (size_t)(TOK + j) * experts;
-        if (by_scores) {
+        if (by_scores == 2) {
+            // (without a correction the logits are compared: the order is the same, and scores that
+            // round to 1 do not tie)
+            for (int e = lane; e < experts; e += 32) {
+                const float sc = 1.0f / (1.0f + expf(-z[e]));
+                score[e] = sc;
+                if (bias) z[e] = sc + bias[e];
+            }
+            __syncwarp();
+        } else if (by_scores) {
             // s = softmax(z) over all outputs; what is compared is s + correction
             float top_z = -INFINITY;
             for (int e = lane; e < experts; e += 32) top_z = fmaxf(top_z, z[e]);
@@ -145,7 +157,7 @@ moe_route_kernel(int* __restrict__ expert_of, float* __restrict__ weight_of, con
             float* w = weight_of + (size_t)t * top;
             float sum = 0.f;
             for (int k = 0; k < top; ++k) sum += w[k];
-            const float f = weight_scale / (sum + 1e-20f);
+            const float f = renormalize ? weight_scale / (sum + 1e-20f) : weight_scale;
             for (int k = 0; k < top; ++k) w[k] *= f;
         } else if (lane == 0) {
             float* w = weight_of + (size_t)t * top;
@@ -221,10 +233,11 @@ moe_padded_lists_kernel(int* __restrict__ place_of_pair, int* __restrict__ exper
         place_of_pair[p] = expert_of[p] >= 0 ? atomicAdd(&cursor[expert_of[p]], 1) : -1;
 }
 
-// dst[place_of_pair[p], :] = src[p / top, :], 16 bytes per thread and step (bfloat16 rows of 8 n elements).
+// dst[place_of_pair[p], :] = src[p / top, :], 16 bytes per thread and step (bfloat16 rows of 8 n elements);
+// weight_of given: times the pair's weight, in float32, rounded once.
 __global__ void __launch_bounds__(256)
 moe_gather_rows_kernel(uint4* __restrict__ dst, const uint4* __restrict__ src, long long ld_src16, int row16,
-                       const int* __restrict__ place_of_pair, int pairs, int top) {
+                       const int* __restrict__ place_of_pair, const float* __restrict__ weight_of, int pairs, int top) {
     pdl_launch_dependents();
     pdl_wait();
     const int p = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
@@ -232,6 +245,17 @@ moe_gather_rows_kernel(uint4* __restrict__ dst, const uint4* __restrict__ src, l
     if (place_of_pair[p] < 0) return;                    // a pair without an expert's product
     const uint4* from = src + (size_t)(p / top) * ld_src16;
     uint4* to = dst + (size_t)place_of_pair[p] * row16;
+    if (weight_of != nullptr) {
+        const float w = weight_of[p];
+        for (int i = threadIdx.x & 31; i < row16; i += 32) {
+            uint4 v = from[i];
+            __nv_bfloat162* e = reinterpret_cast<__nv_bfloat162*>(&v);
+#pragma unroll
+            for (int j = 0; j < 4; ++j) e[j] = __floats2bfloat162_rn(w * __low2float(e[j]), w * __high2float(e[j]));
+            to[i] = v;
+        }
+        return;
+    }
     for (int i = threadIdx.x & 31; i < row16; i += 32) to[i] = from[i];
 }
 
@@ -241,6 +265,7 @@ struct GemmArgs {
     const void* w; long long w_expert;      // elements between two experts' matrices [N, K]
     int N, K, top, gather, scatter, act;
     const int* sorted_pair; const int* tile_info; const int* n_tiles;
+    const float* a_weight;                  // [pairs] or null: a gathered row is multiplied by its pair's weight
 };
 
 // CUDA cores: a block of 256 threads per 64 x 64 tile, each thread 4 x 4 results.
@@ -250,6 +275,7 @@ moe_gemm_kernel(const GemmArgs g) {
     __shared__ float As[BK][BM + 4];
     __shared__ float Ws[BK][BN + 4];
     __shared__ int arow[BM], orow[BM];
+    __shared__ float aw[BM];
     pdl_launch_dependents();
     pdl_wait();
     const int tile = blockIdx.y;
@@ -260,6 +286,7 @@ moe_gemm_kernel(const GemmArgs g) {
         const int pair = tid < rows ? g.sorted_pair[r0 + tid] : -1;
         arow[tid] = pair < 0 ? -1 : (g.gather ? pair / g.top : r0 + tid);
         orow[tid] = pair < 0 ? -1 : (g.scatter ? pair : r0 + tid);
+        aw[tid] = pair >= 0 && g.a_weight != nullptr ? g.a_weight[pair] : 1.f;
     }
     __syncthreads();
     const T* A = static_cast<const T*>(g.a);
@@ -272,11 +299,12 @@ moe_gemm_kernel(const GemmArgs g) {
         for (int j = 0; j < TN; ++j) acc[i][j] = 0.f;
     const int lrow = tid >> 2, lk = (tid & 3) * 4;
     const int ar = arow[lrow];
+    const float rw = aw[lrow];
     for (int k0 = 0; k0 < K; k0 += BK) {
 #pragma unroll
         for (int i = 0; i < 4; ++i) {
             const int k = k0 + lk + i, wn = n0 + lrow;
-            As[lk + i][lrow] = (ar >= 0 && k < K) ? to_f32(A[(size_t)ar * g.lda + k]) : 0.f;
+            As[lk + i][lrow] = (ar >= 0 && k < K) ? rw * to_f32(A[(size_t)ar * g.lda + k]) : 0.f;
             Ws[lk + i][lrow] = (wn < N && k < K) ? to_f32(W[(size_t)wn * K + k]) : 0.f;
         }
         __syncthreads();
@@ -313,23 +341,24 @@ moe_combine_kernel(float* __restrict__ y, const float* __restrict__ rows, const 
     pdl_launch_dependents();
     pdl_wait();
     const int t = blockIdx.x;
-    const float* w = weight_of + (size_t)t * top;
+    const float* w = weight_of ? weight_of + (size_t)t * top : nullptr;      // null: rows that carry their weight
     for (int i = threadIdx.x; i < hidden; i += blockDim.x) {
         float acc = 0.f;
         for (int k = 0; k < top; ++k) {
             const size_t row = place_of_pair ? (size_t)place_of_pair[(size_t)t * top + k] : (size_t)t * top + k;
-            acc = fmaf(w[k], rows[row * hidden + i], acc);
+            acc = weight_of ? fmaf(w[k], rows[row * hidden + i], acc) : acc + rows[row * hidden + i];
         }
         y[(size_t)t * hidden + i] += acc;
     }
 }
 
-// The combine where some pairs are identity experts (expert_of < 0): their row is the token's input.
+// The combine where some pairs are identity experts (expert_of < 0): their row is weight x the token's input
+// (weighted: the other rows carry their weight already).
 template <typename T>
 __global__ void __launch_bounds__(512)
 moe_combine_identity_kernel(float* __restrict__ y, const float* __restrict__ rows, const float* __restrict__ weight_of,
                             const int* __restrict__ expert_of, const T* __restrict__ h, long long ldh, int hidden, int top,
-                            const int* __restrict__ place_of_pair) {
+                            const int* __restrict__ place_of_pair, int weighted) {
     pdl_launch_dependents();
     pdl_wait();
     const int t = blockIdx.x;
@@ -342,7 +371,7 @@ moe_combine_identity_kernel(float* __restrict__ y, const float* __restrict__ row
                 acc = fmaf(w[k], to_f32(h[(size_t)t * ldh + i]), acc);
             } else {
                 const size_t row = place_of_pair ? (size_t)place_of_pair[(size_t)t * top + k] : (size_t)t * top + k;
-                acc = fmaf(w[k], rows[row * hidden + i], acc);
+                acc = weighted ? acc + rows[row * hidden + i] : fmaf(w[k], rows[row * hidden + i], acc);
             }
         }
         y[(size_t)t * hidden + i] += acc;
@@ -355,8 +384,8 @@ extern "C" int kipp_moe_max_tiles(int pairs, int experts) { return (pairs + BM -
 
 // expert_of, weight_of [tokens, top]: the chosen experts in the order of their logits and their weights.
 static int moe_route_any(int* expert_of, float* weight_of, const void* h, long long ldh, int dtype, const float* router,
-                         const float* bias, int tokens, int hidden, int experts, int top, int by_scores, int real_experts,
-                         float weight_scale, void* stream) {
+                         const float* bias, int tokens, int hidden, int experts, int top, int by_scores, int renormalize,
+                         int real_experts, float weight_scale, void* stream) {
     if (tokens <= 0) return 0;
     if (hidden <= 0 || experts <= 0 || top <= 0 || top > experts || experts > 2048) return KIPP_ERR_ARG;
     cudaStream_t s = (cudaStream_t)stream;
@@ -370,32 +399,33 @@ static int moe_route_any(int* expert_of, float* weight_of, const void* h, long l
     if (dtype == KIPP_DT_F32) {
         if (tok == 4)
             return kipp_launch(moe_route_kernel<float, 4>, grid, block, smem, s, 1, expert_of, weight_of, (const float*)h,
-                               ldh, router, bias, tokens, hidden, experts, top, vec, by_scores, real_experts, weight_scale);
+                               ldh, router, bias, tokens, hidden, experts, top, vec, by_scores, renormalize, real_experts, weight_scale);
         return kipp_launch(moe_route_kernel<float, 1>, grid, block, smem, s, 1, expert_of, weight_of, (const float*)h, ldh,
-                           router, bias, tokens, hidden, experts, top, vec, by_scores, real_experts, weight_scale);
+                           router, bias, tokens, hidden, experts, top, vec, by_scores, renormalize, real_experts, weight_scale);
     }
     if (dtype == KIPP_DT_BF16) {
         if (tok == 4)
             return kipp_launch(moe_route_kernel<bf16, 4>, grid, block, smem, s, 1, expert_of, weight_of, (const bf16*)h, ldh,
-                               router, bias, tokens, hidden, experts, top, vec, by_scores, real_experts, weight_scale);
+                               router, bias, tokens, hidden, experts, top, vec, by_scores, renormalize, real_experts, weight_scale);
         return kipp_launch(moe_route_kernel<bf16, 1>, grid, block, smem, s, 1, expert_of, weight_of, (const bf16*)h, ldh,
-                           router, bias, tokens, hidden, experts, top, vec, by_scores, real_experts, weight_scale);
+                           router, bias, tokens, hidden, experts, top, vec, by_scores, renormalize, real_experts, weight_scale);
     }
     return KIPP_ERR_DTYPE;
 }
 extern "C" int kipp_moe_route(int* expert_of, float* weight_of, const void* h, long long ldh, int dtype, const float* router,
                               const float* bias, int tokens, int hidden, int experts, int top, void* stream) {
-    return moe_route_any(expert_of, weight_of, h, ldh, dtype, router, bias, tokens, hidden, experts, top, 0, experts, 1.f, stream);
+    return moe_route_any(expert_of, weight_of, h, ldh, dtype, router, bias, tokens, hidden, experts, top, 0, 1, experts, 1.f, stream);
 }
-// Routing by scores: s = softmax(W_r h) over `outputs` router rows, the `top` largest of s + correction
-// (correction null: of s), weights s / (sum of the chosen + 1e-20) * weight_scale.  Outputs from
+// Routing by scores: s = softmax(W_r h) over `outputs` router rows (sigmoid: s = sigmoid(W_r h) row by row), the
+// `top` largest of s + correction (correction null: of s), weights s / (sum of the chosen + 1e-20) * weight_scale
+// (renormalize 0: s * weight_scale).  Outputs from
 // `experts` on are identity experts: expert_of holds -1 - (output - experts) for them.
 extern "C" int kipp_moe_route_scores(int* expert_of, float* weight_of, const void* h, long long ldh, int dtype,
                                      const float* router, const float* correction, int tokens, int hidden, int outputs,
-                                     int experts, int top, float weight_scale, void* stream) {
+                                     int experts, int top, int sigmoid, int renormalize, float weight_scale, void* stream) {
     if (experts < 0 || experts > outputs) return KIPP_ERR_ARG;
-    return moe_route_any(expert_of, weight_of, h, ldh, dtype, router, correction, tokens, hidden, outputs, top, 1, experts,
-                         weight_scale, stream);
+    return moe_route_any(expert_of, weight_of, h, ldh, dtype, router, correction, tokens, hidden, outputs, top, sigmoid ? 2 : 1,
+                         renormalize, experts, weight_scale, stream);
 }
 
 // sorted_pair [pairs], tile_info [3 x kipp_moe_max_tiles], n_tiles [1]
@@ -408,18 +438,19 @@ extern "C" int kipp_moe_lists(int* sorted_pair, int* tile_info, int* n_tiles, co
 }
 
 // One product of every tile: out rows = act(A rows x W[expert]^T).  gather: a row of A is the pair's
-// token (else its place in the sorted list); scatter: a row of out is the pair (else its place in the
+// token (else its place in the sorted list), times a_weight[pair] where that is given; scatter: a row of out is the pair (else its place in the
 // sorted list).  A and W in `dtype`; out in `out_dtype`.  On the CUDA cores: float32, and sizes the
 // grouped tensor-core products cannot take.
 extern "C" int kipp_moe_gemm(void* out, int out_dtype, long long ldo, const void* a, long long lda, const void* w,
                              long long w_expert, int dtype, int N, int K, int top, int gather, int scatter, int act,
                              const int* sorted_pair, const int* tile_info, const int* n_tiles, int pairs, int experts,
-                             void* stream) {
+                             const float* a_weight, void* stream) {
     if (pairs <= 0) return 0;
     if (N <= 0 || K <= 0 || top <= 0 || experts <= 0) return KIPP_ERR_ARG;
     GemmArgs g;
     g.out = out; g.ldo = ldo; g.a = a; g.lda = lda; g.w = w; g.w_expert = w_expert;
     g.N = N; g.K = K; g.top = top; g.gather = gather; g.scatter = scatter; g.act = act;
+    g.a_weight = gather ? a_weight : nullptr;
     g.sorted_pair = sorted_pair; g.tile_info = tile_info; g.n_tiles = n_tiles;
     const int tiles = kipp_moe_max_tiles(pairs, experts);
     cudaStream_t s = (cudaStream_t)stream;
@@ -430,7 +461,7 @@ extern "C" int kipp_moe_gemm(void* out, int out_dtype, long long ldo, const void
     return KIPP_ERR_DTYPE;
 }
 
-// y[t, :] += sum_k weight_of[t, k] * rows[r, :], k in order; r = t * top + k, or place_of_pair[t * top + k] if given.
+// y[t, :] += sum_k weight_of[t, k] * rows[r, :] (weight_of null: the rows as they are), k in order; r = t * top + k, or place_of_pair[t * top + k] if given.
 extern "C" int kipp_moe_combine(float* y, const float* rows, const float* weight_of, int tokens, int hidden, int top,
                                 const int* place_of_pair, void* stream) {
     if (tokens <= 0) return 0;
@@ -443,15 +474,15 @@ extern "C" int kipp_moe_combine(float* y, const float* rows, const float* weight
 // The same where pairs with expert_of < 0 stand for the token's own input h [tokens, ldh] (`dtype`).
 extern "C" int kipp_moe_combine_identity(float* y, const float* rows, const float* weight_of, const int* expert_of,
                                          const void* h, long long ldh, int dtype, int tokens, int hidden, int top,
-                                         const int* place_of_pair, void* stream) {
+                                         const int* place_of_pair, int weighted, void* stream) {
     if (tokens <= 0) return 0;
     if (hidden <= 0 || top <= 0 || expert_of == nullptr || h == nullptr) return KIPP_ERR_ARG;
     if (dtype == KIPP_DT_F32)
         return kipp_launch(moe_combine_identity_kernel<float>, dim3((unsigned)tokens), dim3(hidden >= 2048 ? 512 : hidden >= 512 ? 256 : 128), 0, (cudaStream_t)stream, 1, y,
-                           rows, weight_of, expert_of, (const float*)h, ldh, hidden, top, place_of_pair);
+                           rows, weight_of, expert_of, (const float*)h, ldh, hidden, top, place_of_pair, weighted);
     if (dtype == KIPP_DT_BF16)
         return kipp_launch(moe_combine_identity_kernel<bf16>, dim3((unsigned)tokens), dim3(hidden >= 2048 ? 512 : hidden >= 512 ? 256 : 128), 0, (cudaStream_t)stream, 1, y,
-                           rows, weight_of, expert_of, (const bf16*)h, ldh, hidden, top, place_of_pair);
+                           rows, weight_of, expert_of, (const bf16*)h, ldh, hidden, top, place_of_pair, weighted);
     return KIPP_ERR_DTYPE;
 }
 
@@ -470,11 +501,12 @@ extern "C" int kipp_moe_padded_lists(int* place_of_pair, int* expert_of_tile, in
                        1, place_of_pair, expert_of_tile, n_tiles, expert_of, pairs, experts, tile_rows);
 }
 
-// dst[place_of_pair[p], 0 .. hidden) = src[p / top, 0 .. hidden), bfloat16, hidden and ld_src multiples of 8.
+// dst[place_of_pair[p], 0 .. hidden) = src[p / top, 0 .. hidden), bfloat16, hidden and ld_src multiples of 8;
+// weight_of [pairs] or null: times the pair's weight.
 extern "C" int kipp_moe_gather_rows(void* dst, const void* src, long long ld_src, const int* place_of_pair, int pairs,
-                                    int top, int hidden, void* stream) {
+                                    const float* weight_of, int top, int hidden, void* stream) {
     if (pairs <= 0) return 0;
     if (hidden <= 0 || hidden % 8 || ld_src % 8 || top <= 0 || (((uintptr_t)dst | (uintptr_t)src) & 15)) return KIPP_ERR_ARG;
     return kipp_launch(moe_gather_rows_kernel, dim3((unsigned)((pairs + 7) / 8)), dim3(256), 0, (cudaStream_t)stream, 1,
-                       (uint4*)dst, (const uint4*)src, ld_src / 8, hidden / 8, place_of_pair, pairs, top);
+                       (uint4*)dst, (const uint4*)src, ld_src / 8, hidden / 8, place_of_pair, weight_of, pairs, top);
 }
