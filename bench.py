@@ -208,6 +208,18 @@ def zunilorn_of(size: str, vocab: int = 32000) -> dict:
             "streams": 4, "logit_softcap": 30.0, "layers": [order[i % 4] for i in range(layers)]}
 
 
+def panolorn_of(size: str, vocab: int = 32000) -> dict:
+    """Attention in blocks of positions in every layer, beside a dense gated feed-forward and, in every
+    other layer, sixteen experts of a quarter of its width of which a token takes four, with a
+    shared expert of the same width."""
+    width, heads, kv, dim, ff, layers = DESIGN_SIZES[size]
+    att = {"heads": heads, "kv_heads": kv, "dim": dim, "vdim": dim, "scale": 4.0 / dim, "softcap": 50.0, "mask": {"size": DESIGN_WINDOW}}
+    moe = {"kind": "moe", "expert": {"ff": ff // 4}, "router": {"experts": 16, "top": 4}, "shared": {"ff": ff // 4}}
+    mlps = [{"kind": "dense", "ff": ff}, moe]
+    return {"architecture": "Panolorn", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "embedding": {"scale": width ** 0.5},
+            "layers": [{"type": "attention", "mixer": att, "mlp": mlps[i % 2]} for i in range(layers)]}
+
+
 def qwen3_of(size: str, vocab: int = 32000) -> dict:
     width, heads, kv, dim, ff, layers = DESIGN_SIZES[size]
     return dict(architectures=["Qwen3ForCausalLM"], model_type="qwen3", vocab_size=vocab, hidden_size=width,
@@ -228,7 +240,8 @@ def compare_designs(args) -> int:
     T, B, ctx = args.designs_prompt, args.batch, args.designs_prompt
     families = {"venizen": [("venizen", venizen_of)], "varunex": [("varunex", varunex_of), ("venizen", venizen_of)],
                 "zasudra": [("zasudra", zasudra_of), ("venizen", venizen_of)],
-                "zunilorn": [("zunilorn", zunilorn_of), ("zasudra", zasudra_of)]}
+                "zunilorn": [("zunilorn", zunilorn_of), ("zasudra", zasudra_of)],
+                "panolorn": [("panolorn", panolorn_of), ("zasudra", zasudra_of)]}
     designs = families[args.design_family] + [("qwen3", qwen3_of)]
     out = {"metric": "prefill and decode tokens/s, " + " and ".join(d.capitalize() for d, _ in designs[:-1]) +
                      " beside Qwen3 at equal layer sizes", "dtype": "bf16",
@@ -315,9 +328,9 @@ def main() -> int:
                     help="instead of the default workload: a design (--design-family) beside Qwen3 at equal layer sizes, "
                          f"a list of {','.join(DESIGN_SIZES)} (prefill and decode tokens/s, time per kernel)")
     ap.add_argument("--designs-prompt", type=int, default=2048, help="prompt and decode context of --designs")
-    ap.add_argument("--design-family", default="venizen", choices=["venizen", "varunex", "zasudra", "zunilorn"],
+    ap.add_argument("--design-family", default="venizen", choices=["venizen", "varunex", "zasudra", "zunilorn", "panolorn"],
                     help="the design --designs measures: venizen, or varunex or zasudra (with Venizen, their closest "
-                         "relative, beside it), or zunilorn (with Zasudra beside it)")
+                         "relative, beside it), or zunilorn or panolorn (with Zasudra beside it)")
     args = ap.parse_args()
     if args.impl == "reference":
         return reference_arm(args)

@@ -1,7 +1,7 @@
 from .attention import AttentionMixer
 from .base import (Block, EmbeddingStage, FeedForward, Mixer, Norm, PagedKVSpec, Part, PlanContext,
                    PositionEncoding, StateSpec)
-from .block import HyperConnectionBlock, ParallelBlock, PreNormBlock
+from .block import HyperConnectionBlock, ParallelBlock, PreNormBlock, SandwichNormBlock
 from .latent import LatentAttentionMixer
 from .embedding import OutputHead, TokenEmbedding
 from .mlp import DenseFeedForward, GatedFeedForward, SwiGLUFeedForward
@@ -15,4 +15,4 @@ __all__ = ["AttentionMixer", "Block", "EmbeddingStage", "FeedForward", "Mixer", 
            "SwiGLUFeedForward", "RMSNorm", "NoPositionEncoding", "RotaryEncoding", "DeltaRuleMixer", "ParallelMixer",
            "PolyNormFeedForward", "RetentionMixer", "ParallelBlock", "LatentAttentionMixer", "DenseFeedForward",
            "LayerNorm", "GatedMemoryMixer", "StretchedRotaryEncoding", "HyperConnectionBlock", "GatedFeedForward",
-           "StateSpaceMixer", "YarnRotaryEncoding"]
+           "StateSpaceMixer", "YarnRotaryEncoding", "SandwichNormBlock"]

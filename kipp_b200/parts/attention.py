@@ -52,12 +52,14 @@ class AttentionMixer(Mixer):
         self.lambda_init, self.combine_eps = lambda_init, combine_eps
         # sink: none, learned (a number per head in the softmax's denominator) or unit; head_gate: a sigmoid gate
         # per head from the mixer's input; softcap c > 0: scores c tanh(s / c); `more`: further options of the
-        # part by their plan names (norm_whole, interleaved, chunk, values_are_keys, shared_kv)
+        # part by their plan names (norm_whole, unit_norm, interleaved, chunk, forget_blocks, distance_slopes,
+        # element_gate, values_are_keys, shared_kv)
         self.sink, self.head_gate, self.softcap, self.more = sink, bool(head_gate), float(softcap), dict(more)
 
     def cache_spec(self) -> PagedKVSpec:
         # (the maps of a key head lie side by side in one row of the key pages)
-        return PagedKVSpec(self.num_kv_heads, self.score_maps * self.head_dim, self.window,
+        return PagedKVSpec(self.num_kv_heads, self.score_maps * self.head_dim,
+                           self.more["chunk"] if self.more.get("forget_blocks") else self.window,
                            self.value_dim or (self.head_dim if self.score_maps > 1 else None),
                            self.keep_first if self.window else 0)
 

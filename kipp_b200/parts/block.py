@@ -39,6 +39,25 @@ class ParallelBlock(Block):
         return {"names": list(self.names), "norm": described[0], "mixer": described[1], "ffn": described[2]}
 
 
+class SandwichNormBlock(Block):
+    """x += residual_mult * mixer_out_norm(mixer(input_norm(x))); x += residual_mult *
+    ffn_out_norm(ffn(post_norm(x))): an RMS norm on either side of every sublayer.  ``ffn``
+    None (with its two norms): the mixer only.  ``names``: prefixes of the six parts in this
+    order.  The part itself: csrc/host/parts.hpp."""
+    kind = "sandwich_norm_block"
+
+    def __init__(self, input_norm: Norm, mixer: Mixer, mixer_out_norm: Norm, post_norm: Norm | None = None,
+                 ffn: FeedForward | None = None, ffn_out_norm: Norm | None = None, *, residual_mult: float = 1.0,
+                 names: tuple = ("", "mix.", "", "", "mlp.", "")):
+        self.parts = (input_norm, mixer, mixer_out_norm, post_norm, ffn, ffn_out_norm)
+        self.residual_mult, self.names = float(residual_mult), tuple(names)
+
+    def params(self, prefix, ctx) -> dict:
+        roles = ("input_norm", "mixer", "mixer_out_norm", "post_norm", "ffn", "ffn_out_norm")
+        described = {r: None if p is None else p.describe(prefix + n, ctx) for r, p, n in zip(roles, self.parts, self.names)}
+        return {"names": list(self.names), "residual_mult": self.residual_mult, **described}
+
+
 class HyperConnectionBlock(Block):
     """The residual stream as ``streams`` copies: sublayer q reads
     u = sum_s in_q[s] x_s through its RMS norm and its output y joins every copy,

@@ -1,6 +1,6 @@
 """Token embedding and output head.
 
-x_t = float(E[id_t, :]) with no scale (src/kipp.c:2940-2942); logits = W_lm n
+x_t = float(E[id_t, :]), times ``scale`` where given (src/kipp.c:2940-2942); logits = W_lm n
 for the wanted rows only, W_lm being the embedding when tied
 (src/kipp.c:951-956, 3013-3018).  The parts themselves: csrc/host/parts.hpp."""
 from __future__ import annotations
@@ -13,13 +13,15 @@ from .base import EmbeddingStage, Part
 class TokenEmbedding(EmbeddingStage):
     kind = "token_embedding"
 
-    def __init__(self, vocab_size: int, hidden_size: int, weight_name: str = "weight"):
+    def __init__(self, vocab_size: int, hidden_size: int, weight_name: str = "weight", scale: float = 1.0):
+        self.scale = float(scale)
         self.vocab_size = vocab_size
         self.hidden_size = hidden_size
         self.weight_name = weight_name
 
     def params(self, prefix, ctx) -> dict:
-        return {"vocab_size": self.vocab_size, "hidden_size": self.hidden_size, "weight_name": self.weight_name}
+        return {"vocab_size": self.vocab_size, "hidden_size": self.hidden_size, "weight_name": self.weight_name,
+                "scale": self.scale}
 
 
 class OutputHead(Part):

@@ -33,18 +33,20 @@ class DenseFeedForward(FeedForward):
 
 
 class GatedFeedForward(FeedForward):
-    """x += W_down (g sigmoid(alpha g) (u + 1)) with g = min(W_gate n, limit) and
-    u = clamp(W_up n, -limit, limit) (limit 0: none); ``bias``: biases on all three
-    projections; ``row_gate``: the output is also multiplied by sigmoid(w . n), one
+    """x += W_down (act(g) (u + up_add)) with g = min(W_gate n, limit) and
+    u = clamp(W_up n, -limit, limit) (limit 0: none); ``activation``: ``swish``
+    (g sigmoid(alpha g)) or ``gelu_tanh``; ``bias``: biases on all three projections; ``row_gate``: the output is also multiplied by sigmoid(w . n), one
     number per token."""
     kind = "gated_mlp"
 
     def __init__(self, hidden_size: int, intermediate_size: int, *, limit: float = 0.0, alpha: float = 1.0,
-                 bias: bool = False, row_gate: bool = False, names: dict | None = None):
+                 bias: bool = False, row_gate: bool = False, activation: str = "swish", up_add: float = 1.0,
+                 names: dict | None = None):
         self.hidden_size, self.intermediate_size = hidden_size, intermediate_size
+        self.activation, self.up_add = activation, float(up_add)
         self.limit, self.alpha, self.bias, self.row_gate = float(limit), float(alpha), bool(bias), bool(row_gate)
         self.names = dict(names or {})
 
     def params(self, prefix, ctx) -> dict:
         return {"hidden_size": self.hidden_size, "intermediate_size": self.intermediate_size, "limit": self.limit,
-                "alpha": self.alpha, "bias": self.bias, "row_gate": self.row_gate, "names": self.names}
+                "alpha": self.alpha, "activation": self.activation, "up_add": self.up_add, "bias": self.bias, "row_gate": self.row_gate, "names": self.names}
