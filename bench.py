@@ -130,6 +130,7 @@ def reference_arm(args) -> int:
 # (width, heads, kv heads, head size, feed-forward width, layers): layers of real models' sizes
 DESIGN_SIZES = {"1b": (2048, 16, 4, 128, 6144, 4), "4b": (2560, 32, 8, 128, 9728, 4), "8b": (4096, 32, 8, 128, 12288, 2)}
 DESIGN_WINDOW, DESIGN_KEEP = 1024, 4
+DESIGN_BLOCK = 1280         # Panolorn's blocks: a 2,048-token prompt ends in the middle of one
 
 
 def venizen_of(size: str, vocab: int = 32000) -> dict:
@@ -209,11 +210,11 @@ def zunilorn_of(size: str, vocab: int = 32000) -> dict:
 
 
 def panolorn_of(size: str, vocab: int = 32000) -> dict:
-    """Attention in blocks of positions in every layer, beside a dense gated feed-forward and, in every
+    """Attention in blocks of DESIGN_BLOCK positions in every layer, beside a dense gated feed-forward and, in every
     other layer, sixteen experts of a quarter of its width of which a token takes four, with a
     shared expert of the same width."""
     width, heads, kv, dim, ff, layers = DESIGN_SIZES[size]
-    att = {"heads": heads, "kv_heads": kv, "dim": dim, "vdim": dim, "scale": 4.0 / dim, "softcap": 50.0, "mask": {"size": DESIGN_WINDOW}}
+    att = {"heads": heads, "kv_heads": kv, "dim": dim, "vdim": dim, "scale": 4.0 / dim, "softcap": 50.0, "mask": {"size": DESIGN_BLOCK}}
     moe = {"kind": "moe", "expert": {"ff": ff // 4}, "router": {"experts": 16, "top": 4}, "shared": {"ff": ff // 4}}
     mlps = [{"kind": "dense", "ff": ff}, moe]
     return {"architecture": "Panolorn", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "embedding": {"scale": width ** 0.5},

@@ -42,6 +42,7 @@
 // loads, forms all heads' scores from there, mixes and masks them, advances the softmax of each
 // head, and adds the weighted values.  Any sizes, both element types.
 #include "common.cuh"
+#include "attention_extras.cuh"
 #include <math.h>
 #include <algorithm>
 
@@ -85,31 +86,12 @@ __device__ __forceinline__ float dot_row(const float* __restrict__ qs, const bf1
 }
 
 // The visible keys of position p as two runs: [0, kept) and [first, p].
-__device__ __forceinline__ int first_visible(int pos, int window, int chunk) {
-    return chunk > 0 ? pos - pos % chunk : (window > 0 ? max(0, pos - window + 1) : 0);
-}
 __device__ __forceinline__ void visible_runs(int pos, int window, int keep_first, int chunk, int& first, int& kept) {
     first = first_visible(pos, window, chunk);
     kept = chunk > 0 ? 0 : min(keep_first, first);
 }
 
 constexpr int SPLIT_TILES = 2;     // key tiles per run when a step's tokens are cut into runs
-
-// The layout is the host's AttentionExtras (kernels.hpp).
-struct MixExtras {
-    const float* sink;         // [n_q] or null
-    int key_maps;              // score maps per head (at least 1)
-    int values_in_keys;
-    int diff;                  // 1: two maps per head are combined (key_maps must be 2)
-    float lambda, diff_eps, diff_scale;
-    const void* gate;          // [tokens, ld_gate] in the compute type, or null
-    long long ld_gate;
-    int gate_off;
-    int chunk;                 // > 0: blocks of this many positions bound what a query sees (no window then)
-    float softcap;             // > 0: a scaled score s becomes softcap * tanh(s / softcap) (before mix, mask and softmax)
-    int gate_dims;             // 1: the gate is a number per element of every head instead of one per head
-    const float* slopes;       // [n_q] or null
-};
 
 __device__ __forceinline__ float sigmoid_(float x) { return 1.0f / (1.0f + expf(-x)); }
 // the scaled score, capped where the mixer asks for it

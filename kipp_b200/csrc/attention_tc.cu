@@ -49,7 +49,17 @@
 //
 // Sizes: head_dim 64 or 128; page size 8, 16, 32 or a multiple of 64.  Cache
 // layout of a layer: [page][kv_head][slot][D].
+//
+// A second form of the kernel (X, kipp_attn_prefill_tc_ex) takes what the attention_mix kernels take
+// without a mix of the heads: blocks of positions as the mask, capped scores, a number per head taken
+// off per position of distance, a sink in the denominator, a gate per head or per element, a factor on
+// the output, and heads of any multiple of 8 up to 128 whose values may have a size of their own (a
+// tile of 64 columns that a head does not fill is filled with zeros by the TMA unit: the maps end at
+// the head).  The cap is c tanh(x / c) = c - 2 c / (1 + e^(2x / c)), an exponential and a reciprocal per
+// score in float32.  The weights keep float32 precision through the 16-bit product: p = hi + lo with
+// hi = bf16(p), lo = bf16(p - hi), both in the tile's own score buffer, two products per tile.
 #include "common.cuh"
+#include "attention_extras.cuh"
 #include "mbarrier.cuh"
 #include <cuda.h>
 #include <math.h>
@@ -105,6 +115,13 @@ __device__ __forceinline__ void tma_store_2d(const CUtensorMap* map, uint32_t sr
 __device__ __forceinline__ void bulk_commit() { asm volatile("cp.async.bulk.commit_group;" ::: "memory"); }
 // the sources of all earlier bulk-groups of this thread have been read
 __device__ __forceinline__ void bulk_wait_read() { asm volatile("cp.async.bulk.wait_group.read 0;" ::: "memory"); }
+// Box of a 3-dimensional map: columns x, head y, token z.
+__device__ __forceinline__ void tma_load_3d(uint32_t dst, const CUtensorMap* map, uint64_t* bar, int x, int y, int z) {
+    asm volatile(
+        "cp.async.bulk.tensor.3d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%3, %4, %5}], [%2];"
+        ::"r"(dst), "l"(map), "r"(smem_u32(bar)), "r"(x), "r"(y), "r"(z)
+        : "memory");
+}
 // Box of a 4-dimensional map: columns x, slot y, kv head z, page w.
 __device__ __forceinline__ void tma_load_4d(uint32_t dst, const CUtensorMap* map, uint64_t* bar, int x, int y, int z,
                                             int w) {
@@ -192,6 +209,12 @@ __device__ __forceinline__ float fast_exp2(float x) {
     asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
     return y;
 }
+// 1 / x, single instruction (1 / inf = 0)
+__device__ __forceinline__ float fast_rcp(float x) {
+    float y;
+    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
 // true in one lane of the (converged) warp
 __device__ __forceinline__ bool elect_one() {
     uint32_t chosen;
@@ -254,31 +277,40 @@ struct Params {
     float scale_log2;
     uint32_t v_lbo, v_sbo;      // descriptor strides of the MN-major value tile
     int* status;
+    // the X form only
+    int head_dim, v_dim;        // real sizes (the tiles hold D and DV columns)
+    int chunk;
+    float cap_in, cap_out;      // scores capped: e^(2 s scale / c) = 2^(s cap_in), c log2(e) = cap_out; 0: no cap
+    const float* slopes;        // [n_q] or null
+    const float* sink;          // [n_q] or null
+    const bf16* gate; long long ld_gate; int gate_dims;
+    float out_scale;
 };
 
-template <int D> struct Cfg {
-    static constexpr int HALVES = D / 64;
+// D, DV: columns of the query / key tiles and of the value tile (64 or 128)
+template <int D, int DV> struct Cfg {
+    static constexpr int HALVES = D / 64, V_HALVES = DV / 64;
     static constexpr int Q_BYTES = BM * D * 2;
-    static constexpr int KV_BYTES = BN * D * 2;       // one of K or V, one stage
+    static constexpr int K_BYTES = BN * D * 2, V_BYTES = BN * DV * 2;       // one stage
     static constexpr int XCHG_BYTES = 2 * 2 * BM * 4;  // row maxima of the two halves, two parities
     static constexpr int TMEM_COLS = 256;                       // two score buffers (64 each) + O (D), power of two
     // 100,480 bytes at head_dim 128: two CTAs (plus the 1 KB the system keeps per CTA) fit in 227 KB
-    static constexpr size_t SMEM = Q_BYTES + 4 * KV_BYTES + XCHG_BYTES + 144;   // 16 barriers, 2 words
+    static constexpr size_t SMEM = Q_BYTES + 2 * K_BYTES + 2 * V_BYTES + XCHG_BYTES + 144;   // 16 barriers, 2 words
 };
 
-template <int D>
+template <int D, int DV, bool X>
 __global__ void __launch_bounds__(THREADS, 2)
 attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v,
                        const __grid_constant__ CUtensorMap map_k4, const __grid_constant__ CUtensorMap map_v4,
                        const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_out,
                        const Params p) {
-    using C = Cfg<D>;
+    using C = Cfg<D, DV>;
     extern __shared__ __align__(1024) uint8_t smem[];     // swizzled tiles need 1024-byte alignment
     const uint32_t q_tile = smem_u32(smem);
     const uint32_t k_tiles = q_tile + C::Q_BYTES;                  // [2 stages]
-    const uint32_t v_tiles = k_tiles + 2 * C::KV_BYTES;            // [2 stages]
-    float* xchg = reinterpret_cast<float*>(smem + C::Q_BYTES + 4 * C::KV_BYTES);      // [parity][half][row]
-    uint64_t* bars = reinterpret_cast<uint64_t*>(smem + C::Q_BYTES + 4 * C::KV_BYTES + C::XCHG_BYTES);
+    const uint32_t v_tiles = k_tiles + 2 * C::K_BYTES;             // [2 stages]
+    float* xchg = reinterpret_cast<float*>(smem + C::Q_BYTES + 2 * C::K_BYTES + 2 * C::V_BYTES);      // [parity][half][row]
+    uint64_t* bars = reinterpret_cast<uint64_t*>(smem + C::Q_BYTES + 2 * C::K_BYTES + 2 * C::V_BYTES + C::XCHG_BYTES);
     uint64_t* q_full = bars;            // the query tile is in shared memory            (1 + bytes)
     uint64_t* k_full = bars + 1;        // [2] a key stage has landed                    (1 + bytes)
     uint64_t* k_empty = bars + 3;       // [2] its S product has read it                 (1, by commit)
@@ -298,6 +330,9 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
     // Grid (heads, tiles), the last tile of the list first: within an entry the later
     // tiles see more keys, and the long ones should not be the last to start; the
     // heads of a tile, which share its keys and values, start together.
+    // (The X form also runs inside bursts of decoded steps, whose lengths a kernel of the same
+    // graph moves on: it waits first.)
+    if constexpr (X) pdl_wait();
     const int item = gridDim.y - 1 - blockIdx.y;
     const int entry = p.work[2 * item], tile_tok = p.work[2 * item + 1];
     const int h = blockIdx.x, g = h / (p.n_q / p.n_kv);
@@ -305,7 +340,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
     const int ctx = p.context_len[entry];
     // keys the tile may see: from the first token's window start to the last token
     const int tile_first = ctx + tile_tok, tile_last = ctx + min(tile_tok + BM - 1, q_len - 1);
-    const int lo = p.window > 0 ? max(0, tile_first - p.window + 1) : 0, hi = tile_last;
+    const int lo = first_visible(tile_first, p.window, X ? p.chunk : 0), hi = tile_last;
     const int first_tile = lo / BN, last_tile = hi / BN;
     const int n_tiles = last_tile - first_tile + 1;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -341,13 +376,20 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
         const int rb = lane / C::HALVES, half = lane % C::HALVES;
         const bool has_box = rb * p.box_rows < BN;
         const uint32_t dst_off = (uint32_t)(half * (BN * 128) + rb * p.box_rows * 128);
+        // (the value tile's boxes: the same lanes where it is as wide as the key tile)
+        const int v_rb = lane / C::V_HALVES, v_half = lane % C::V_HALVES;
+        const bool v_has_box = v_rb * p.box_rows < BN;
+        const uint32_t v_dst_off = (uint32_t)(v_half * (BN * 128) + v_rb * p.box_rows * 128);
         bool ok = true;
         // The query tile first: rows [qs + tile_tok, + 128) of head h, a box per 64-column half.
         // Rows past the entry's end are another entry's queries (or zeros past the step's last
         // token): their scores are masked and their output rows are never stored.
         if (lane == 0) mbar_expect_tx(q_full, C::Q_BYTES);
         __syncwarp();
-        if (lane < C::HALVES) tma_load_2d(q_tile + lane * (BM * 128), &map_q, q_full, h * D + lane * 64, qs + tile_tok);
+        if (lane < C::HALVES) {
+            if constexpr (X) tma_load_3d(q_tile + lane * (BM * 128), &map_q, q_full, lane * 64, h, qs + tile_tok);
+            else tma_load_2d(q_tile + lane * (BM * 128), &map_q, q_full, h * D + lane * 64, qs + tile_tok);
+        }
         // (This warp shares its scheduler with busy softmax warps and the stages come
         // back to it just in time: every instruction between a stage's release and
         // the issue of its load counts, so what can be is computed before the loop.)
@@ -359,7 +401,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
             // map instead (a box costs the TMA unit about as much whatever its size).
             const int last_slot = min(hi / p.page_size, p.table_width - 1);
             const int page_rows = p.n_kv * p.page_size, head_row = g * p.page_size;
-            const uint32_t whole_off = (uint32_t)(half * (BN * 128));
+            const uint32_t whole_off = (uint32_t)(half * (BN * 128)), v_whole_off = (uint32_t)(v_half * (BN * 128));
             for (int i = 0; i < n_tiles; ++i) {
                 const int kt = first_tile + i, b = i & 1, use = i >> 1;
                 const int slot = kt * p.pages_per_box + rb;
@@ -367,21 +409,27 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
                 const int first_page = __shfl_sync(0xffffffffu, page, 0);
                 const bool whole = __all_sync(0xffffffffu, !has_box || page == first_page + rb) && first_page >= 0;
                 const int row_coord = page >= 0 ? page * page_rows + head_row : p.rows_total;   // beyond the pool: zeros
+                int v_row_coord = row_coord;
+                if constexpr (C::V_HALVES != C::HALVES) {
+                    const int v_slot = kt * p.pages_per_box + v_rb;
+                    const int v_page = (v_has_box && v_slot <= last_slot) ? __ldg(table + v_slot) : -1;
+                    v_row_coord = v_page >= 0 ? v_page * page_rows + head_row : p.rows_total;
+                }
                 if (i >= 2 && ok && !mbar_wait(&k_empty[b], (use - 1) & 1, abort_flag)) ok = false;
-                if (lane == 0) mbar_expect_tx(&k_full[b], C::KV_BYTES);
+                if (lane == 0) mbar_expect_tx(&k_full[b], C::K_BYTES);
                 __syncwarp();
                 if (whole) {
-                    if (rb == 0 && ok) tma_load_4d(k_tiles + b * C::KV_BYTES + whole_off, &map_k4, &k_full[b], half * 64, 0, g, first_page);
+                    if (rb == 0 && ok) tma_load_4d(k_tiles + b * C::K_BYTES + whole_off, &map_k4, &k_full[b], half * 64, 0, g, first_page);
                 } else if (has_box && ok) {
-                    tma_load_2d(k_tiles + b * C::KV_BYTES + dst_off, &map_k, &k_full[b], half * 64, row_coord);
+                    tma_load_2d(k_tiles + b * C::K_BYTES + dst_off, &map_k, &k_full[b], half * 64, row_coord);
                 }
                 if (i >= 2 && ok && !mbar_wait(&v_empty[b], (use - 1) & 1, abort_flag)) ok = false;
-                if (lane == 0) mbar_expect_tx(&v_full[b], C::KV_BYTES);
+                if (lane == 0) mbar_expect_tx(&v_full[b], C::V_BYTES);
                 __syncwarp();
                 if (whole) {
-                    if (rb == 0 && ok) tma_load_4d(v_tiles + b * C::KV_BYTES + whole_off, &map_v4, &v_full[b], half * 64, 0, g, first_page);
-                } else if (has_box && ok) {
-                    tma_load_2d(v_tiles + b * C::KV_BYTES + dst_off, &map_v, &v_full[b], half * 64, row_coord);
+                    if (v_rb == 0 && ok) tma_load_4d(v_tiles + b * C::V_BYTES + v_whole_off, &map_v4, &v_full[b], v_half * 64, 0, g, first_page);
+                } else if (v_has_box && ok) {
+                    tma_load_2d(v_tiles + b * C::V_BYTES + v_dst_off, &map_v, &v_full[b], v_half * 64, v_row_coord);
                 }
             }
         } else {
@@ -389,20 +437,20 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
             for (int i = 0; i < n_tiles; ++i) {
                 const int kt = first_tile + i, b = i & 1, use = i >> 1;
                 int row_coord = p.rows_total;                  // beyond the pool: zeros
-                if (has_box) {
+                if (has_box || v_has_box) {
                     const int j = kt * BN;
                     const int slot = j / p.page_size;
                     const int page = (j <= hi && slot < p.table_width) ? __ldg(table + slot) : -1;
                     if (page >= 0) row_coord = (page * p.n_kv + g) * p.page_size + (j - slot * p.page_size);
                 }
                 if (i >= 2 && ok && !mbar_wait(&k_empty[b], (use - 1) & 1, abort_flag)) ok = false;
-                if (lane == 0) mbar_expect_tx(&k_full[b], C::KV_BYTES);
+                if (lane == 0) mbar_expect_tx(&k_full[b], C::K_BYTES);
                 __syncwarp();
-                if (has_box && ok) tma_load_2d(k_tiles + b * C::KV_BYTES + dst_off, &map_k, &k_full[b], half * 64, row_coord);
+                if (has_box && ok) tma_load_2d(k_tiles + b * C::K_BYTES + dst_off, &map_k, &k_full[b], half * 64, row_coord);
                 if (i >= 2 && ok && !mbar_wait(&v_empty[b], (use - 1) & 1, abort_flag)) ok = false;
-                if (lane == 0) mbar_expect_tx(&v_full[b], C::KV_BYTES);
+                if (lane == 0) mbar_expect_tx(&v_full[b], C::V_BYTES);
                 __syncwarp();
-                if (has_box && ok) tma_load_2d(v_tiles + b * C::KV_BYTES + dst_off, &map_v, &v_full[b], half * 64, row_coord);
+                if (v_has_box && ok) tma_load_2d(v_tiles + b * C::V_BYTES + v_dst_off, &map_v, &v_full[b], v_half * 64, row_coord);
             }
         }
     } else if (warp == 9) {
@@ -424,7 +472,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
             ok = __all_sync(0xffffffffu, ok);
             tc_fence_after();
             const uint32_t acc = tmem_s + b * BN;
-            const uint32_t k_stage = k_tiles + b * C::KV_BYTES;
+            const uint32_t k_stage = k_tiles + b * C::K_BYTES;
             if (elect_one()) {
 #pragma unroll
                 for (int hh = 0; hh < C::HALVES; ++hh) {
@@ -441,7 +489,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
         }
     } else if (warp == 10) {
         // ------------------------------------------------------------ MMA issuer: outputs
-        constexpr uint32_t IDESC_O = idesc(BM, D, 1);
+        constexpr uint32_t IDESC_O = idesc(BM, DV, 1);
         bool ok = true;
         for (int i = 0; i < n_tiles; ++i) {
             const int b = i & 1, use = i >> 1;
@@ -450,13 +498,18 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
             if (ok && !mbar_wait(&p_full[b], use & 1, abort_flag)) ok = false;
             ok = __all_sync(0xffffffffu, ok);
             tc_fence_after();
-            const uint64_t vd = smem_desc(v_tiles + b * C::KV_BYTES, p.v_lbo, p.v_sbo);
+            const uint64_t vd = smem_desc(v_tiles + b * C::V_BYTES, p.v_lbo, p.v_sbo);
             const uint32_t weights = tmem_s + b * BN;
             if (elect_one()) {
 #pragma unroll
                 for (int k = 0; k < BN / 16; ++k)
                     // 16 keys further: 8 columns of P; 16 rows = 2048 bytes in the value tile
                     umma_bf16_a_tmem(tmem_o, weights + 8 * k, vd + 128 * k, IDESC_O, (i > 0 || k > 0) ? 1u : 0u);
+                if constexpr (X) {                         // what the weights' first halves rounded off
+#pragma unroll
+                    for (int k = 0; k < BN / 16; ++k)
+                        umma_bf16_a_tmem(tmem_o, weights + BN / 2 + 8 * k, vd + 128 * k, IDESC_O, 1u);
+                }
                 umma_commit(&v_empty[b]);
                 umma_commit(&p_empty[b]);
                 if (i == n_tiles - 1) umma_commit(o_final);
@@ -471,7 +524,9 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
         const int tok = tile_tok + row;
         const bool live = tok < q_len;
         const int pos = ctx + tok;
-        const int lo_row = p.window > 0 ? max(0, pos - p.window + 1) : 0;
+        const int lo_row = first_visible(pos, p.window, X ? p.chunk : 0);
+        float slope_log2 = 0.f;
+        if constexpr (X) slope_log2 = p.slopes != nullptr ? p.slopes[h] * 1.4426950408889634f : 0.f;
         const uint32_t t_lane = (uint32_t)((warp & 3) * 32) << 16;   // this warp's tensor-memory lanes
         float m_run = -INFINITY, l_run = 0.f;
         bool ok = true;
@@ -485,6 +540,22 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
             float s[HB];
             tmem_ld32(tmem_s + b * BN + t_lane + ch * HB, s);
             const int j0 = kt * BN + ch * HB;
+            if constexpr (X) {
+                // scaled (in units of log2), capped, less the distance term
+                if (p.cap_out > 0.f) {
+#pragma unroll
+                    for (int j = 0; j < HB; ++j)
+                        s[j] = fmaf(-2.f * p.cap_out, fast_rcp(1.f + fast_exp2(s[j] * p.cap_in)), p.cap_out);
+                } else {
+#pragma unroll
+                    for (int j = 0; j < HB; ++j) s[j] *= p.scale_log2;
+                }
+                if (slope_log2 != 0.f) {
+                    const float behind = (float)(j0 - pos);
+#pragma unroll
+                    for (int j = 0; j < HB; ++j) s[j] = fmaf(slope_log2, behind + (float)j, s[j]);
+                }
+            }
             // Masking only where the tile crosses a row's limits (the diagonal, a
             // window's edge, rows beyond the entry): decided per warp.
             if (!__all_sync(0xffffffffu, live && j0 + HB - 1 <= pos && j0 >= lo_row)) {
@@ -508,20 +579,24 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
             // tile's maximum exceeds it by more than RESCALE_SLACK (weights up to
             // 2^RESCALE_SLACK, far inside bfloat16 and the fp32 sums); numerator and
             // denominator carry the same reference, so the quotient is unchanged.
-            const float cand = raw * p.scale_log2;                  // scale > 0: the maximum commutes
+            const float cand = X ? raw : raw * p.scale_log2;        // scale > 0: the maximum commutes
             const float mx = (cand > m_run + RESCALE_SLACK || m_run == -INFINITY) ? fmaxf(m_run, cand) : m_run;
             const float corr = (m_run == -INFINITY) ? 0.f : (mx == m_run ? 1.f : fast_exp2(m_run - mx));
             const float neg_base = (mx == -INFINITY) ? 0.f : -mx;
             float2 sum2 = make_float2(0.f, 0.f);
             const float2 scale2 = make_float2(p.scale_log2, p.scale_log2), base2 = make_float2(neg_base, neg_base);
-            uint32_t packed[HB / 2];
+            uint32_t packed[HB / 2], rest[X ? HB / 2 : 1];
 #pragma unroll
             for (int j = 0; j < HB; j += 2) {
-                const float2 x = fma2(make_float2(s[j], s[j + 1]), scale2, base2);
+                const float2 x = X ? add2(make_float2(s[j], s[j + 1]), base2) : fma2(make_float2(s[j], s[j + 1]), scale2, base2);
                 const float2 pw = make_float2(fast_exp2(x.x), fast_exp2(x.y));
                 sum2 = add2(sum2, pw);
                 __nv_bfloat162 pk = __floats2bfloat162_rn(pw.x, pw.y);
                 packed[j / 2] = *reinterpret_cast<uint32_t*>(&pk);
+                if constexpr (X) {
+                    __nv_bfloat162 lo2 = __floats2bfloat162_rn(pw.x - __low2float(pk), pw.y - __high2float(pk));
+                    rest[j / 2] = *reinterpret_cast<uint32_t*>(&lo2);
+                }
             }
             l_run = l_run * corr + (sum2.x + sum2.y);      // this thread's half of the row's sum
             m_run = mx;
@@ -529,6 +604,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
             // score buffer: both threads of the row hold their scores in registers since
             // they met at the exchange of the maxima above.
             tmem_st16_words(tmem_s + b * BN + t_lane + ch * (HB / 2), packed);
+            if constexpr (X) tmem_st16_words(tmem_s + b * BN + BN / 2 + t_lane + ch * (HB / 2), rest);
             // rescale the output accumulator when some row of the warp moved its maximum
             // (this thread: its half of the columns), once O += P V of the tile before
             // is complete: that is the latest product (the one before it was complete before
@@ -537,7 +613,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
                 if (!mbar_wait(&p_empty[b ^ 1], ((i - 1) >> 1) & 1, abort_flag)) { if (ok) atomicMax(&p.status[2], 2); ok = false; }
                 tc_fence_after();
 #pragma unroll 1
-                for (int c = ch * (D / 2); c < (ch + 1) * (D / 2); c += 32) {
+                for (int c = ch * (DV / 2); c < (ch + 1) * (DV / 2); c += 32) {
                     float o[32];
                     tmem_ld32(tmem_o + t_lane + c, o);
 #pragma unroll
@@ -560,19 +636,43 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
         xl[ch * BM + row] = l_run;
         named_barrier(1 + (warp & 3), 64);
         const float l_row = l_run + xl[(ch ^ 1) * BM + row];
-        const float inv = l_row > 0.f ? 1.f / l_row : 0.f;
-        bf16* dst = p.out + ((size_t)(qs + (live ? tok : 0)) * p.n_q + h) * D;
+        float inv = l_row > 0.f ? 1.f / l_row : 0.f;
+        const int v_dim = X ? p.v_dim : DV;
+        const size_t token = (size_t)(qs + (live ? tok : 0));
+        bf16* dst = p.out + (token * p.n_q + h) * v_dim;
+        const bf16* gate = nullptr;                        // this row's and head's gate, an element per column
+        if constexpr (X) {
+            if (p.sink != nullptr && live) inv = 1.f / (l_row + fast_exp2(p.sink[h] * 1.4426950408889634f - m_run));
+            inv *= p.out_scale;
+            if (p.gate != nullptr && p.gate_dims) gate = p.gate + token * p.ld_gate + (size_t)h * v_dim;
+            else if (p.gate != nullptr) inv *= 1.f / (1.f + expf(-__bfloat162float(p.gate[token * p.ld_gate + h])));
+        }
         // Where all 32 rows of the warp belong to the entry, its 32 x 64 block of the output goes
         // through shared memory (the query tile's, no product reads it any more; 128-byte rows,
         // swizzled as the unit expects) and leaves as ONE box: a thread's own stores would touch 16
         // bytes of 32 different lines each.  A warp at the entry's ragged end writes its rows itself.
         const int w4 = warp & 3;
-        const bool as_box = (D == 128) && tile_tok + w4 * 32 + 31 < q_len;
+        const bool as_box = D == 128 && DV == 128 && v_dim == DV && tile_tok + w4 * 32 + 31 < q_len;
         const uint32_t box = q_tile + ch * (BM * 128) + w4 * (32 * 128);     // 4 KB, 1,024-byte aligned
 #pragma unroll 1
-        for (int c = ch * (D / 2); c < (ch + 1) * (D / 2); c += 32) {
+        for (int c = ch * (DV / 2); c < (ch + 1) * (DV / 2); c += 32) {
             float o[32];
             tmem_ld32(tmem_o + t_lane + c, o);
+            if constexpr (X) {
+                if (gate != nullptr && live) {
+#pragma unroll
+                    for (int k = 0; k < 4; ++k) {
+                        if (c + 8 * k >= v_dim) break;
+                        const uint4 raw4 = *reinterpret_cast<const uint4*>(gate + c + 8 * k);
+                        const __nv_bfloat162* g2 = reinterpret_cast<const __nv_bfloat162*>(&raw4);
+#pragma unroll
+                        for (int e = 0; e < 4; ++e) {
+                            o[8 * k + 2 * e] *= fast_rcp(1.f + fast_exp2(-1.4426950408889634f * __low2float(g2[e])));
+                            o[8 * k + 2 * e + 1] *= fast_rcp(1.f + fast_exp2(-1.4426950408889634f * __high2float(g2[e])));
+                        }
+                    }
+                }
+            }
             if (ok && (live || as_box)) {
                 uint4 pk[4];
                 uint32_t* w = reinterpret_cast<uint32_t*>(pk);
@@ -582,13 +682,14 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
                     w[k] = *reinterpret_cast<uint32_t*>(&h2);
                 }
                 if (as_box) {
-                    const int chunk0 = (c - ch * (D / 2)) >> 3;               // 16-byte chunk of the 128-byte row
+                    const int chunk0 = (c - ch * (DV / 2)) >> 3;               // 16-byte chunk of the 128-byte row
 #pragma unroll
                     for (int k = 0; k < 4; ++k)
                         st_shared_v4(box + lane * 128 + (((chunk0 + k) ^ (lane & 7)) << 4), pk[k]);
                 } else {
 #pragma unroll
-                    for (int k = 0; k < 4; ++k) reinterpret_cast<uint4*>(dst + c)[k] = pk[k];
+                    for (int k = 0; k < 4; ++k)
+                        if (!X || c + 8 * k < v_dim) reinterpret_cast<uint4*>(dst + c)[k] = pk[k];
                 }
             }
         }
@@ -596,7 +697,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
             fence_async_proxy();                           // these stores before the unit's read
             __syncwarp();
             if (lane == 0 && ok) {
-                tma_store_2d(&map_out, box, h * D + ch * 64, qs + tile_tok + w4 * 32);
+                tma_store_2d(&map_out, box, h * DV + ch * 64, qs + tile_tok + w4 * 32);
                 bulk_commit();
                 bulk_wait_read();                          // the shared memory outlives the read
             }
@@ -691,17 +792,31 @@ int pool_map4(CUtensorMap* out, const void* ptr, int n_pages, int n_kv, int page
     return 0;
 }
 
-template <int D> int launch(const CUtensorMap& mk, const CUtensorMap& mv, const CUtensorMap& mk4, const CUtensorMap& mv4,
+// The queries as [tokens][n_q][head_dim]; box = [128 tokens, one head, 64 columns], zeros beyond the head.
+int query_map(CUtensorMap* out, const void* ptr, int tokens, int n_q, int head_dim) {
+    EncodeTiled fn = encode_fn();
+    if (!fn) return (int)cudaErrorNotSupported;
+    cuuint64_t dims[3] = {(cuuint64_t)head_dim, (cuuint64_t)n_q, (cuuint64_t)tokens};
+    cuuint64_t strides[2] = {(cuuint64_t)head_dim * 2, (cuuint64_t)n_q * head_dim * 2};
+    cuuint32_t box[3] = {64u, 1u, (cuuint32_t)BM};
+    cuuint32_t estr[3] = {1, 1, 1};
+    CUresult r = fn(out, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(ptr), dims, strides, box, estr,
+                    CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
+                    CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+    return r != CUDA_SUCCESS ? 1000 + (int)r : 0;
+}
+
+template <int D, int DV, bool X> int launch(const CUtensorMap& mk, const CUtensorMap& mv, const CUtensorMap& mk4, const CUtensorMap& mv4,
                             const CUtensorMap& mq, const CUtensorMap& mo, const Params& p, int items, cudaStream_t s) {
-    using C = Cfg<D>;
+    using C = Cfg<D, DV>;
     static bool configured = false;
     if (!configured) {
-        cudaError_t e = cudaFuncSetAttribute(attn_prefill_tc_kernel<D>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+        cudaError_t e = cudaFuncSetAttribute(attn_prefill_tc_kernel<D, DV, X>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                              (int)C::SMEM);
         if (e != cudaSuccess) return (int)e;
         configured = true;
     }
-    return kipp_launch(attn_prefill_tc_kernel<D>, dim3(p.n_q, items), dim3(THREADS), C::SMEM, s, 1, mk, mv, mk4, mv4, mq, mo, p);
+    return kipp_launch(attn_prefill_tc_kernel<D, DV, X>, dim3(p.n_q, items), dim3(THREADS), C::SMEM, s, 1, mk, mv, mk4, mv4, mq, mo, p);
 }
 }  // namespace
 
@@ -719,21 +834,26 @@ extern "C" int kipp_attn_prefill_tc_page_ok(int page_size) {
 // q: bf16 [tokens][n_q][head_dim], all of the step's tokens (the query tiles come by TMA, which
 // fills what lies past the last token with zeros).
 // k_pages and v_pages: one layer's pool, bf16 [n_pages][n_kv][page_size][head_dim].
-extern "C" int kipp_attn_prefill_tc(void* out, const void* q, int tokens, const void* k_pages, const void* v_pages,
-                                    int n_pages, const int* q_start, const int* context_len,
-                                    const int* block_table, int table_width, int page_size, const int* work,
-                                    int items, int n_q, int n_kv, int head_dim, float scale, int window,
-                                    int* status, void* stream) {
+//
+// `extras` (or null) with v_dim and out_scale: the X form (blocks, cap, slopes, sink, gate; see the head of this
+// file).  Of the options of MixExtras it takes neither score maps nor values that lie in their key rows.
+extern "C" int kipp_attn_prefill_tc_ex_supported(int head_dim, int v_dim, int n_q, int n_kv) {
+    return head_dim >= 16 && head_dim <= 128 && head_dim % 8 == 0 && v_dim >= 16 && v_dim <= 128 && v_dim % 8 == 0 && n_kv > 0 &&
+           n_q % n_kv == 0;
+}
+static int prefill_tc(void* out, const void* q, int tokens, const void* k_pages, const void* v_pages, int n_pages,
+                      const int* q_start, const int* context_len, const int* block_table, int table_width, int page_size,
+                      const int* work, int items, int n_q, int n_kv, int head_dim, int v_dim, float scale, int window,
+                      float out_scale, const MixExtras* ex, int* status, void* stream) {
     if (items <= 0) return 0;
     if (items > 65535) return KIPP_ERR_ARG;
-    if (!kipp_attn_prefill_tc_supported(head_dim, n_q, n_kv) || !kipp_attn_prefill_tc_page_ok(page_size) ||
-        n_pages <= 0 || window < 0 || status == nullptr || tokens <= 0)
+    if (!kipp_attn_prefill_tc_page_ok(page_size) || n_pages <= 0 || window < 0 || status == nullptr || tokens <= 0)
         return KIPP_ERR_ARG;
     if (((uintptr_t)q & 15) || ((uintptr_t)k_pages & 15) || ((uintptr_t)v_pages & 15) || ((uintptr_t)out & 15))
         return -3;
     const long long rows = (long long)n_pages * n_kv * page_size;
     if (rows + BN > 0x7fffffffLL) return KIPP_ERR_ARG;
-    Params p;
+    Params p = {};
     p.out = (bf16*)out; p.q = (const bf16*)q;
     p.q_start = q_start; p.context_len = context_len; p.block_table = block_table; p.work = work;
     p.table_width = table_width; p.page_size = page_size; p.n_q = n_q; p.n_kv = n_kv; p.window = window;
@@ -749,7 +869,7 @@ extern "C" int kipp_attn_prefill_tc(void* out, const void* q, int tokens, const 
     CUtensorMap mk, mv;
     int rc = pool_map(&mk, k_pages, rows, head_dim, p.box_rows);
     if (rc) return rc;
-    rc = pool_map(&mv, v_pages, rows, head_dim, p.box_rows);
+    rc = pool_map(&mv, v_pages, rows, v_dim, p.box_rows);
     if (rc) return rc;
     // pages of fewer than 64 slots: maps whose box is the whole 64-key half of a tile
     CUtensorMap mk4 = mk, mv4 = mv;
@@ -757,16 +877,54 @@ extern "C" int kipp_attn_prefill_tc(void* out, const void* q, int tokens, const 
     if (p.pages_per_box > 1) {
         rc = pool_map4(&mk4, k_pages, n_pages, n_kv, page_size, head_dim, p.pages_per_box);
         if (rc) return rc;
-        rc = pool_map4(&mv4, v_pages, n_pages, n_kv, page_size, head_dim, p.pages_per_box);
+        rc = pool_map4(&mv4, v_pages, n_pages, n_kv, page_size, v_dim, p.pages_per_box);
         if (rc) return rc;
     }
     CUtensorMap mq;
-    rc = pool_map(&mq, q, tokens, n_q * head_dim, BM);
+    rc = ex != nullptr ? query_map(&mq, q, tokens, n_q, head_dim) : pool_map(&mq, q, tokens, n_q * head_dim, BM);
     if (rc) return rc;
-    CUtensorMap mo;                                  // the output as [tokens, n_q x head_dim]: boxes of 32 rows
-    rc = pool_map(&mo, out, tokens, n_q * head_dim, 32);
+    CUtensorMap mo;                                  // the output as [tokens, n_q x v_dim]: boxes of 32 rows
+    rc = pool_map(&mo, out, tokens, n_q * v_dim, 32);
     if (rc) return rc;
     cudaStream_t s = (cudaStream_t)stream;
-    return head_dim == 64 ? launch<64>(mk, mv, mk4, mv4, mq, mo, p, items, s)
-                          : launch<128>(mk, mv, mk4, mv4, mq, mo, p, items, s);
+    if (ex == nullptr)
+        return head_dim == 64 ? launch<64, 64, false>(mk, mv, mk4, mv4, mq, mo, p, items, s)
+                              : launch<128, 128, false>(mk, mv, mk4, mv4, mq, mo, p, items, s);
+    p.head_dim = head_dim; p.v_dim = v_dim; p.chunk = ex->chunk; p.out_scale = out_scale;
+    p.cap_in = ex->softcap > 0.f ? 2.f * p.scale_log2 / ex->softcap : 0.f;
+    p.cap_out = ex->softcap > 0.f ? ex->softcap * 1.4426950408889634f : 0.f;
+    p.slopes = ex->slopes; p.sink = ex->sink;
+    p.gate = static_cast<const bf16*>(ex->gate) + (ex->gate != nullptr ? ex->gate_off : 0);
+    p.ld_gate = ex->ld_gate; p.gate_dims = ex->gate_dims;
+    if (head_dim <= 64)
+        return v_dim <= 64 ? launch<64, 64, true>(mk, mv, mk4, mv4, mq, mo, p, items, s)
+                           : launch<64, 128, true>(mk, mv, mk4, mv4, mq, mo, p, items, s);
+    return v_dim <= 64 ? launch<128, 64, true>(mk, mv, mk4, mv4, mq, mo, p, items, s)
+                       : launch<128, 128, true>(mk, mv, mk4, mv4, mq, mo, p, items, s);
+}
+
+extern "C" int kipp_attn_prefill_tc(void* out, const void* q, int tokens, const void* k_pages, const void* v_pages,
+                                    int n_pages, const int* q_start, const int* context_len,
+                                    const int* block_table, int table_width, int page_size, const int* work,
+                                    int items, int n_q, int n_kv, int head_dim, float scale, int window,
+                                    int* status, void* stream) {
+    if (items > 0 && !kipp_attn_prefill_tc_supported(head_dim, n_q, n_kv)) return KIPP_ERR_ARG;
+    return prefill_tc(out, q, tokens, k_pages, v_pages, n_pages, q_start, context_len, block_table, table_width, page_size, work,
+                      items, n_q, n_kv, head_dim, head_dim, scale, window, 1.f, nullptr, status, stream);
+}
+
+extern "C" int kipp_attn_prefill_tc_ex(void* out, const void* q, int tokens, const void* k_pages, const void* v_pages,
+                                       int n_pages, const int* q_start, const int* context_len,
+                                       const int* block_table, int table_width, int page_size, const int* work,
+                                       int items, int n_q, int n_kv, int head_dim, int v_dim, float scale, int window,
+                                       float out_scale, const void* extras, int* status, void* stream) {
+    if (items <= 0) return 0;
+    const MixExtras* ex = static_cast<const MixExtras*>(extras);
+    if (ex == nullptr || !kipp_attn_prefill_tc_ex_supported(head_dim, v_dim, n_q, n_kv) || ex->key_maps != 1 ||
+        ex->values_in_keys || ex->diff || ex->chunk < 0 || (ex->chunk > 0 && window > 0))
+        return KIPP_ERR_ARG;
+    // a gate per element is read 16 bytes at a time
+    if (ex->gate != nullptr && ex->gate_dims && ((((uintptr_t)ex->gate + 2 * (size_t)ex->gate_off) & 15) || (ex->ld_gate & 7))) return -3;
+    return prefill_tc(out, q, tokens, k_pages, v_pages, n_pages, q_start, context_len, block_table, table_width, page_size, work,
+                      items, n_q, n_kv, head_dim, v_dim, scale, window, out_scale, ex, status, stream);
 }

@@ -409,18 +409,20 @@ inline void AttentionMixer::forward(StepContext& ctx, const LayerRun& run, int m
                                    m.entry_of_token, T, heads_, kv_heads_, head_dim_, write, v_dim_);
         }
         extras.softcap = (float)opt_.softcap;
-        const int* tiles = nullptr;
-        int n_tiles = 0;
+        const int *tiles = nullptr, *wide = nullptr;
+        int n_tiles = 0, n_wide = 0;
         if (mix_planner_) {
             auto it = m.work.find(mix_planner_->key());
             if (it != m.work.end()) {
                 tiles = it->second[0];
+                wide = it->second[1];
                 n_tiles = m.work_sizes.at(mix_planner_->key())[0] / 2;
+                n_wide = m.work_sizes.at(mix_planner_->key())[1] / 2;
             }
         }
         ops.attention_mix(attn, q, cache, ctx.dtype, head_mix_, m.positions, m.entry_of_token, T, heads_ * maps_, kv_heads_,
                           head_dim_, v_dim_, scale_, window_, window_ > 0 ? opt_.keep_first : 0,
-                          (float)opt_.output_scale, tiles, n_tiles, m.q_start, m.context_len, &extras);
+                          (float)opt_.output_scale, tiles, n_tiles, m.q_start, m.context_len, &extras, wide, n_wide);
         const NormFold* emit = fold_emit(ctx, fold_out, hidden_);
         ops.gemm(residual, F32, hidden_, attn, o_dim_, w_o_, o_dim_, dtype_, T, hidden_, o_dim_, EPI_ADD, emit);
         fold_emitted(ctx, emit, hidden_);
@@ -1551,6 +1553,7 @@ inline std::string Engine::info_json() {
     counters.set("stream_decode_launches", ops_.stream_decode_launches);
     counters.set("projections_to_heads", ops_.projections_to_heads);
     counters.set("mix_mma_launches", ops_.mix_mma_launches);
+    counters.set("mix_tc_launches", ops_.mix_tc_launches);
     counters.set("shared_key_launches", ops_.shared_key_launches);
     counters.set("glu_epilogues", ops_.glu_epilogues);
     j.set("counters", std::move(counters));

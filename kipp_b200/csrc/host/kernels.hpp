@@ -76,7 +76,7 @@ struct PagedCacheView {
 };
 
 // Options of the mixed-head attention kernel beside the mix (the layout is the kernel library's
-// MixExtras, attention_mix.cu): a sink per head in the softmax's denominator, several score maps
+// MixExtras, attention_extras.cuh): a sink per head in the softmax's denominator, several score maps
 // per head that share their values (n_q then counts the maps), the combination of two maps into
 // one head, values that are the head of their key rows, a gate per head and token.
 struct AttentionExtras {
@@ -296,12 +296,14 @@ public:
     // shorter ones are cut into runs of keys on the CUDA-core kernel.
     static constexpr int MIX_MMA_MIN_TOKENS = 64;
     // `tiles`: (entry, first token) per attention_mix_tile() tokens over every entry of the step
-    // (MixTilePlanner), or null.
+    // (MixTilePlanner), or null; `wide_tiles`: the same per 128 tokens.  The tcgen05 kernel is taken
+    // where an average tile holds at least this many tokens.
+    static constexpr int WIDE_TILE_MIN_ROWS = 16;
     void attention_mix(void* out, const void* q, const PagedCacheView& cache, int dtype, const float* head_mix,
                        const int* positions, const int* entry_of_token, int tokens, int n_q, int n_kv, int head_dim,
                        int v_dim, float scale, int window, int keep_first, float out_scale, const int* tiles = nullptr,
                        int n_tiles = 0, const int* q_start = nullptr, const int* context_len = nullptr,
-                       const AttentionExtras* extras = nullptr) {
+                       const AttentionExtras* extras = nullptr, const int* wide_tiles = nullptr, int n_wide_tiles = 0) {
         using Fn = int (*)(void*, const void*, const void*, const void*, int, const float*, const int*, const int*,
                            const int*, int, int, int, int, int, int, int, float, int, int, float, int, float*, const void*,
                            int*, void*);
@@ -320,6 +322,22 @@ public:
         // (the tensor-core prompt kernel takes every option but values that lie in their key rows)
         const bool in_keys = extras != nullptr && extras->values_in_keys;
         const int maps = extras != nullptr ? extras->key_maps : 1;
+        // heads that need nothing of one another: a prompt on the tcgen05 kernel, one head of 128 tokens a block
+        const bool separate = head_mix == nullptr && maps == 1 && !in_keys && (window == 0 || keep_first == 0) && extras != nullptr &&
+                              !extras->diff;
+        if (dtype == BF16 && mix_tensor_core && prefill_tensor_core && separate && tokens > MIX_MMA_MIN_TOKENS && wide_tiles != nullptr &&
+            n_wide_tiles > 0 && tokens >= WIDE_TILE_MIN_ROWS * n_wide_tiles && aligned &&
+            attention_tc_ex_supported(*extras, head_dim, v_dim, n_q, n_kv, cache.page_size)) {
+            using Ft = int (*)(void*, const void*, int, const void*, const void*, int, const int*, const int*, const int*, int, int,
+                               const int*, int, int, int, int, int, float, int, float, const void*, int*, void*);
+            static Ft tc = kernel_symbol<Ft>("attention_tc", "kipp_attn_prefill_tc_ex");
+            run(tc(out, q, tokens, cache.k_pages, cache.v_pages, cache.n_pages, q_start, context_len, cache.block_table,
+                   cache.table_width, cache.page_size, wide_tiles, n_wide_tiles, n_q, n_kv, head_dim, v_dim, scale, window, out_scale,
+                   extras, status, stream),
+                "attn_prefill_tc");
+            ++mix_tc_launches;
+            return;
+        }
         if (dtype == BF16 && mix_tensor_core && !in_keys && tokens > MIX_MMA_MIN_TOKENS && tiles != nullptr && n_tiles > 0 &&
             aligned && (maps == 1 || head_mix == nullptr) &&
             mma_ok(n_q, n_kv, head_dim, v_dim, maps, head_mix != nullptr ? 1 : 0) > 0) {
@@ -819,6 +837,16 @@ public:
         return f(head_dim, n_q, n_kv) != 0 && g(page_size) != 0;
     }
 
+    static bool attention_tc_ex_supported(const AttentionExtras& ex, int head_dim, int v_dim, int n_q, int n_kv, int page_size) {
+        using Fn = int (*)(int, int, int, int);
+        using Fp = int (*)(int);
+        static Fn f = kernel_symbol<Fn>("attention_tc", "kipp_attn_prefill_tc_ex_supported");
+        static Fp g = kernel_symbol<Fp>("attention_tc", "kipp_attn_prefill_tc_page_ok");
+        const bool gate_ok = ex.gate == nullptr || !ex.gate_dims ||
+                             ((((uintptr_t)ex.gate + 2 * (size_t)ex.gate_off) & 15) == 0 && ex.ld_gate % 8 == 0);
+        return f(head_dim, v_dim, n_q, n_kv) != 0 && g(page_size) != 0 && gate_ok;
+    }
+
     // The stream cut of a step's decoded tokens, where the planner asks for it and the kernel takes the step.
     static bool decode_stream_ok(int n_decode) {
         using Fn = int (*)(int, int);
@@ -1027,6 +1055,7 @@ public:
     long long stream_decode_launches = 0;   // decode attention dealt out as a stream
     long long projections_to_heads = 0;     // q/k/v projections with norm, rotation and cache write inside
     long long mix_mma_launches = 0;         // launches of the tensor-core kernel of the mixed-head attention
+    long long mix_tc_launches = 0;          // launches of the tcgen05 prompt kernel with the options of that attention
     long long shared_key_launches = 0;      // launches of the tensor-core kernel for one shared key row per token
     long long glu_epilogues = 0;            // gated activations with limits that ran inside a tensor-core product
 };

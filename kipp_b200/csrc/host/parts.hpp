@@ -433,27 +433,31 @@ private:
     bool own_length_;
 };
 
-// The work list of the mixed-head attention's tensor-core prompt kernel: (entry, first token)
-// per tile of `tile` tokens over every entry of the step.
+// The work lists of the mixed-head attention's tensor-core prompt kernels: (entry, first token)
+// per tile of `tile` tokens (mma.sync) and of 128 tokens (tcgen05) over every entry of the step.
 class MixTilePlanner : public WorkPlanner {
 public:
+    static constexpr int WIDE = 128;
     explicit MixTilePlanner(int tile) : tile_(std::max(tile, 1)) {}
     static std::string key_for(int tile) { return format("attention_mix/tiles%d", tile); }
     std::string key() const override { return key_for(tile_); }
-    int sections() const override { return 1; }
+    int sections() const override { return 2; }
     void sizes(const StepShape& s, int* n) const override {
-        int items = 0;
-        for (int q : s.q_lens) items += (q + tile_ - 1) / tile_;
-        n[0] = 2 * items;
+        n[0] = n[1] = 0;
+        for (int q : s.q_lens)
+            for (int k = 0; k < 2; ++k) n[k] += 2 * ((q + width(k) - 1) / width(k));
     }
     void fill(const StepShape& s, int* const* sec) const override {
-        int a = 0;
-        for (int i = 0; i < s.entries; ++i)
-            for (int t = 0; t < s.q_lens[(size_t)i]; t += tile_) { sec[0][a++] = i; sec[0][a++] = t; }
+        for (int k = 0; k < 2; ++k) {
+            int a = 0;
+            for (int i = 0; i < s.entries; ++i)
+                for (int t = 0; t < s.q_lens[(size_t)i]; t += width(k)) { sec[k][a++] = i; sec[k][a++] = t; }
+        }
     }
 
 private:
     int tile_;
+    int width(int section) const { return section == 0 ? tile_ : WIDE; }
 };
 
 // ---------------------------------------------------------------------------------------------

@@ -100,6 +100,44 @@ def test_attention_alone(name, layer, dtype):
     close(out, want, dtype, f"{name} layer {layer}")
 
 
+TENSOR_CORE_SIZES = [  # heads, kv heads, key size, value size, cap, block, page
+    (4, 2, 128, 128, 20.0, 300, 16), (3, 1, 64, 64, None, 77, 8), (2, 2, 96, 96, 30.0, 130, 16), (4, 1, 40, 104, 5.0, 64, 32),
+    (2, 1, 128, 24, 9.0, None, 64), (5, 5, 16, 128, None, None, 16), (2, 1, 72, 64, 15.0, 500, 128), (6, 3, 64, 128, 12.0, 40, 16)]
+
+
+@pytest.mark.parametrize("heads,kv,dim,vdim,cap,block,page", TENSOR_CORE_SIZES)
+def test_prompts_on_the_tensor_cores(heads, kv, dim, vdim, cap, block, page, tmp_path):
+    """Portions of more than 64 tokens on the tcgen05 kernel: head sizes that do not fill its tiles, key and
+    value tiles of unequal width, every page size, several entries in one step (one of them a single
+    token), portions that start anywhere, rows of a tile that see different blocks."""
+    from kipp_b200.engine import Engine, StepEntry
+    cfg = {"architecture": "Panolorn", "vocab": 30, "width": 64, "norm": {"eps": 1e-5},
+           "layers": [attention_layer(heads, kv, dim, vdim, None, 6.0 / dim, cap, block)]}
+    folder = write_folder(str(tmp_path / "m"), cfg, dict(seed=heads + dim, sigma=0.2, norm_jitter=0.1))
+    w = f64(read_weights(folder))
+    eng = Engine.from_folder(folder, dtype="bfloat16", page_size=page, cache_tokens=2048, max_requests=3, max_batch_tokens=1024,
+                             cuda_graphs=False)
+    lengths = {"a": 450, "b": 333, "c": 90}
+    h = {r: torch.randn(n, 64, generator=torch.Generator().manual_seed(n), dtype=torch.float64).bfloat16() for r, n in lengths.items()}
+    want = {r: P.attention(cfg["layers"][0]["mixer"], w, "l0.mix.", h[r].double(), 1e-5) for r in lengths}
+    got = {r: torch.zeros(n, 64) for r, n in lengths.items()}
+    at, launches = dict.fromkeys(lengths, 0), 0
+    for step in ({"a": 200, "b": 129}, {"a": 1, "b": 128, "c": 70}, {"b": 76}, {"a": 249, "c": 20}):
+        rows = torch.cat([h[r][at[r]:at[r] + k] for r, k in step.items()]).cuda().contiguous()
+        out = torch.zeros(len(rows), 64, device="cuda")
+        eng.run_part([StepEntry(r, [0] * k, []) for r, k in step.items()], 0, "mixer", input=rows, residual=out)
+        row, out = 0, out.cpu()
+        for r, k in step.items():
+            got[r][at[r]:at[r] + k] = out[row:row + k]
+            row, at[r] = row + k, at[r] + k
+        launches += 1
+    for r in lengths:
+        close(got[r], want[r], "bfloat16", r, factor=0.1)
+        worst = (((got[r].double() - want[r]) ** 2).sum(1) / (want[r] ** 2).sum(1)).max()
+        assert float(worst) < 2e-3, f"{r}: worst row {float(worst):.2e}"
+    assert eng.info()["counters"]["mix_tc_launches"] == launches
+
+
 def test_small_queries_and_keys_meet_the_eps_of_their_norm(tmp_path):
     """Projections so small that eps is most of the mean square: the norm is x / sqrt(mean(x^2) + eps)."""
     from kipp_b200.engine import Engine, StepEntry
