@@ -374,6 +374,7 @@ attention_mix_merge_kernel(T* __restrict__ out, const float* __restrict__ partia
         const int hl = e / v_dim, d = e % v_dim;
         const float* p = src + (size_t)(h_first + hl) * (v_dim + 2) + 2 + d;
         float o = 0.f;
+#pragma unroll 8
         for (int r = 0; r < runs; ++r) o = fmaf(p[(size_t)r * n_q * (v_dim + 2)], wts[hl * max_runs + r], o);
         merged[e] = o * fac[hl];
     }
@@ -856,6 +857,88 @@ struct SharedKeySmem {
     }
 };
 
+// The softmax step of 16 head rows over a tile of 32 keys: four rows per warp, lane = key (`vis`: the lane's
+// key is seen).  sraw [16][lds] scores; the weights go to phi + plo [16][ldp].
+__device__ __forceinline__ void head_rows_softmax(const float* __restrict__ sraw, int lds, bf16* __restrict__ phi,
+                                                  bf16* __restrict__ plo, int ldp, float* m_run, float* l_run, float* corr,
+                                                  bool vis, int warp, int lane) {
+    float sv[4], mx[4], p[4], ps[4], m_old[4], cf[4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        const int r = warp * 4 + i;
+        sv[i] = vis ? sraw[r * lds + lane] : -INFINITY;
+        m_old[i] = m_run[r];
+        mx[i] = sv[i];
+    }
+#pragma unroll
+    for (int x = 16; x > 0; x >>= 1) {
+#pragma unroll
+        for (int i = 0; i < 4; ++i) mx[i] = fmaxf(mx[i], __shfl_xor_sync(0xffffffffu, mx[i], x));
+    }
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        mx[i] = fmaxf(mx[i], m_old[i]);
+        p[i] = 0.f;
+        cf[i] = 1.f;
+        if (mx[i] != -INFINITY) {
+            p[i] = sv[i] == -INFINITY ? 0.f : expf(sv[i] - mx[i]);
+            cf[i] = m_old[i] == -INFINITY ? 0.f : expf(m_old[i] - mx[i]);
+        }
+        ps[i] = p[i];
+    }
+#pragma unroll
+    for (int x = 16; x > 0; x >>= 1) {
+#pragma unroll
+        for (int i = 0; i < 4; ++i) ps[i] += __shfl_xor_sync(0xffffffffu, ps[i], x);
+    }
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        const int r = warp * 4 + i;
+        const bf16 hi = __float2bfloat16_rn(p[i]);
+        phi[r * ldp + lane] = hi;
+        plo[r * ldp + lane] = __float2bfloat16_rn(p[i] - __bfloat162float(hi));
+        if (lane == 0) {
+            l_run[r] = l_run[r] * cf[i] + ps[i];
+            m_run[r] = mx[i];
+            corr[r] = cf[i];
+        }
+    }
+}
+// o[b] += P V over a tile of 32 keys: 16 head rows, value columns col0 + 8 b of the rows v [32][ldv].
+template <int VB>
+__device__ __forceinline__ void head_rows_accumulate(float (*o)[4], const bf16* __restrict__ phi, const bf16* __restrict__ plo, int ldp,
+                                                     const float* corr, const bf16* __restrict__ v, int ldv, int col0, int v_dim,
+                                                     int gid, int tig) {
+    const float c0 = corr[gid], c1 = corr[gid + 8];
+    uint32_t ah[2][4], al[2][4];
+#pragma unroll
+    for (int s2 = 0; s2 < 2; ++s2) {
+        const int at = gid * ldp + s2 * 16 + tig * 2;
+        ah[s2][0] = *reinterpret_cast<const uint32_t*>(phi + at);
+        ah[s2][1] = *reinterpret_cast<const uint32_t*>(phi + at + 8 * ldp);
+        ah[s2][2] = *reinterpret_cast<const uint32_t*>(phi + at + 8);
+        ah[s2][3] = *reinterpret_cast<const uint32_t*>(phi + at + 8 * ldp + 8);
+        al[s2][0] = *reinterpret_cast<const uint32_t*>(plo + at);
+        al[s2][1] = *reinterpret_cast<const uint32_t*>(plo + at + 8 * ldp);
+        al[s2][2] = *reinterpret_cast<const uint32_t*>(plo + at + 8);
+        al[s2][3] = *reinterpret_cast<const uint32_t*>(plo + at + 8 * ldp + 8);
+    }
+#pragma unroll
+    for (int b = 0; b < VB; ++b) {
+        const int col = col0 + b * 8;
+        if (col >= v_dim) break;
+        o[b][0] *= c0; o[b][1] *= c0; o[b][2] *= c1; o[b][3] *= c1;
+#pragma unroll
+        for (int s2 = 0; s2 < 2; ++s2) {
+            const unsigned short* v0 = reinterpret_cast<const unsigned short*>(v) + (size_t)(s2 * 16 + tig * 2) * ldv + col + gid;
+            const uint32_t b0 = (uint32_t)v0[0] | ((uint32_t)v0[ldv] << 16);
+            const uint32_t b1 = (uint32_t)v0[8 * ldv] | ((uint32_t)v0[9 * ldv] << 16);
+            mma_16816(o[b], ah[s2], b0, b1);
+            mma_16816(o[b], al[s2], b0, b1);
+        }
+    }
+}
+
 template <int VB>
 __global__ void __launch_bounds__(SK_THREADS)
 attention_shared_key_kernel(bf16* __restrict__ out, const bf16* __restrict__ q, const bf16* __restrict__ k_pages,
@@ -946,83 +1029,10 @@ attention_shared_key_kernel(bf16* __restrict__ out, const bf16* __restrict__ q, 
             sraw[(gid + 8) * lds + key + 1] = capped(c[3] * scale, ex.softcap);
         }
         __syncthreads();
-        // ---- a softmax step for four head rows per warp (lane = key)
-        {
-            const bool vis = pg[lane] >= 0;
-            float sv[4], mx[4], p[4], ps[4], m_old[4], cf[4];
-#pragma unroll
-            for (int i = 0; i < 4; ++i) {
-                const int r = warp * 4 + i;
-                sv[i] = vis ? sraw[r * lds + lane] : -INFINITY;
-                m_old[i] = m_run[r];
-                mx[i] = sv[i];
-            }
-#pragma unroll
-            for (int x = 16; x > 0; x >>= 1) {
-#pragma unroll
-                for (int i = 0; i < 4; ++i) mx[i] = fmaxf(mx[i], __shfl_xor_sync(0xffffffffu, mx[i], x));
-            }
-#pragma unroll
-            for (int i = 0; i < 4; ++i) {
-                mx[i] = fmaxf(mx[i], m_old[i]);
-                p[i] = 0.f;
-                cf[i] = 1.f;
-                if (mx[i] != -INFINITY) {
-                    p[i] = sv[i] == -INFINITY ? 0.f : expf(sv[i] - mx[i]);
-                    cf[i] = m_old[i] == -INFINITY ? 0.f : expf(m_old[i] - mx[i]);
-                }
-                ps[i] = p[i];
-            }
-#pragma unroll
-            for (int x = 16; x > 0; x >>= 1) {
-#pragma unroll
-                for (int i = 0; i < 4; ++i) ps[i] += __shfl_xor_sync(0xffffffffu, ps[i], x);
-            }
-#pragma unroll
-            for (int i = 0; i < 4; ++i) {
-                const int r = warp * 4 + i;
-                const bf16 hi = __float2bfloat16_rn(p[i]);
-                phi[r * ldp + lane] = hi;
-                plo[r * ldp + lane] = __float2bfloat16_rn(p[i] - __bfloat162float(hi));
-                if (lane == 0) {
-                    l_run[r] = l_run[r] * cf[i] + ps[i];
-                    m_run[r] = mx[i];
-                    corr[r] = cf[i];
-                }
-            }
-        }
+        head_rows_softmax(sraw, lds, phi, plo, ldp, m_run, l_run, corr, pg[lane] >= 0, warp, lane);
         __syncthreads();
         // ---- O += P V: the value of a key is the head of its row
-        {
-            const float c0 = corr[gid], c1 = corr[gid + 8];
-            uint32_t ah[2][4], al[2][4];
-#pragma unroll
-            for (int s2 = 0; s2 < 2; ++s2) {
-                const int at = gid * ldp + s2 * 16 + tig * 2;
-                ah[s2][0] = *reinterpret_cast<const uint32_t*>(phi + at);
-                ah[s2][1] = *reinterpret_cast<const uint32_t*>(phi + at + 8 * ldp);
-                ah[s2][2] = *reinterpret_cast<const uint32_t*>(phi + at + 8);
-                ah[s2][3] = *reinterpret_cast<const uint32_t*>(phi + at + 8 * ldp + 8);
-                al[s2][0] = *reinterpret_cast<const uint32_t*>(plo + at);
-                al[s2][1] = *reinterpret_cast<const uint32_t*>(plo + at + 8 * ldp);
-                al[s2][2] = *reinterpret_cast<const uint32_t*>(plo + at + 8);
-                al[s2][3] = *reinterpret_cast<const uint32_t*>(plo + at + 8 * ldp + 8);
-            }
-#pragma unroll
-            for (int b = 0; b < VB; ++b) {
-                const int col = col0 + b * 8;
-                if (col >= v_dim) break;
-                o[b][0] *= c0; o[b][1] *= c0; o[b][2] *= c1; o[b][3] *= c1;
-#pragma unroll
-                for (int s2 = 0; s2 < 2; ++s2) {
-                    const unsigned short* v0 = reinterpret_cast<const unsigned short*>(ks) + (size_t)(s2 * 16 + tig * 2) * ldq + col + gid;
-                    const uint32_t b0 = (uint32_t)v0[0] | ((uint32_t)v0[ldq] << 16);
-                    const uint32_t b1 = (uint32_t)v0[8 * ldq] | ((uint32_t)v0[9 * ldq] << 16);
-                    mma_16816(o[b], ah[s2], b0, b1);
-                    mma_16816(o[b], al[s2], b0, b1);
-                }
-            }
-        }
+        head_rows_accumulate<VB>(o, phi, plo, ldp, corr, ks, ldq, col0, v_dim, gid, tig);
     }
     __syncthreads();
     // rows gid and gid + 8 are heads h0 + gid and h0 + gid + 8; a thread holds columns col + 2 tig, + 1
@@ -1076,7 +1086,231 @@ int launch_shared_key(void* out, const void* q, const void* k_pages, const int* 
     if (rc || !split) return rc;
     return launch_merge<bf16>(out, partial, positions, tokens, n_q, v_dim, window, 0, runs, out_scale, ex, s);
 }
+// ---------------------------------------------------------------------------
+// Heads that need nothing of one another over keys and values of their own (grouped-query attention with the
+// options of MixExtras but the mix, the maps and values in keys), for the tokens a step of few tokens brings, in
+// bfloat16 on the tensor cores: the heads of a kv head's group are the rows of the instruction's M, as the heads
+// of a shared key row are above.  A block of 4 warps takes (token, kv head, up to 16 heads of its group[, run of
+// key tiles]); keys and values of the next tile are on their way while the one before is worked on.  Tiles, runs
+// and partial results are those of the CUDA-core kernel, so the same merge kernel finishes.
+struct GroupSmem {
+    int ldk, ldv, lds, ldp;
+    size_t qs, ks, vs, phi, plo, sraw, m_run, l_run, corr, pg, bytes;     // ks, vs, pg: two stages each
+    __host__ __device__ GroupSmem(int head_dim, int v_dim) {
+        ldk = head_dim + 8;
+        ldv = v_dim + 8;
+        lds = KT + 1;
+        ldp = KT + 8;
+        size_t at = 0;
+        qs = at; at += (size_t)SK_ROWS * ldk * 2;
+        ks = at; at += (size_t)2 * KT * ldk * 2;
+        vs = at; at += (size_t)2 * KT * ldv * 2;
+        phi = at; at += (size_t)SK_ROWS * ldp * 2;
+        plo = at; at += (size_t)SK_ROWS * ldp * 2;
+        sraw = at; at += (size_t)SK_ROWS * lds * 4;
+        m_run = at; at += SK_ROWS * 4;
+        l_run = at; at += SK_ROWS * 4;
+        corr = at; at += SK_ROWS * 4;
+        pg = at; at += 2 * KT * 4;
+        bytes = at;
+    }
+};
+
+template <int VB>
+__global__ void __launch_bounds__(SK_THREADS)
+attention_group_kernel(bf16* __restrict__ out, const bf16* __restrict__ q, const bf16* __restrict__ k_pages,
+                       const bf16* __restrict__ v_pages, const int* __restrict__ positions,
+                       const int* __restrict__ entry_of_token, const int* __restrict__ block_table, int table_width,
+                       int page_size, int n_q, int n_kv, int head_dim, int v_dim, float scale, int window, float out_scale,
+                       int split, float* __restrict__ partial, int* __restrict__ status, const MixExtras ex) {
+    extern __shared__ __align__(16) unsigned char raw[];
+    const GroupSmem L(head_dim, v_dim);
+    bf16* qs = reinterpret_cast<bf16*>(raw + L.qs);
+    bf16* phi = reinterpret_cast<bf16*>(raw + L.phi);
+    bf16* plo = reinterpret_cast<bf16*>(raw + L.plo);
+    float* sraw = reinterpret_cast<float*>(raw + L.sraw);
+    float* m_run = reinterpret_cast<float*>(raw + L.m_run);
+    float* l_run = reinterpret_cast<float*>(raw + L.l_run);
+    float* corr = reinterpret_cast<float*>(raw + L.corr);
+    const int ldk = L.ldk, ldv = L.ldv, lds = L.lds, ldp = L.ldp;
+    pdl_launch_dependents();
+    pdl_wait();
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int gid = lane >> 2, tig = lane & 3;
+    const int group = n_q / n_kv, per_kv = (group + SK_ROWS - 1) / SK_ROWS;
+    const int t = blockIdx.x, g = blockIdx.y / per_kv;
+    const int h0 = g * group + (blockIdx.y % per_kv) * SK_ROWS, h_end = (g + 1) * group;
+    const int pos = positions[t];
+    const int first = first_visible(pos, window, ex.chunk);
+    const int win0 = first / KT;
+    const int n_tiles = pos / KT - win0 + 1;
+    const int it0 = split ? blockIdx.z * SPLIT_TILES : 0;
+    if (it0 >= n_tiles) return;                    // this token has fewer runs than the step's longest
+    const int it1 = split ? min(n_tiles, it0 + SPLIT_TILES) : n_tiles;
+    const int* table = block_table + (size_t)entry_of_token[t] * table_width;
+    const int kchunks = head_dim / 8, vchunks = v_dim / 8;
+
+    // four threads per row of the tile: its page, then its 16-byte chunks
+    auto fetch = [&](int it, int stage) {
+        const int rr = tid >> 2, j = (win0 + it) * KT + rr;
+        int page = -1;
+        if (j >= first && j <= pos) {
+            page = j / page_size < table_width ? table[j / page_size] : -1;
+            if (page < 0 && (tid & 3) == 0) atomicExch(status, 3);        // a needed key is not mapped
+        }
+        const bool ok = page >= 0;
+        const size_t row = ok ? ((size_t)page * n_kv + g) * page_size + j % page_size : 0;
+        const uint32_t kd = smem_address(reinterpret_cast<bf16*>(raw + L.ks) + (size_t)(stage * KT + rr) * ldk);
+        const uint32_t vd = smem_address(reinterpret_cast<bf16*>(raw + L.vs) + (size_t)(stage * KT + rr) * ldv);
+        for (int c = tid & 3; c < kchunks; c += 4) cp_async16(kd + c * 16, k_pages + row * head_dim + c * 8, ok ? 16 : 0);
+        for (int c = tid & 3; c < vchunks; c += 4) cp_async16(vd + c * 16, v_pages + row * v_dim + c * 8, ok ? 16 : 0);
+        if ((tid & 3) == 0) reinterpret_cast<int*>(raw + L.pg)[stage * KT + rr] = page;
+    };
+    static_assert(SK_THREADS / 4 == KT, "four threads per row of a tile");
+
+    fetch(it0, 0);
+    cp_async_commit();
+    for (int i = tid; i < SK_ROWS * kchunks; i += SK_THREADS) {
+        const int c = i % kchunks, r = i / kchunks;
+        uint4 v = make_uint4(0u, 0u, 0u, 0u);
+        if (h0 + r < h_end) v = *reinterpret_cast<const uint4*>(q + ((size_t)t * n_q + h0 + r) * head_dim + c * 8);
+        *reinterpret_cast<uint4*>(qs + (size_t)r * ldk + c * 8) = v;
+    }
+    if (tid < SK_ROWS) { m_run[tid] = -INFINITY; l_run[tid] = 0.f; corr[tid] = 1.f; }
+    float o[VB][4];
+#pragma unroll
+    for (int b = 0; b < VB; ++b) o[b][0] = o[b][1] = o[b][2] = o[b][3] = 0.f;
+    const int col0 = warp * VB * 8;                                 // this warp's value columns
+    // rows beyond the group repeat its last head's slope (their scores are not stored)
+    const float slope0 = ex.slopes != nullptr ? ex.slopes[min(h0 + gid, h_end - 1)] : 0.f;
+    const float slope1 = ex.slopes != nullptr ? ex.slopes[min(h0 + gid + 8, h_end - 1)] : 0.f;
+
+    for (int it = it0; it < it1; ++it) {
+        const int stage = (it - it0) & 1;
+        if (it + 1 < it1) fetch(it + 1, stage ^ 1);                 // (the tile before has left that stage: the barrier below)
+        cp_async_commit();
+        cp_async_wait<1>();
+        __syncthreads();
+        const bf16* ks = reinterpret_cast<const bf16*>(raw + L.ks) + (size_t)stage * KT * ldk;
+        const bf16* vs = reinterpret_cast<const bf16*>(raw + L.vs) + (size_t)stage * KT * ldv;
+        // ---- S = Q K^T: this warp's 8 keys
+        {
+            float c[4] = {0.f, 0.f, 0.f, 0.f};
+            const bf16* kr = ks + (size_t)(warp * 8 + gid) * ldk + tig * 2;
+            const bf16* qa = qs + (size_t)gid * ldk + tig * 2;
+            for (int k0 = 0; k0 < head_dim; k0 += 16) {
+                uint32_t a[4];
+                a[0] = *reinterpret_cast<const uint32_t*>(qa + k0);
+                a[1] = *reinterpret_cast<const uint32_t*>(qa + 8 * ldk + k0);
+                a[2] = *reinterpret_cast<const uint32_t*>(qa + k0 + 8);
+                a[3] = *reinterpret_cast<const uint32_t*>(qa + 8 * ldk + k0 + 8);
+                mma_16816(c, a, *reinterpret_cast<const uint32_t*>(kr + k0), *reinterpret_cast<const uint32_t*>(kr + k0 + 8));
+            }
+            const int key = warp * 8 + tig * 2, apart = pos - (win0 + it) * KT - key;
+            sraw[gid * lds + key] = fmaf(-slope0, (float)apart, capped(c[0] * scale, ex.softcap));
+            sraw[gid * lds + key + 1] = fmaf(-slope0, (float)(apart - 1), capped(c[1] * scale, ex.softcap));
+            sraw[(gid + 8) * lds + key] = fmaf(-slope1, (float)apart, capped(c[2] * scale, ex.softcap));
+            sraw[(gid + 8) * lds + key + 1] = fmaf(-slope1, (float)(apart - 1), capped(c[3] * scale, ex.softcap));
+        }
+        __syncthreads();
+        head_rows_softmax(sraw, lds, phi, plo, ldp, m_run, l_run, corr, reinterpret_cast<const int*>(raw + L.pg)[stage * KT + lane] >= 0,
+                          warp, lane);
+        __syncthreads();
+        head_rows_accumulate<VB>(o, phi, plo, ldp, corr, vs, ldv, col0, v_dim, gid, tig);
+        __syncthreads();                                            // this stage and the weights may be overwritten
+    }
+    // rows gid and gid + 8 are heads h0 + gid and h0 + gid + 8; a thread holds columns col + 2 tig, + 1
+    const bf16* gate = static_cast<const bf16*>(ex.gate);
+#pragma unroll
+    for (int half = 0; half < 2; ++half) {
+        const int r = gid + 8 * half, h = h0 + r;
+        if (h >= h_end) continue;
+        if (split) {
+            float* dst = partial + (((size_t)t * gridDim.z + blockIdx.z) * n_q + h) * (v_dim + 2);
+            if (warp == 0 && tig == 0) { dst[0] = m_run[r]; dst[1] = l_run[r]; }
+#pragma unroll
+            for (int b = 0; b < VB; ++b) {
+                const int col = col0 + b * 8 + tig * 2;
+                if (col0 + b * 8 >= v_dim) break;
+                dst[2 + col] = o[b][2 * half];
+                dst[2 + col + 1] = o[b][2 * half + 1];
+            }
+            continue;
+        }
+        float f = softmax_factor(m_run[r], l_run[r], ex.sink, h) * out_scale;
+        const bf16* gr = gate == nullptr ? nullptr : gate + (size_t)t * ex.ld_gate + ex.gate_off + (ex.gate_dims ? (size_t)h * v_dim : h);
+        if (gr != nullptr && !ex.gate_dims) f *= sigmoid_(to_f32(*gr));
+        bf16* dst = out + ((size_t)t * n_q + h) * v_dim;
+#pragma unroll
+        for (int b = 0; b < VB; ++b) {
+            const int col = col0 + b * 8 + tig * 2;
+            if (col0 + b * 8 >= v_dim) break;
+            float y0 = o[b][2 * half] * f, y1 = o[b][2 * half + 1] * f;
+            if (gr != nullptr && ex.gate_dims) {
+                y0 *= sigmoid_(to_f32(gr[col]));
+                y1 *= sigmoid_(to_f32(gr[col + 1]));
+            }
+            *reinterpret_cast<__nv_bfloat162*>(dst + col) = __floats2bfloat162_rn(y0, y1);
+        }
+    }
+}
+
+template <int VB>
+int launch_group(void* out, const void* q, const void* k_pages, const void* v_pages, const int* positions,
+                 const int* entry_of_token, const int* block_table, int table_width, int page_size, int tokens, int n_q,
+                 int n_kv, int head_dim, int v_dim, float scale, int window, float out_scale, int runs, float* partial,
+                 int* status, const MixExtras& ex, cudaStream_t s) {
+    const size_t smem = GroupSmem(head_dim, v_dim).bytes;
+    auto kernel = attention_group_kernel<VB>;
+    static size_t allowed = 0;
+    if (smem > 48 * 1024 && smem > allowed) {
+        cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        if (e != cudaSuccess) { cudaGetLastError(); return (int)e; }
+        allowed = smem;
+    }
+    const int split = runs > 1 ? 1 : 0, per_kv = (n_q / n_kv + SK_ROWS - 1) / SK_ROWS;
+    const dim3 grid((unsigned)tokens, (unsigned)(n_kv * per_kv), (unsigned)(split ? runs : 1));
+    int rc = kipp_launch(kernel, grid, dim3(SK_THREADS), smem, s, 1, (bf16*)out, (const bf16*)q, (const bf16*)k_pages,
+                         (const bf16*)v_pages, positions, entry_of_token, block_table, table_width, page_size, n_q, n_kv,
+                         head_dim, v_dim, scale, window, out_scale, split, partial, status, ex);
+    if (rc || !split) return rc;
+    return launch_merge<bf16>(out, partial, positions, tokens, n_q, v_dim, window, 0, runs, out_scale, ex, s);
+}
 }  // namespace
+
+// Whether the tensor-core kernel for groups of heads takes these sizes (bfloat16 only).
+extern "C" int kipp_attention_group_ok(int n_q, int n_kv, int head_dim, int v_dim) {
+    if (n_q <= 0 || n_kv <= 0 || n_q % n_kv || head_dim <= 0 || head_dim % 16 || v_dim <= 0 || v_dim % 8 || v_dim > 256) return 0;
+    if ((long long)n_kv * ((n_q / n_kv + SK_ROWS - 1) / SK_ROWS) > 65535) return 0;
+    return GroupSmem(head_dim, v_dim).bytes <= 200 * 1024 ? 1 : 0;
+}
+
+// n_q heads over n_kv key and value heads; of the options of MixExtras: blocks, cap, slopes, sink and gate.
+extern "C" int kipp_attention_group(void* out, const void* q, const void* k_pages, const void* v_pages,
+                                    const int* positions, const int* entry_of_token, const int* block_table,
+                                    int table_width, int page_size, int tokens, int n_q, int n_kv, int head_dim, int v_dim,
+                                    float scale, int window, float out_scale, int runs, float* partial, const void* extras,
+                                    int* status, void* stream) {
+    if (tokens <= 0) return 0;
+    if (!kipp_attention_group_ok(n_q, n_kv, head_dim, v_dim) || page_size <= 0 || window < 0 || runs < 1 ||
+        (runs > 1 && partial == nullptr) || runs > 65535)
+        return KIPP_ERR_ARG;
+    if ((((uintptr_t)q | (uintptr_t)k_pages | (uintptr_t)v_pages | (uintptr_t)out) & 15) != 0) return -3;
+    MixExtras ex = {};
+    ex.key_maps = 1;
+    if (extras != nullptr) ex = *static_cast<const MixExtras*>(extras);
+    if (ex.key_maps != 1 || ex.diff || ex.values_in_keys || ex.chunk < 0 || (ex.chunk > 0 && window > 0)) return KIPP_ERR_ARG;
+    cudaStream_t s = (cudaStream_t)stream;
+    const int vb = (v_dim + 31) / 32;
+#define KIPP_GROUP(V)                                                                                                  \
+    return launch_group<V>(out, q, k_pages, v_pages, positions, entry_of_token, block_table, table_width, page_size,   \
+                           tokens, n_q, n_kv, head_dim, v_dim, scale, window, out_scale, runs, partial, status, ex, s)
+    if (vb <= 1) KIPP_GROUP(1);
+    if (vb <= 2) KIPP_GROUP(2);
+    if (vb <= 4) KIPP_GROUP(4);
+    KIPP_GROUP(8);
+#undef KIPP_GROUP
+}
 
 // Whether the tensor-core kernel for one shared key row per token takes these sizes (bfloat16 only).
 extern "C" int kipp_attention_shared_key_ok(int n_q, int head_dim, int v_dim) {

@@ -52,6 +52,7 @@ struct SegmentArgs {
     const int* positions; const int* entry_of_token; const int* block_table;
     int table_width, page_size, tokens, write_cache;
     float eps;
+    int vec;                                 // every row of every segment starts on 16 bytes and holds whole 16-byte pieces
 };
 
 template <typename T>
@@ -120,9 +121,22 @@ head_segments_kernel(const SegmentArgs a, int* __restrict__ status) {
         if (norm_w != nullptr) norm_w += (size_t)hh * D;
     } else if (divided) {
         float ss = 0.f;
-        for (int i = lane; i < D; i += 32) {
-            const float v = to_f32(src[i]) + (bias ? bias[i] : 0.f);
-            ss = fmaf(v, v, ss);
+        if (a.vec && bias == nullptr) {
+            constexpr int VEC = 16 / (int)sizeof(T);
+            for (int i = VEC * lane; i < D; i += 32 * VEC) {
+                const uint4 raw = *reinterpret_cast<const uint4*>(src + i);
+                const T* e = reinterpret_cast<const T*>(&raw);
+#pragma unroll
+                for (int j = 0; j < VEC; ++j) {
+                    const float v = to_f32(e[j]);
+                    ss = fmaf(v, v, ss);
+                }
+            }
+        } else {
+            for (int i = lane; i < D; i += 32) {
+                const float v = to_f32(src[i]) + (bias ? bias[i] : 0.f);
+                ss = fmaf(v, v, ss);
+            }
         }
         inv = 1.0f / sqrtf(warp_sum(ss) / (float)D + a.eps);
     }
@@ -135,6 +149,29 @@ head_segments_kernel(const SegmentArgs a, int* __restrict__ status) {
         if (norm_w != nullptr) v *= norm_w[i];
         return v;
     };
+    if (a.vec && bias == nullptr && cs == nullptr) {
+        // nothing is rotated: 16 bytes per lane and step
+        constexpr int VEC = 16 / (int)sizeof(T);
+        for (int i = VEC * lane; i < D; i += 32 * VEC) {
+            const uint4 raw = *reinterpret_cast<const uint4*>(src + i);
+            const T* e = reinterpret_cast<const T*>(&raw);
+            uint4 packed;
+            T* to = reinterpret_cast<T*>(&packed);
+#pragma unroll
+            for (int j = 0; j < VEC; ++j) {
+                float v = to_f32(e[j]);
+                if (divided) v = v * inv;
+                if (norm_w != nullptr) v *= norm_w[i + j];
+                if (into_cache) {
+                    if (a.write_cache & 2) v = __bfloat162float(__float2bfloat16_rn(v));
+                    v = cache_value(v);
+                }
+                to[j] = from_f32<T>(v);
+            }
+            *reinterpret_cast<uint4*>(dst + i) = packed;
+        }
+        return;
+    }
     for (int i = lane; i < D; i += 32) {
         float v = value(i);
         const int r = i - g.rot_off;
@@ -368,6 +405,16 @@ extern "C" int kipp_head_segments(const void* src, long long ld_src, int dtype, 
         a.total_heads += g.heads;
     }
     a.n_segments = n_segments;
+    // whether every head starts on 16 bytes on both sides and holds whole 16-byte pieces
+    const int piece = dtype == KIPP_DT_F32 ? 4 : 8;
+    uintptr_t bases = (uintptr_t)src | (uintptr_t)k_pages | (uintptr_t)v_pages;
+    long long lengths = ld_src | (long long)(k_pages ? k_row : 0) | (v_pages ? v_row : 0);
+    for (int i = 0; i < n_segments; ++i) {
+        const HeadSegment& g = a.seg[i];
+        bases |= (uintptr_t)g.dst;
+        lengths |= (long long)g.src_off | g.src_stride | g.dim | g.dst_off | (g.target == 0 ? g.dst_stride | g.ld_dst : 0);
+    }
+    a.vec = (bases & 15) == 0 && lengths % piece == 0;
     a.src = src; a.ld_src = ld_src; a.k_pages = k_pages; a.v_pages = v_pages;
     a.k_row = k_row; a.v_row = v_row; a.n_kv = n_kv;
     a.positions = positions; a.entry_of_token = entry_of_token; a.block_table = block_table;

@@ -338,7 +338,9 @@ public:
             ++mix_tc_launches;
             return;
         }
-        if (dtype == BF16 && mix_tensor_core && !in_keys && tokens > MIX_MMA_MIN_TOKENS && tiles != nullptr && n_tiles > 0 &&
+        // (single tokens of many requests are the group kernel's below)
+        const bool group_ok = dtype == BF16 && mix_tensor_core && separate && aligned && attention_group_supported(n_q, n_kv, head_dim, v_dim);
+        if (dtype == BF16 && mix_tensor_core && !in_keys && tokens > MIX_MMA_MIN_TOKENS && !(group_ok && tokens < 2 * n_tiles) && tiles != nullptr && n_tiles > 0 &&
             aligned && (maps == 1 || head_mix == nullptr) &&
             mma_ok(n_q, n_kv, head_dim, v_dim, maps, head_mix != nullptr ? 1 : 0) > 0) {
             run(mma(out, q, cache.k_pages, cache.v_pages, head_mix, tiles, n_tiles, q_start, context_len, cache.block_table,
@@ -355,6 +357,17 @@ public:
                                  cache.table_width * cache.page_size);
         float* partial = runs > 1 ? workspace->get<float>("attention_mix_runs", (size_t)scratch_of(tokens, runs, n_q, v_dim))
                                   : nullptr;
+        if (group_ok) {                            // few tokens: the heads of a kv head are the rows of a tensor-core tile
+            using Fg = int (*)(void*, const void*, const void*, const void*, const int*, const int*, const int*, int, int, int, int,
+                               int, int, int, float, int, float, int, float*, const void*, int*, void*);
+            static Fg group = kernel_symbol<Fg>("attention_mix", "kipp_attention_group");
+            run(group(out, q, cache.k_pages, cache.v_pages, positions, entry_of_token, cache.block_table, cache.table_width,
+                      cache.page_size, tokens, n_q, n_kv, head_dim, v_dim, scale, window, out_scale, runs, partial, extras, status,
+                      stream),
+                "attention_group", runs > 1 ? 2 : 1);
+            ++group_launches;
+            return;
+        }
         // one key row per token that is also its value (a latent), all heads on it: the heads of a
         // token are the rows of a tensor-core tile
         using Fk = int (*)(int, int, int);
@@ -837,6 +850,11 @@ public:
         return f(head_dim, n_q, n_kv) != 0 && g(page_size) != 0;
     }
 
+    static bool attention_group_supported(int n_q, int n_kv, int head_dim, int v_dim) {
+        using Fn = int (*)(int, int, int, int);
+        static Fn f = kernel_symbol<Fn>("attention_mix", "kipp_attention_group_ok");
+        return f(n_q, n_kv, head_dim, v_dim) != 0;
+    }
     static bool attention_tc_ex_supported(const AttentionExtras& ex, int head_dim, int v_dim, int n_q, int n_kv, int page_size) {
         using Fn = int (*)(int, int, int, int);
         using Fp = int (*)(int);
@@ -1055,6 +1073,7 @@ public:
     long long stream_decode_launches = 0;   // decode attention dealt out as a stream
     long long projections_to_heads = 0;     // q/k/v projections with norm, rotation and cache write inside
     long long mix_mma_launches = 0;         // launches of the tensor-core kernel of the mixed-head attention
+    long long group_launches = 0;           // launches of the tensor-core kernel for groups of heads (few tokens)
     long long mix_tc_launches = 0;          // launches of the tcgen05 prompt kernel with the options of that attention
     long long shared_key_launches = 0;      // launches of the tensor-core kernel for one shared key row per token
     long long glu_epilogues = 0;            // gated activations with limits that ran inside a tensor-core product

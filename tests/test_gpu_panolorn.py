@@ -138,6 +138,51 @@ def test_prompts_on_the_tensor_cores(heads, kv, dim, vdim, cap, block, page, tmp
     assert eng.info()["counters"]["mix_tc_launches"] == launches
 
 
+@pytest.mark.parametrize("heads,kv,dim,vdim,cap,block,page", [
+    (4, 2, 128, 128, 20.0, 300, 16), (3, 1, 64, 64, None, 77, 8), (2, 2, 96, 40, 30.0, 130, 16), (20, 1, 48, 104, 5.0, None, 4),
+    (36, 2, 16, 200, 9.0, 50, 64), (5, 5, 32, 8, None, None, 16)])
+def test_few_tokens_on_the_tensor_cores(heads, kv, dim, vdim, cap, block, page, tmp_path):
+    """Steps of at most 64 tokens (decoded tokens, short portions, both) and a step of 70 single tokens on the
+    kernel whose rows are the heads of a group: groups of one head to more than a tile's sixteen, value
+    heads up to 200, contexts of several runs of key tiles."""
+    from kipp_b200.engine import Engine, StepEntry
+    cfg = {"architecture": "Panolorn", "vocab": 30, "width": 64, "norm": {"eps": 1e-5},
+           "layers": [attention_layer(heads, kv, dim, vdim, None, 6.0 / dim, cap, block)]}
+    folder = write_folder(str(tmp_path / "m"), cfg, dict(seed=heads + dim, sigma=0.2, norm_jitter=0.1))
+    w = f64(read_weights(folder))
+    eng = Engine.from_folder(folder, dtype="bfloat16", page_size=page, cache_tokens=8192, max_requests=72, max_batch_tokens=128,
+                             cuda_graphs=False)
+    h = {r: torch.randn(n, 64, generator=torch.Generator().manual_seed(n), dtype=torch.float64).bfloat16()
+         for r, n in (("a", 400), ("b", 170))}
+    want = {r: P.attention(cfg["layers"][0]["mixer"], w, "l0.mix.", x.double(), 1e-5) for r, x in h.items()}
+    got, at, tick = {r: torch.zeros(len(x), 64) for r, x in h.items()}, dict.fromkeys(h, 0), 0
+    while at["a"] < 400:
+        step = {"a": min([31, 1, 40, 2, 1][tick % 5], 400 - at["a"]), "b": min([1, 24, 1, 1, 17][tick % 5], 170 - at["b"])}
+        step = {r: k for r, k in step.items() if k}
+        rows = torch.cat([h[r][at[r]:at[r] + k] for r, k in step.items()]).cuda().contiguous()
+        out = torch.zeros(len(rows), 64, device="cuda")
+        eng.run_part([StepEntry(r, [0] * k, []) for r, k in step.items()], 0, "mixer", input=rows, residual=out)
+        row, out = 0, out.cpu()
+        for r, k in step.items():
+            got[r][at[r]:at[r] + k] = out[row:row + k]
+            row, at[r] = row + k, at[r] + k
+        tick += 1
+    assert at["b"] == 170
+    for r in h:
+        close(got[r], want[r], "bfloat16", r, factor=0.1)
+        worst = (((got[r].double() - want[r]) ** 2).sum(1) / (want[r] ** 2).sum(1)).max()
+        assert float(worst) < 2e-3, f"{r}: worst row {float(worst):.2e}"
+        eng.finish(r)
+    assert eng.info()["counters"]["group_launches"] == tick
+    x = torch.randn(70, 3, 64, generator=torch.Generator().manual_seed(1), dtype=torch.float64).bfloat16()
+    for k in range(3):
+        out = torch.zeros(70, 64, device="cuda")
+        eng.run_part([StepEntry(i, [0], []) for i in range(70)], 0, "mixer", input=x[:, k].cuda().contiguous(), residual=out)
+    wanted = torch.stack([P.attention(cfg["layers"][0]["mixer"], w, "l0.mix.", x[i].double(), 1e-5)[2] for i in range(70)])
+    close(out, wanted, "bfloat16", "70 single tokens", factor=0.1)
+    assert eng.info()["counters"]["group_launches"] == tick + 3
+
+
 def test_small_queries_and_keys_meet_the_eps_of_their_norm(tmp_path):
     """Projections so small that eps is most of the mean square: the norm is x / sqrt(mean(x^2) + eps)."""
     from kipp_b200.engine import Engine, StepEntry
