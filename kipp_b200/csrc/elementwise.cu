@@ -552,6 +552,188 @@ extern "C" int kipp_norm_add_norm(float* x, float* y, int clear, const void* w_y
     return KIPP_ERR_DTYPE;
 }
 
+// One pass over the residual stream: x[r, :] += mult * sum_b y_b[r, :] * rsqrt(mean(y_b^2) + eps_b) * w_b for up to two
+// outputs y_b that join it normed, and of the new x up to two norms h_q[r, :] = x * rsqrt(mean(x^2) + eps_q) * w_q (what
+// sublayers of the next block read) and its rounded copy.  All float32, h and the copy in the compute type; weights keep
+// their storage type.  A block per row; a thread keeps its first 4 JOIN_KEPT values of every array in registers between
+// the passes over a row, what lies beyond them is read again.  (The layout is the host's Ops::Join.)
+namespace {
+struct JoinArgs {
+    float* x;
+    const float* y[2];
+    const void* w_y[2];
+    void* h[2];
+    const void* w_h[2];
+    void* copy;
+    int w_y_dtype[2], w_h_dtype[2];
+    float eps_y[2], eps_h[2];
+    float mult;
+    int size;
+};
+constexpr int JOIN_KEPT = 2;
+
+// four values of a row at column i (fewer at the end of a row that does not go by fours: VEC false)
+template <bool VEC> __device__ __forceinline__ float4 load_four(const float* p, int i, int n) {
+    if (VEC) return *reinterpret_cast<const float4*>(p + i);
+    return make_float4(p[i], i + 1 < n ? p[i + 1] : 0.f, i + 2 < n ? p[i + 2] : 0.f, i + 3 < n ? p[i + 3] : 0.f);
+}
+template <bool VEC> __device__ __forceinline__ float4 weight_four(const void* w, int dtype, int i, int n) {
+    if (VEC) return weights4(w, dtype, i);
+    return make_float4(load_w(w, dtype, i), i + 1 < n ? load_w(w, dtype, i + 1) : 0.f, i + 2 < n ? load_w(w, dtype, i + 2) : 0.f,
+                       i + 3 < n ? load_w(w, dtype, i + 3) : 0.f);
+}
+template <bool VEC, typename TO> __device__ __forceinline__ void store_four(TO* p, int i, int n, float4 v) {
+    if (VEC) {
+        store4(p + i, v);
+        return;
+    }
+    const float e[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+    for (int k = 0; k < 4; ++k)
+        if (i + k < n) p[i + k] = from_f32<TO>(e[k]);
+}
+
+template <typename TO, int NY, bool VEC>
+__global__ void __launch_bounds__(512)
+stream_join_kernel(const JoinArgs a) {
+    __shared__ float scratch[32];
+    pdl_launch_dependents();
+    pdl_wait();
+    const int n = a.size, tid = threadIdx.x, step = 4 * blockDim.x;
+    const size_t row = (size_t)blockIdx.x * n;
+    float* xr = a.x + row;
+    const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+    float4 xs[JOIN_KEPT], ys[NY > 0 ? NY : 1][JOIN_KEPT];
+    float inv[NY > 0 ? NY : 1];
+#pragma unroll
+    for (int j = 0; j < JOIN_KEPT; ++j) {
+        const int i = 4 * tid + j * step;
+        xs[j] = i < n ? load_four<VEC>(xr, i, n) : zero;
+#pragma unroll
+        for (int b = 0; b < NY; ++b) ys[b][j] = i < n ? load_four<VEC>(a.y[b] + row, i, n) : zero;
+    }
+#pragma unroll
+    for (int b = 0; b < NY; ++b) {
+        float ss = 0.f;
+#pragma unroll
+        for (int j = 0; j < JOIN_KEPT; ++j) ss = squares4(ys[b][j], ss);
+        for (int i = 4 * tid + JOIN_KEPT * step; i < n; i += step) ss = squares4(load_four<VEC>(a.y[b] + row, i, n), ss);
+        inv[b] = a.mult / sqrtf(block_sum(ss, scratch) / (float)n + a.eps_y[b]);
+    }
+    auto joined = [&](float4 x, const float4* y, int i) {
+#pragma unroll
+        for (int b = 0; b < NY; ++b) {
+            const float4 w = weight_four<VEC>(a.w_y[b], a.w_y_dtype[b], i, n);
+            x.x = fmaf(y[b].x * inv[b], w.x, x.x); x.y = fmaf(y[b].y * inv[b], w.y, x.y);
+            x.z = fmaf(y[b].z * inv[b], w.z, x.z); x.w = fmaf(y[b].w * inv[b], w.w, x.w);
+        }
+        if (NY > 0) store_four<VEC>(xr, i, n, x);
+        if (a.copy != nullptr) store_four<VEC>(static_cast<TO*>(a.copy) + row, i, n, x);
+        return x;
+    };
+    float ss = 0.f;
+#pragma unroll
+    for (int j = 0; j < JOIN_KEPT; ++j) {
+        const int i = 4 * tid + j * step;
+        if (i < n) {
+            float4 y[NY > 0 ? NY : 1];
+#pragma unroll
+            for (int b = 0; b < NY; ++b) y[b] = ys[b][j];
+            xs[j] = joined(xs[j], y, i);
+            ss = squares4(xs[j], ss);
+        }
+    }
+    for (int i = 4 * tid + JOIN_KEPT * step; i < n; i += step) {
+        float4 y[NY > 0 ? NY : 1];
+#pragma unroll
+        for (int b = 0; b < NY; ++b) y[b] = load_four<VEC>(a.y[b] + row, i, n);
+        ss = squares4(joined(load_four<VEC>(xr, i, n), y, i), ss);
+    }
+    if (a.h[0] == nullptr) return;
+    const float mean = block_sum(ss, scratch) / (float)n;
+#pragma unroll
+    for (int q = 0; q < 2; ++q) {
+        if (a.h[q] == nullptr) continue;
+        TO* hr = static_cast<TO*>(a.h[q]) + row;
+        const float f = 1.0f / sqrtf(mean + a.eps_h[q]);
+        auto normed = [&](float4 x, int i) {
+            const float4 w = weight_four<VEC>(a.w_h[q], a.w_h_dtype[q], i, n);
+            store_four<VEC>(hr, i, n, make_float4(x.x * f * w.x, x.y * f * w.y, x.z * f * w.z, x.w * f * w.w));
+        };
+#pragma unroll
+        for (int j = 0; j < JOIN_KEPT; ++j) {
+            const int i = 4 * tid + j * step;
+            if (i < n) normed(xs[j], i);
+        }
+        for (int i = 4 * tid + JOIN_KEPT * step; i < n; i += step) normed(load_four<VEC>(xr, i, n), i);
+    }
+}
+
+template <typename TO>
+int launch_stream_join(const JoinArgs& a, int ny, bool vec, int rows, cudaStream_t s) {
+    const dim3 grid((unsigned)rows), block(std::min(512, std::max(64, (a.size / (4 * JOIN_KEPT) + 31) / 32 * 32)));
+#define KIPP_JOIN(N) \
+    return vec ? kipp_launch(stream_join_kernel<TO, N, true>, grid, block, 0, s, 1, a) : kipp_launch(stream_join_kernel<TO, N, false>, grid, block, 0, s, 1, a)
+    if (ny == 0) KIPP_JOIN(0);
+    if (ny == 1) KIPP_JOIN(1);
+    KIPP_JOIN(2);
+#undef KIPP_JOIN
+}
+
+// g[t, k] = gelu(z[t, k]) * e with e the token's row of the table from column `off` on; zeros from dim up to ld_g
+template <typename T>
+__global__ void token_side_gate_kernel(T* __restrict__ g, long long ld_g, const float* __restrict__ z, long long ld_z,
+                                       const T* __restrict__ table, long long ld_table, int off, const int* __restrict__ ids,
+                                       int tokens, int dim, int vocab) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i >= tokens * ld_g) return;
+    const long long t = i / ld_g;
+    const int k = (int)(i % ld_g), id = ids[t];
+    float v = 0.f;
+    if (k < dim && id >= 0 && id < vocab)                  // (the embedding stage reports ids outside the vocabulary)
+        v = kipp_activation(z[t * ld_z + k], 2) * to_f32(table[(size_t)id * ld_table + off + k]);
+    g[i] = from_f32<T>(v);
+}
+}  // namespace
+
+extern "C" int kipp_stream_join(const void* join, int dtype, int rows, void* stream) {
+    if (rows <= 0) return 0;
+    if (join == nullptr) return KIPP_ERR_ARG;
+    const JoinArgs a = *static_cast<const JoinArgs*>(join);
+    if (a.x == nullptr || a.size <= 0 || (a.y[0] == nullptr && a.y[1] != nullptr) || (a.h[0] == nullptr && a.h[1] != nullptr))
+        return KIPP_ERR_ARG;
+    const int ny = a.y[1] != nullptr ? 2 : a.y[0] != nullptr ? 1 : 0;
+    uintptr_t at = (uintptr_t)a.x | (uintptr_t)a.copy;
+    for (int b = 0; b < 2; ++b) {
+        if (a.y[b] != nullptr && (a.w_y[b] == nullptr || !(a.eps_y[b] > 0.f) || (a.w_y_dtype[b] != KIPP_DT_F32 && a.w_y_dtype[b] != KIPP_DT_BF16)))
+            return KIPP_ERR_ARG;
+        if (a.h[b] != nullptr && (a.w_h[b] == nullptr || !(a.eps_h[b] > 0.f) || (a.w_h_dtype[b] != KIPP_DT_F32 && a.w_h_dtype[b] != KIPP_DT_BF16)))
+            return KIPP_ERR_ARG;
+        at |= (uintptr_t)a.y[b] | (uintptr_t)a.h[b] | (a.y[b] ? (uintptr_t)a.w_y[b] : 0) | (a.h[b] ? (uintptr_t)a.w_h[b] : 0);
+    }
+    const bool vec = a.size % 4 == 0 && (at & 15) == 0;
+    if (dtype == KIPP_DT_F32) return launch_stream_join<float>(a, ny, vec, rows, (cudaStream_t)stream);
+    if (dtype == KIPP_DT_BF16) return launch_stream_join<bf16>(a, ny, vec, rows, (cudaStream_t)stream);
+    return KIPP_ERR_DTYPE;
+}
+
+extern "C" int kipp_token_side_gate(void* g, long long ld_g, const float* z, long long ld_z, const void* table, long long ld_table,
+                                    int off, int dtype, const int* ids, int tokens, int dim, int vocab, void* stream) {
+    if (tokens <= 0) return 0;
+    if (dim <= 0 || ld_g < dim || ld_z < dim || off < 0 || off + dim > ld_table || vocab <= 0) return KIPP_ERR_ARG;
+    const dim3 grid((unsigned)((tokens * ld_g + 255) / 256));
+    cudaStream_t s = (cudaStream_t)stream;
+    if (dtype == KIPP_DT_F32)
+        return kipp_launch(token_side_gate_kernel<float>, grid, dim3(256), 0, s, 1, (float*)g, ld_g, z, ld_z, (const float*)table,
+                           ld_table, off, ids, tokens, dim, vocab);
+    if (dtype == KIPP_DT_BF16)
+        return kipp_launch(token_side_gate_kernel<bf16>, grid, dim3(256), 0, s, 1, (bf16*)g, ld_g, z, ld_z, (const bf16*)table,
+                           ld_table, off, ids, tokens, dim, vocab);
+    return KIPP_ERR_DTYPE;
+}
+
 // x *= scale over n float32 values (logits of a head with a scale).
 __global__ void scale_f32_kernel(float* __restrict__ x, long long n, float scale) {
     pdl_launch_dependents();

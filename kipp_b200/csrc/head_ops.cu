@@ -17,7 +17,7 @@
 // states its layout as data: keys made of parts, biases, rotation of a head's tail.
 //
 // kipp_head_matmul: out[t, h, :] = W_h a[t, h, :] for every head h, W_h [n, k] row-major, with
-// float32 accumulation, all heads in one launch: in bfloat16 on the tensor cores (mma.sync); in
+// float32 accumulation, optionally each element times the sigmoid of a gate of its own, all heads in one launch: in bfloat16 on the tensor cores (mma.sync); in
 // 32-bit, or where rows do not start on 16-byte boundaries, few tokens by a kernel that reads the
 // weights once and more tokens in tiles on the CUDA cores.  (Products with a latent: keys absorbed into queries, values expanded after the
 // weighted sum.)
@@ -191,12 +191,19 @@ head_segments_kernel(const SegmentArgs a, int* __restrict__ status) {
 }
 
 // ---------------------------------------------------------------------------
+// the factor of element n of head h of token m: sigmoid(gate[m, h * N + n]), or 1
+template <typename T>
+__device__ __forceinline__ float gate_factor(const T* __restrict__ gate, long long ld_gate, int m, int h, int N, int n) {
+    return gate == nullptr ? 1.f : 1.0f / (1.0f + expf(-to_f32(gate[(size_t)m * ld_gate + (size_t)h * N + n])));
+}
+
 constexpr int BM = 64, BN = 64, BK = 16, TM = 4, TN = 4;
 
 template <typename T>
 __global__ void __launch_bounds__(256)
 head_matmul_kernel(T* __restrict__ C, const T* __restrict__ A, const T* __restrict__ W, int M, int N, int K,
-                   long long lda, long long a_head, long long w_head, long long ldc, long long c_head) {
+                   long long lda, long long a_head, long long w_head, long long ldc, long long c_head,
+                   const T* __restrict__ gate, long long ld_gate) {
     __shared__ float As[BK][BM + 4];
     __shared__ float Ws[BK][BN + 4];
     pdl_launch_dependents();
@@ -242,7 +249,7 @@ head_matmul_kernel(T* __restrict__ C, const T* __restrict__ A, const T* __restri
 #pragma unroll
         for (int j = 0; j < TN; ++j) {
             const int n = n0 + tx * TN + j;
-            if (n < N) C[(size_t)m * ldc + n] = from_f32<T>(acc[i][j]);
+            if (n < N) C[(size_t)m * ldc + n] = from_f32<T>(acc[i][j] * gate_factor(gate, ld_gate, m, h, N, n));
         }
     }
 }
@@ -253,7 +260,8 @@ constexpr int MT = 8;
 template <typename T>
 __global__ void __launch_bounds__(256)
 head_matvec_kernel(T* __restrict__ C, const T* __restrict__ A, const T* __restrict__ W, int M, int N, int K,
-                   long long lda, long long a_head, long long w_head, long long ldc, long long c_head) {
+                   long long lda, long long a_head, long long w_head, long long ldc, long long c_head,
+                   const T* __restrict__ gate, long long ld_gate) {
     pdl_launch_dependents();
     pdl_wait();
     const int lane = threadIdx.x & 31;
@@ -274,7 +282,7 @@ head_matvec_kernel(T* __restrict__ C, const T* __restrict__ A, const T* __restri
 #pragma unroll
     for (int i = 0; i < MT; ++i) {
         const float s = warp_sum(acc[i]);
-        if (i < rows && lane == 0) C[(size_t)h * c_head + (size_t)(m0 + i) * ldc + n] = from_f32<T>(s);
+        if (i < rows && lane == 0) C[(size_t)h * c_head + (size_t)(m0 + i) * ldc + n] = from_f32<T>(s * gate_factor(gate, ld_gate, m0 + i, h, N, n));
     }
 }
 
@@ -289,7 +297,8 @@ __device__ __forceinline__ void mma_bf16_16816(float* c, const uint32_t* a, uint
 }
 __global__ void __launch_bounds__(128)
 head_matmul_mma_kernel(bf16* __restrict__ C, const bf16* __restrict__ A, const bf16* __restrict__ W, int M, int N, int K,
-                       long long lda, long long a_head, long long w_head, long long ldc, long long c_head) {
+                       long long lda, long long a_head, long long w_head, long long ldc, long long c_head,
+                       const bf16* __restrict__ gate, long long ld_gate) {
     __shared__ __align__(16) bf16 As[HM * HLD];
     __shared__ __align__(16) bf16 Ws[HN * HLD];
     pdl_launch_dependents();
@@ -339,9 +348,11 @@ head_matmul_mma_kernel(bf16* __restrict__ C, const bf16* __restrict__ A, const b
         for (int j = 0; j < HN / 8; ++j) {
             const int n = n0 + j * 8 + tig * 2;
             if (n + 1 < N) {
-                *reinterpret_cast<__nv_bfloat162*>(C + (size_t)m * ldc + n) = __floats2bfloat162_rn(acc[j][2 * half], acc[j][2 * half + 1]);
+                *reinterpret_cast<__nv_bfloat162*>(C + (size_t)m * ldc + n) =
+                    __floats2bfloat162_rn(acc[j][2 * half] * gate_factor(gate, ld_gate, m, h, N, n),
+                                          acc[j][2 * half + 1] * gate_factor(gate, ld_gate, m, h, N, n + 1));
             } else if (n < N) {
-                C[(size_t)m * ldc + n] = __float2bfloat16_rn(acc[j][2 * half]);
+                C[(size_t)m * ldc + n] = __float2bfloat16_rn(acc[j][2 * half] * gate_factor(gate, ld_gate, m, h, N, n));
             }
         }
     }
@@ -359,7 +370,8 @@ __global__ void transpose_heads_kernel(T* __restrict__ out, const T* __restrict_
 
 template <typename T>
 int launch_head_matmul(void* C, const void* A, const void* W, int M, int N, int K, int heads, long long lda,
-                       long long a_head, long long w_head, long long ldc, long long c_head, cudaStream_t s) {
+                       long long a_head, long long w_head, long long ldc, long long c_head, const void* gate, long long ld_gate,
+                       cudaStream_t s) {
     // the tensor-core kernel: bfloat16 at any number of tokens (a decoded token and a prompt's token
     // then sum in the same order), rows of both operands on 16-byte boundaries, results on 4-byte ones
     if (sizeof(T) == 2 && K % 8 == 0 && lda % 8 == 0 && a_head % 8 == 0 && w_head % 8 == 0 && ldc % 2 == 0 &&
@@ -367,17 +379,17 @@ int launch_head_matmul(void* C, const void* A, const void* W, int M, int N, int 
         const dim3 grid((unsigned)((N + HN - 1) / HN), (unsigned)((M + HM - 1) / HM), (unsigned)heads);
         if (grid.y > 65535) return KIPP_ERR_ARG;
         return kipp_launch(head_matmul_mma_kernel, grid, dim3(128), 0, s, 1, (bf16*)C, (const bf16*)A, (const bf16*)W, M, N, K,
-                           lda, a_head, w_head, ldc, c_head);
+                           lda, a_head, w_head, ldc, c_head, (const bf16*)gate, ld_gate);
     }
     if (M <= 2 * MT) {
         const dim3 grid((unsigned)((N + 7) / 8), (unsigned)((M + MT - 1) / MT), (unsigned)heads);
         return kipp_launch(head_matvec_kernel<T>, grid, dim3(256), 0, s, 1, (T*)C, (const T*)A, (const T*)W, M, N, K, lda,
-                           a_head, w_head, ldc, c_head);
+                           a_head, w_head, ldc, c_head, (const T*)gate, ld_gate);
     }
     const dim3 grid((unsigned)((N + BN - 1) / BN), (unsigned)((M + BM - 1) / BM), (unsigned)heads);
     if (grid.y > 65535) return KIPP_ERR_ARG;
     return kipp_launch(head_matmul_kernel<T>, grid, dim3(256), 0, s, 1, (T*)C, (const T*)A, (const T*)W, M, N, K, lda,
-                       a_head, w_head, ldc, c_head);
+                       a_head, w_head, ldc, c_head, (const T*)gate, ld_gate);
 }
 }  // namespace
 
@@ -430,16 +442,24 @@ extern "C" int kipp_head_segments(const void* src, long long ld_src, int dtype, 
 }
 
 // C[t, h, 0:N] = W_h A[t, h, 0:K]: row t of head h of A at A + h * a_head + t * lda, W_h at
-// W + h * w_head as [N, K], the result at C + h * c_head + t * ldc; all in `dtype`.
+// W + h * w_head as [N, K], the result at C + h * c_head + t * ldc; all in `dtype`.  gate (or null), of the same
+// type: the element is also multiplied by sigmoid(gate[t * ld_gate + h * N + n]).
+extern "C" int kipp_head_matmul_gated(void* C, const void* A, const void* W, int dtype, int M, int N, int K, int heads,
+                                      long long lda, long long a_head, long long w_head, long long ldc, long long c_head,
+                                      const void* gate, long long ld_gate, void* stream) {
+    if (M <= 0 || N <= 0 || heads <= 0) return 0;
+    if (K <= 0 || heads > 65535 || (gate != nullptr && ld_gate < (long long)heads * N)) return KIPP_ERR_ARG;
+    cudaStream_t s = (cudaStream_t)stream;
+    if (dtype == KIPP_DT_F32)
+        return launch_head_matmul<float>(C, A, W, M, N, K, heads, lda, a_head, w_head, ldc, c_head, gate, ld_gate, s);
+    if (dtype == KIPP_DT_BF16)
+        return launch_head_matmul<bf16>(C, A, W, M, N, K, heads, lda, a_head, w_head, ldc, c_head, gate, ld_gate, s);
+    return KIPP_ERR_DTYPE;
+}
 extern "C" int kipp_head_matmul(void* C, const void* A, const void* W, int dtype, int M, int N, int K, int heads,
                                 long long lda, long long a_head, long long w_head, long long ldc, long long c_head,
                                 void* stream) {
-    if (M <= 0 || N <= 0 || heads <= 0) return 0;
-    if (K <= 0 || heads > 65535) return KIPP_ERR_ARG;
-    cudaStream_t s = (cudaStream_t)stream;
-    if (dtype == KIPP_DT_F32) return launch_head_matmul<float>(C, A, W, M, N, K, heads, lda, a_head, w_head, ldc, c_head, s);
-    if (dtype == KIPP_DT_BF16) return launch_head_matmul<bf16>(C, A, W, M, N, K, heads, lda, a_head, w_head, ldc, c_head, s);
-    return KIPP_ERR_DTYPE;
+    return kipp_head_matmul_gated(C, A, W, dtype, M, N, K, heads, lda, a_head, w_head, ldc, c_head, nullptr, 0, stream);
 }
 
 // out[h] = in[h]^T for `heads` row-major matrices of [rows, cols] in `dtype`.

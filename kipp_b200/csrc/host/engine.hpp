@@ -21,7 +21,7 @@
 #include "expert_parts.hpp"
 #include "zasudra.hpp"
 #include "zunilorn.hpp"
-#include "panolorn.hpp"
+#include "nogavik.hpp"
 
 namespace kipp {
 
@@ -327,7 +327,7 @@ inline void AttentionMixer::forward(StepContext& ctx, const LayerRun& run, int m
     Ops& ops = *ctx.ops;
     const StepMeta& m = *ctx.meta;
     const int qkv_cols = proj_ld_;                                      // the row pitch of the fused projection
-    NormFold fold_in, fold_out;
+    NormFold fold_in;
     const PagedCacheView cache = ctx.cache_view(run, mixer_slot);       // pages of this run's cache id
     const int rot = position_->rotary_dim();
     const bool to_heads = !mix_path_ && ctx.dtype == dtype_ && !ctx.kv_round_bf16 &&
@@ -347,8 +347,8 @@ inline void AttentionMixer::forward(StepContext& ctx, const LayerRun& run, int m
         void* q = ctx.workspace->buffer("q", (size_t)T * q_dim_ * es);
         const int write = (run.writes_cache ? 1 : 0) | (ctx.kv_round_bf16 && ctx.dtype == F32 ? 2 : 0);
         AttentionExtras extras;
-        if (segments_ && !opt_.bias && maps_ == 1) {
-            // the norm over the whole projection, the pairing of the rotation, keys that are also the
+        if (segments_ && maps_ == 1) {
+            // biases, the norm over the whole projection, the pairing of the rotation, keys that are also the
             // values, a mixer without keys of its own: each a property of a run of heads
             if (opt_.shared_kv == run.writes_cache)
                 fail(KIPP_E_CONFIG, "attention: a mixer with shared_kv runs with writes_cache false, any other with true");
@@ -358,18 +358,18 @@ inline void AttentionMixer::forward(StepContext& ctx, const LayerRun& run, int m
             const float* kw = qk_norm_ ? static_cast<const float*>(k_norm_) : nullptr;
             HeadSegment& sq = seg[n++];
             sq.src_off = 0; sq.heads = heads_; sq.dim = head_dim_; sq.src_stride = head_dim_;
-            sq.norm_w = qw; sq.norm_all = opt_.norm_whole ? 1 : 0; sq.unit_norm = opt_.unit_norm ? 1 : 0;
+            sq.norm_w = qw; sq.norm_all = opt_.norm_whole ? 1 : 0; sq.unit_norm = opt_.unit_norm ? 1 : 0; sq.bias = q_bias_;
             sq.rot = rot; sq.cos_sin = cos_sin; sq.interleaved = opt_.interleaved ? 1 : 0;
             sq.target = 0; sq.dst = q; sq.ld_dst = q_dim_; sq.dst_stride = head_dim_;
             if (k_cols_) {
                 HeadSegment& sk = seg[n++];
                 sk.src_off = q_dim_; sk.heads = kv_heads_; sk.dim = head_dim_; sk.src_stride = head_dim_;
-                sk.norm_w = kw; sk.norm_all = opt_.norm_whole ? 1 : 0; sk.unit_norm = opt_.unit_norm ? 1 : 0;
+                sk.norm_w = kw; sk.norm_all = opt_.norm_whole ? 1 : 0; sk.unit_norm = opt_.unit_norm ? 1 : 0; sk.bias = k_bias_;
                 sk.rot = rot; sk.cos_sin = cos_sin; sk.interleaved = opt_.interleaved ? 1 : 0;
                 sk.target = 1; sk.heads_per_row = 1;
                 HeadSegment& sv = seg[n++];                              // the values: W_v's rows, or the keys as projected
                 sv.src_off = opt_.values_are_keys ? q_dim_ : q_dim_ + k_cols_;
-                sv.heads = kv_heads_; sv.dim = v_dim_; sv.src_stride = v_dim_;
+                sv.heads = kv_heads_; sv.dim = v_dim_; sv.src_stride = v_dim_; sv.bias = v_bias_;
                 sv.target = 2; sv.heads_per_row = 1;
             }
             ops.head_segments(qkv, qkv_cols, ctx.dtype, seg, n, &cache, head_dim_, v_dim_, kv_heads_, m.positions,
@@ -384,7 +384,7 @@ inline void AttentionMixer::forward(StepContext& ctx, const LayerRun& run, int m
                 extras.gate_off = 0;
             }
         } else if (segments_) {
-            // biases and score maps: every map of every head is a head of head_dim for the bias and
+            // score maps (with biases): every map of every head is a head of head_dim for the bias and
             // the rotation; the maps of a key head go side by side into one row of the key pages
             HeadSegment seg[3];
             seg[0].src_off = 0; seg[0].heads = heads_ * maps_; seg[0].dim = head_dim_; seg[0].src_stride = head_dim_;
@@ -423,9 +423,7 @@ inline void AttentionMixer::forward(StepContext& ctx, const LayerRun& run, int m
         ops.attention_mix(attn, q, cache, ctx.dtype, head_mix_, m.positions, m.entry_of_token, T, heads_ * maps_, kv_heads_,
                           head_dim_, v_dim_, scale_, window_, window_ > 0 ? opt_.keep_first : 0,
                           (float)opt_.output_scale, tiles, n_tiles, m.q_start, m.context_len, &extras, wide, n_wide);
-        const NormFold* emit = fold_emit(ctx, fold_out, hidden_);
-        ops.gemm(residual, F32, hidden_, attn, o_dim_, w_o_, o_dim_, dtype_, T, hidden_, o_dim_, EPI_ADD, emit);
-        fold_emitted(ctx, emit, hidden_);
+        output_product(ctx, residual, attn, o_dim_, w_o_, o_dim_, dtype_, hidden_, o_dim_);
         return;
     }
     const AttentionWork work = planner_->work_of(m);
@@ -456,9 +454,7 @@ inline void AttentionMixer::forward(StepContext& ctx, const LayerRun& run, int m
                           heads_, kv_heads_, head_dim_, scale_, window_);
         }
     }
-    const NormFold* emit = fold_emit(ctx, fold_out, hidden_);
-    ops.gemm(residual, F32, hidden_, attn, q_dim_, w_o_, q_dim_, dtype_, T, hidden_, q_dim_, EPI_ADD, emit);
-    fold_emitted(ctx, emit, hidden_);
+    output_product(ctx, residual, attn, q_dim_, w_o_, q_dim_, dtype_, hidden_, q_dim_);
 }
 
 // ---------------------------------------------------------------------------------------------
@@ -1221,7 +1217,8 @@ inline void Engine::debug_part(const StepEntryView* entries, int n, int run_inde
     } else if (which == "input_norm") {
         need_pre()->input_norm()->forward(ctx, residual, output, nullptr, T);
     } else if (which == "post_norm") {
-        need_pre()->post_norm()->forward(ctx, residual, output, nullptr, T);
+        if (shared_norm != nullptr && shared_norm->ffn_norm() != nullptr) shared_norm->ffn_norm()->forward(ctx, residual, output, nullptr, T);
+        else need_pre()->post_norm()->forward(ctx, residual, output, nullptr, T);
     } else if (which == "mixer" || which.rfind("mixer/", 0) == 0) {
         // "mixer/<k>": the k-th of the mixers a block holds side by side, with its own cache or state
         const int k = which == "mixer" ? 0 : atoi(which.c_str() + 6);

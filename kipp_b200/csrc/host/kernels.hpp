@@ -406,12 +406,14 @@ public:
     // C[t, h, :] = W_h A[t, h, :] for every head: W_h [N, K] at w + h * w_head, rows of head h at
     // a + h * a_head + t * lda, results at c + h * c_head + t * ldc; one launch for all heads
     // (head_ops.cu chooses between its kernels by the number of tokens, the type and the alignment).
+    // gate (or null): element n of head h of token t is also multiplied by sigmoid(gate[t * ld_gate + h * N + n]).
     void head_matmul(void* c, long long ldc, long long c_head, const void* a, long long lda, long long a_head,
-                     const void* w, long long w_head, int dtype, int M, int N, int K, int heads) {
+                     const void* w, long long w_head, int dtype, int M, int N, int K, int heads, const void* gate = nullptr,
+                     long long ld_gate = 0) {
         using Fn = int (*)(void*, const void*, const void*, int, int, int, int, int, long long, long long, long long,
-                           long long, long long, void*);
-        static Fn f = kernel_symbol<Fn>("head_ops", "kipp_head_matmul");
-        run(f(c, a, w, dtype, M, N, K, heads, lda, a_head, w_head, ldc, c_head, stream), "head_matmul");
+                           long long, long long, const void*, long long, void*);
+        static Fn f = kernel_symbol<Fn>("head_ops", "kipp_head_matmul_gated");
+        run(f(c, a, w, dtype, M, N, K, heads, lda, a_head, w_head, ldc, c_head, gate, ld_gate, stream), "head_matmul");
     }
     // out[h] = in[h]^T for `heads` row-major matrices of [rows, cols]
     void transpose_heads(void* out, const void* in, int dtype, int heads, int rows, int cols) {
@@ -426,7 +428,7 @@ public:
         static Fn f = kernel_symbol<Fn>("recurrent", "kipp_recurrent_scan_ok");
         return f(dim, v_dim, delta ? 1 : 0) != 0;
     }
-    // kind: 0 retention, 1 delta rule, 2 gated memory, 3 wkv
+    // kind: 0 retention, 1 delta rule, 2 gated memory, 3 wkv, 4 state space, 5 gated delta rule
     float* recurrent_scratch(int tokens, int heads, int dim, int v_dim, int kind) {
         using Fn = long long (*)(int, int, int, int, int);
         static Fn f = kernel_symbol<Fn>("recurrent", "kipp_recurrent_scratch_floats");
@@ -544,6 +546,34 @@ public:
         static Fn f = kernel_symbol<Fn>("elementwise", "kipp_norm_add_norm");
         run(f(x, y, clear ? 1 : 0, w_y, w_y_dtype, eps_y, mult, w_h, w_h_dtype, eps_h, h, h_dtype, rows, size, stream),
             "norm_add_norm");
+    }
+    // One pass over the residual stream (elementwise.cu): x += mult * sum_b y_b rsqrt(mean(y_b^2) + eps) w_b for up
+    // to two outputs y_b; of the new x up to two norms h_q = x rsqrt(mean(x^2) + eps) w_q and its rounded copy,
+    // both in the compute type.  The layout is the kernel library's JoinArgs.
+    struct Join {
+        float* x = nullptr;
+        const float* y[2] = {nullptr, nullptr};
+        const void* w_y[2] = {nullptr, nullptr};
+        void* h[2] = {nullptr, nullptr};
+        const void* w_h[2] = {nullptr, nullptr};
+        void* copy = nullptr;
+        int w_y_dtype[2] = {F32, F32}, w_h_dtype[2] = {F32, F32};
+        float eps_y[2] = {0.f, 0.f}, eps_h[2] = {0.f, 0.f};
+        float mult = 1.f;
+        int size = 0;
+    };
+    void stream_join(const Join& j, int dtype, int rows) {
+        using Fn = int (*)(const void*, int, int, void*);
+        static Fn f = kernel_symbol<Fn>("elementwise", "kipp_stream_join");
+        run(f(&j, dtype, rows, stream), "stream_join");
+    }
+    // g[t, k] = gelu_tanh(z[t, k]) * table[ids[t], off + k] in the compute type, zeros from dim up to ld_g
+    void token_side_gate(void* g, long long ld_g, const float* z, long long ld_z, const void* table, long long ld_table, int off,
+                         int dtype, const int* ids, int tokens, int dim, int vocab) {
+        using Fn = int (*)(void*, long long, const float*, long long, const void*, long long, int, int, const int*, int, int, int,
+                           void*);
+        static Fn f = kernel_symbol<Fn>("elementwise", "kipp_token_side_gate");
+        run(f(g, ld_g, z, ld_z, table, ld_table, off, dtype, ids, tokens, dim, vocab, stream), "token_side_gate");
     }
     // Hyper-connections (elementwise.cu): the residual stream as `streams` copies, `stride` floats apart.
     // y given: x_t <- sum_s mix[s, t] x_s + mult out_w[t] y; h given: h = rmsnorm(sum_s in_w[s] x_s).
@@ -728,6 +758,34 @@ public:
               norm_groups, state, slot_stride, q_start, entry_of_token, slots, entries, tokens, heads, groups, dim, v_dim, eps,
               scratch, conv_out, stream),
             "ssd_scan", taps > 1 ? 5 : 4);
+    }
+
+    // The gated delta rule (recurrent.cu, kind 5): convolution, unit keys, decays, the recurrence, norm and gate.
+    static bool gated_delta_ok(int dim, int v_dim) {
+        using Fn = int (*)(int, int, int);
+        static Fn f = kernel_symbol<Fn>("recurrent", "kipp_recurrent_scan_ok");
+        return f(dim, v_dim, 5) != 0;
+    }
+    static long long gated_delta_state_floats(int heads, int kv_heads, int dim, int v_dim, int taps) {
+        using Fn = long long (*)(int, int, int, int, int);
+        static Fn f = kernel_symbol<Fn>("recurrent", "kipp_gated_delta_state_floats");
+        return f(heads, kv_heads, dim, v_dim, taps);
+    }
+    void gated_delta_scan(void* out, long long ld_out, const void* proj, long long ld_proj, int dtype, int qkv_off, int b_off,
+                          const float* conv_w, int taps, const float* a_raw, long long ld_a, const float* dt_bias,
+                          const float* a_log, const float* g_raw, long long ld_g, int gate, const float* norm_w, float* state,
+                          long long slot_stride, const int* q_start, const int* entry_of_token, const int* slots, int entries,
+                          int tokens, int heads, int kv_heads, int dim, int v_dim, float q_scale, float eps, float out_scale) {
+        using Fn = int (*)(void*, long long, const void*, long long, int, int, int, const float*, int, const float*, long long,
+                           const float*, const float*, const float*, long long, int, const float*, float*, long long, const int*,
+                           const int*, const int*, int, int, int, int, int, int, float, float, float, float*, float*, void*);
+        static Fn f = kernel_symbol<Fn>("recurrent", "kipp_gated_delta_scan");
+        float* scratch = recurrent_scratch(tokens, heads, dim, v_dim, 5);
+        float* conv_out = workspace->get<float>("gated_delta_conv", (size_t)tokens * (2 * (size_t)kv_heads * dim + (size_t)heads * v_dim));
+        run(f(out, ld_out, proj, ld_proj, dtype, qkv_off, b_off, conv_w, taps, a_raw, ld_a, dt_bias, a_log, g_raw, ld_g, gate, norm_w,
+              state, slot_stride, q_start, entry_of_token, slots, entries, tokens, heads, kv_heads, dim, v_dim, q_scale, eps, out_scale,
+              scratch, conv_out, stream),
+            "gated_delta_scan", taps > 1 ? 5 : 4);
     }
 
     // Routing by scores (moe.cu): softmax over all `outputs` (sigmoid: of each), the choice by score + correction,

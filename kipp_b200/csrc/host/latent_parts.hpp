@@ -6,7 +6,11 @@
 //                      rest, rotated, is one key part shared by all heads.  Per head the plain
 //                      key is W_uk c and the value W_uv c; score = (q_plain . k_plain + q_rot .
 //                      k_rot) * scale.  Options: a sink per head in the softmax's denominator, a
-//                      sigmoid gate per head from a projection of the mixer's input, a window.
+//                      sigmoid gate per head from a projection of the mixer's input (gate), or one
+//                      per element of the concatenated heads (element_gate), a window, a rotation
+//                      that pairs neighbouring dims (interleaved), and a mixer without a latent of
+//                      its own that reads what another run cached (shared_kv: the run order gives it
+//                      that run's cache id and writes_cache false; it has no W_dkv).
 //
 // Only c and the rotated key part are cached: one key row of kv_rank + rot_dim elements per token,
 // no value pages.  The products with W_uk and W_uv are moved to the query's side of the sums:
@@ -35,18 +39,24 @@ public:
         window_ = (int)j.get_int("window", 0);
         sink_on_ = j.get_bool("sink", false);
         gate_ = gate_code(j.get_string("gate", "none"));
+        element_gate_ = j.get_bool("element_gate", false);
+        interleaved_ = j.get_bool("interleaved", false);
+        shared_kv_ = j.get_bool("shared_kv", false);
         position_ = make_position(j.get("position"), ctx);
         names_ = tensor_names(j, {{"dq", "dq"}, {"dq_norm", "dq.norm"}, {"uq", "uq"}, {"dkv", "dkv"}, {"dkv_norm", "dkv.norm"},
                                   {"uk", "uk"}, {"uv", "uv"}, {"sink", "sink"}, {"g", "g"}, {"o", "o"}});
         if (hidden_ <= 0 || heads_ <= 0 || dim_ <= 0 || rot_ < 0 || v_dim_ <= 0 || kv_rank_ <= 0 || q_rank_ <= 0 || window_ < 0)
             fail(KIPP_E_CONFIG, "latent_attention: sizes must be positive");
         if (gate_ == 1) fail(KIPP_E_CONFIG, "latent_attention: the gate is none or sigmoid");
+        if (gate_ && element_gate_) fail(KIPP_E_CONFIG, "latent_attention: gate and element_gate exclude each other");
         if (position_->rotary_dim() != rot_ || rot_ % 2)
             fail(KIPP_E_CONFIG, "latent_attention: the position encoding must rotate all rot_dim dims (an even number)");
         qh_ = dim_ + rot_;
         row_ = kv_rank_ + rot_;
-        g_off_ = q_rank_ + kv_rank_ + rot_;
-        cols1_ = g_off_ + (gate_ ? heads_ : 0);
+        kv_cols_ = shared_kv_ ? 0 : row_;
+        g_off_ = q_rank_ + kv_cols_;
+        g_cols_ = element_gate_ ? heads_ * v_dim_ : gate_ ? heads_ : 0;
+        cols1_ = g_off_ + g_cols_;
         ld1_ = pad8(cols1_);
         q_rank_ld_ = pad8(q_rank_);
         ldq_ = pad8(heads_ * qh_);
@@ -63,12 +73,14 @@ public:
         add("dq", {q_rank_, hidden_});
         add("dq_norm", {q_rank_}, "near_one");
         add("uq", {heads_ * qh_, q_rank_});
-        add("dkv", {row_, hidden_});
-        add("dkv_norm", {kv_rank_}, "near_one");
+        if (!shared_kv_) {
+            add("dkv", {row_, hidden_});
+            add("dkv_norm", {kv_rank_}, "near_one");
+        }
         add("uk", {heads_ * dim_, kv_rank_});
         add("uv", {heads_ * v_dim_, kv_rank_});
         if (sink_on_) add("sink", {heads_});
-        if (gate_) add("g", {heads_, hidden_});
+        if (g_cols_) add("g", {g_cols_, hidden_});
         add("o", {hidden_, heads_ * v_dim_});
         position_->tensor_specs(p, out);
     }
@@ -84,8 +96,8 @@ public:
         w_in_ = b.allocate((size_t)cols1_ * hidden_ * es, p + "dq_dkv_g");
         char* base = static_cast<char*>(w_in_);
         b.load(p + names_.at("dq"), base, dtype_, hidden_, q_rank_, hidden_);
-        b.load(p + names_.at("dkv"), base + (size_t)q_rank_ * hidden_ * es, dtype_, hidden_, row_, hidden_);
-        if (gate_) b.load(p + names_.at("g"), base + (size_t)g_off_ * hidden_ * es, dtype_, hidden_, heads_, hidden_);
+        if (kv_cols_) b.load(p + names_.at("dkv"), base + (size_t)q_rank_ * hidden_ * es, dtype_, hidden_, row_, hidden_);
+        if (g_cols_) b.load(p + names_.at("g"), base + (size_t)g_off_ * hidden_ * es, dtype_, hidden_, g_cols_, hidden_);
         // rows of W_uq padded to a multiple of 8 elements (zeros beyond the latent's size)
         w_uq_ = b.allocate((size_t)heads_ * qh_ * q_rank_ld_ * es, p + names_.at("uq"));
         cuda_check(cudaMemset(w_uq_, 0, (size_t)heads_ * qh_ * q_rank_ld_ * es), "clearing a padded weight");
@@ -102,7 +114,7 @@ public:
         cuda_check(cudaMemset(w_o_, 0, (size_t)hidden_ * ldo_ * es), "clearing a padded weight");
         b.load(p + names_.at("o"), w_o_, dtype_, ldo_, hidden_, (int64_t)heads_ * v_dim_);
         dq_norm_ = load_f32(b, p + names_.at("dq_norm"), q_rank_);
-        dkv_norm_ = load_f32(b, p + names_.at("dkv_norm"), kv_rank_);
+        if (!shared_kv_) dkv_norm_ = load_f32(b, p + names_.at("dkv_norm"), kv_rank_);
         if (sink_on_) sink_ = load_f32(b, p + names_.at("sink"), heads_);
         position_->bind(b, p);
     }
@@ -111,12 +123,15 @@ public:
                 (size_t)hidden_ * heads_ * v_dim_) * dtype_size(dtype_) + (size_t)(q_rank_ + kv_rank_ + heads_) * 4;
     }
     bool folds_rms() const override { return Ops::gemm_scale_ok(dtype_, w_in_, hidden_, w_in_, hidden_); }
+    bool stores_output() const override { return true; }
     void forward(StepContext& ctx, const LayerRun& run, int mixer_slot, const void* h, float* residual) override {
         const int T = ctx.tokens();
         const size_t es = ctx.element();
         Ops& ops = *ctx.ops;
         const StepMeta& m = *ctx.meta;
-        NormFold fold_in, fold_out;
+        NormFold fold_in;
+        if (shared_kv_ == run.writes_cache)
+            fail(KIPP_E_CONFIG, "latent_attention: a mixer with shared_kv runs with writes_cache false, any other with true");
         const PagedCacheView cache = ctx.cache_view(run, mixer_slot);
         const float* cos_sin = step_rope_table(ctx, *position_, false);
         const int write = (run.writes_cache ? 1 : 0) | (ctx.kv_round_bf16 && ctx.dtype == F32 ? 2 : 0);
@@ -133,8 +148,9 @@ public:
         seg[1].norm_w = dkv_norm_; seg[1].target = 1; seg[1].dst_off = 0;
         seg[2].src_off = q_rank_ + kv_rank_; seg[2].heads = 1; seg[2].dim = rot_; seg[2].src_stride = rot_;
         seg[2].rot = rot_; seg[2].cos_sin = cos_sin; seg[2].target = 1; seg[2].dst_off = kv_rank_;
-        ops.head_segments(proj, ld1_, ctx.dtype, seg, rot_ > 0 ? 3 : 2, &cache, row_, 0, 1, m.positions, m.entry_of_token, T,
-                          write, eps_);
+        seg[2].interleaved = interleaved_ ? 1 : 0;
+        ops.head_segments(proj, ld1_, ctx.dtype, seg, shared_kv_ ? 1 : rot_ > 0 ? 3 : 2, &cache, row_, 0, 1, m.positions,
+                          m.entry_of_token, T, write, eps_);
         // -- the queries: up projection, the plain part through W_uk^T, the rotated part turned
         void* q = ctx.workspace->buffer("latent_q_up", (size_t)T * ldq_ * es);
         ops.gemm(q, ctx.dtype, ldq_, cq, q_rank_ld_, w_uq_, q_rank_ld_, dtype_, T, heads_ * qh_, q_rank_ld_, EPI_STORE);
@@ -144,6 +160,7 @@ public:
         if (rot_ > 0) {
             HeadSegment r;
             r.src_off = dim_; r.heads = heads_; r.dim = rot_; r.src_stride = qh_; r.rot = rot_; r.cos_sin = cos_sin;
+            r.interleaved = interleaved_ ? 1 : 0;
             r.target = 0; r.dst = ql; r.ld_dst = (long long)heads_ * row_; r.dst_off = kv_rank_; r.dst_stride = row_;
             ops.head_segments(q, ldq_, ctx.dtype, &r, 1, nullptr, 0, 0, 0, m.positions, m.entry_of_token, T, 0, eps_);
         }
@@ -155,20 +172,19 @@ public:
         void* lat = ctx.workspace->buffer("latent_out", (size_t)T * heads_ * kv_rank_ * es);
         ops.attention_mix(lat, ql, cache, ctx.dtype, nullptr, m.positions, m.entry_of_token, T, heads_, 1, row_, kv_rank_,
                           scale_, window_, 0, out_scale_, nullptr, 0, m.q_start, m.context_len, &extras);
-        // -- W_uv per head, then the output projection
+        // -- W_uv per head (with the gate per element), then the output projection
         void* attn = ctx.workspace->buffer("attn_out", (size_t)T * ldo_ * es);
         if (ldo_ != heads_ * v_dim_) cuda_check(cudaMemsetAsync(attn, 0, (size_t)T * ldo_ * es, ctx.stream), "clearing the padding");
         ops.head_matmul(attn, ldo_, v_dim_, lat, (long long)heads_ * kv_rank_, kv_rank_, w_uv_, (long long)v_dim_ * kv_rank_,
-                        ctx.dtype, T, v_dim_, kv_rank_, heads_);
-        const NormFold* emit = fold_emit(ctx, fold_out, hidden_);
-        ops.gemm(residual, F32, hidden_, attn, ldo_, w_o_, ldo_, dtype_, T, hidden_, ldo_, EPI_ADD, emit);
-        fold_emitted(ctx, emit, hidden_);
+                        ctx.dtype, T, v_dim_, kv_rank_, heads_,
+                        element_gate_ ? static_cast<const char*>(proj) + (size_t)g_off_ * es : nullptr, ld1_);
+        output_product(ctx, residual, attn, ldo_, w_o_, ldo_, dtype_, hidden_, ldo_);
     }
 
 private:
     int hidden_ = 0, heads_ = 0, dim_ = 0, rot_ = 0, v_dim_ = 0, kv_rank_ = 0, q_rank_ = 0, window_ = 0;
-    int qh_ = 0, row_ = 0, g_off_ = 0, cols1_ = 0, ld1_ = 0, q_rank_ld_ = 0, ldq_ = 0, ldo_ = 0, gate_ = 0, dtype_ = BF16;
-    bool sink_on_ = false;
+    int qh_ = 0, row_ = 0, kv_cols_ = 0, g_cols_ = 0, g_off_ = 0, cols1_ = 0, ld1_ = 0, q_rank_ld_ = 0, ldq_ = 0, ldo_ = 0, gate_ = 0, dtype_ = BF16;
+    bool sink_on_ = false, element_gate_ = false, interleaved_ = false, shared_kv_ = false;
     float eps_ = 0.f, scale_ = 1.f, out_scale_ = 1.f;
     std::unique_ptr<PositionEncoding> position_;
     std::map<std::string, std::string> names_;

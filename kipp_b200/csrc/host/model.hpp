@@ -160,6 +160,9 @@ struct StepContext {
     // with a kernel over the whole stream may form the next block's input in that pass and say so here.
     const Block* following_block = nullptr;
     const Block* input_ready_for = nullptr;
+    // The part's residual is a buffer of its own that holds nothing yet: its output product stores instead of
+    // adding (set around the calls of parts that say stores_output(); any other part never sees it set).
+    bool store_output = false;
 
     size_t element() const { return dtype_size(dtype); }
     int tokens() const { return meta->shape.tokens; }
@@ -230,6 +233,8 @@ public:
     // true: the part applies ctx.input_scale to its first product, at every size of step, and may
     // honour ctx.emit_for in its residual add
     virtual bool folds_rms() const { return false; }
+    // true: the part honours ctx.store_output
+    virtual bool stores_output() const { return false; }
     // the mixers this one is made of, each with a cache or state of its own (mixer slot = index);
     // a plain mixer is its own only part
     virtual std::vector<Mixer*> parts() { return {this}; }
@@ -368,7 +373,7 @@ private:
 };
 
 void register_builtin_parts();           // parts.hpp, recurrent_parts.hpp, latent_parts.hpp, expert_parts.hpp
-void register_builtin_architectures();   // qwen3.hpp, venizen.hpp, varunex.hpp, zasudra.hpp, zunilorn.hpp, panolorn.hpp
+void register_builtin_architectures();   // qwen3.hpp, venizen.hpp, varunex.hpp, zasudra.hpp, zunilorn.hpp, panolorn.hpp, nogavik.hpp
 
 inline void ensure_registered() {
     static std::once_flag once;

@@ -123,20 +123,54 @@ private:
     void* weight_ = nullptr;
 };
 
-// y = x * rsqrt(mean(x^2) + eps) * w, computed in float32 (src/kipp.c:2221-2231).
+// A second table [vocab, cols] that layers read by token, each its own columns (token_side): the stage only
+// declares it.
+class TokenSideTable : public EmbeddingStage {
+public:
+    TokenSideTable(int vocab, int cols, std::string weight_name) : vocab_(vocab), cols_(cols), name_(std::move(weight_name)) {
+        if (vocab <= 0 || cols <= 0) fail(KIPP_E_CONFIG, "token_side_table: sizes must be positive");
+    }
+    void tensor_specs(const std::string& prefix, std::vector<TensorSpec>& out) const override {
+        TensorSpec s;
+        s.name = prefix + name_;
+        s.shape = {vocab_, cols_};
+        out.push_back(s);
+    }
+    void bind(Binder& b, const std::string& prefix) override { b.shared(prefix + name_, b.compute_dtype(), vocab_, cols_); }
+    void forward(StepContext&, float*) override {}
+
+private:
+    int vocab_, cols_;
+    std::string name_;
+};
+
+// y = x * rsqrt(mean(x^2) + eps) * (offset + w), computed in float32 (src/kipp.c:2221-2231).  offset 0 is the plain
+// weight; with offset 1 the checkpoint stores the weight's distance from one.
 class RMSNorm : public Norm {
 public:
-    RMSNorm(int size, double eps, std::string weight_name) : size_(size), eps_((float)eps), name_(std::move(weight_name)) {
+    RMSNorm(int size, double eps, std::string weight_name, double offset = 0.0)
+        : size_(size), eps_((float)eps), name_(std::move(weight_name)), offset_((float)offset) {
         if (size <= 0 || !(eps > 0)) fail(KIPP_E_CONFIG, "rmsnorm: size and eps must be positive");
     }
     void tensor_specs(const std::string& prefix, std::vector<TensorSpec>& out) const override {
         TensorSpec s;
         s.name = prefix + name_;
         s.shape = {size_};
-        s.init = "near_one";
+        s.init = offset_ != 0.f ? "normal" : "near_one";
         out.push_back(s);
     }
     void bind(Binder& b, const std::string& prefix) override {
+        if (offset_ != 0.f) {                     // the sum is formed once, in float32
+            wdtype_ = F32;
+            weight_ = b.allocate((size_t)size_ * sizeof(float), prefix + name_);
+            b.load(prefix + name_, weight_, F32, size_, 1, size_);
+            std::vector<float> w((size_t)size_);
+            cuda_check(cudaDeviceSynchronize(), "reading a norm's weight");
+            cuda_check(cudaMemcpy(w.data(), weight_, w.size() * sizeof(float), cudaMemcpyDeviceToHost), "reading a norm's weight");
+            for (auto& v : w) v += offset_;
+            cuda_check(cudaMemcpy(weight_, w.data(), w.size() * sizeof(float), cudaMemcpyHostToDevice), "upload of a norm's weight");
+            return;
+        }
         // the scale keeps its storage type (bfloat16 or float32)
         wdtype_ = storage_dtype(b.stored_dtype(prefix + name_));
         weight_ = b.allocate((size_t)size_ * dtype_size(wdtype_), prefix + name_);
@@ -153,9 +187,18 @@ private:
     int size_;
     float eps_;
     std::string name_;
+    float offset_ = 0.f;
     int wdtype_ = F32;
     void* weight_ = nullptr;
 };
+
+// A norm in a pass over the residual stream (Ops::Join): of an output that joins it, or of the new stream.
+inline void join_output(Ops::Join& j, int b, const float* y, const RmsNormSpec& n) {
+    j.y[b] = y; j.w_y[b] = n.weight; j.w_y_dtype[b] = n.weight_dtype; j.eps_y[b] = n.eps;
+}
+inline void join_norm(Ops::Join& j, int q, void* h, const RmsNormSpec& n) {
+    j.h[q] = h; j.w_h[q] = n.weight; j.w_h_dtype[q] = n.weight_dtype; j.eps_h[q] = n.eps;
+}
 
 // y = (x - mean) / sqrt(var + eps) * w + b with var the mean of the squared deviations, computed in
 // float32; weight and bias are kept in float32.  `bias_name` empty: no bias.
@@ -497,6 +540,20 @@ inline void fold_emitted(StepContext& ctx, const NormFold* f, int hidden) {
     ctx.emitted_scale = RowScale{f->ssq_out, hidden / 32, 1.0f / (float)hidden, ctx.emit_for->eps};
 }
 
+// A mixer's last product: added to the residual, leaving the next norm's deferred form where asked to, or
+// stored into a buffer that holds nothing yet (StepContext::store_output).
+inline void output_product(StepContext& ctx, float* residual, const void* a, long long lda, const void* w, long long ldw, int dtype,
+                           int hidden, int K) {
+    if (ctx.store_output) {
+        ctx.ops->gemm(residual, F32, hidden, a, lda, w, ldw, dtype, ctx.tokens(), hidden, K, EPI_STORE);
+        return;
+    }
+    NormFold out;
+    const NormFold* emit = fold_emit(ctx, out, hidden);
+    ctx.ops->gemm(residual, F32, hidden, a, lda, w, ldw, dtype, ctx.tokens(), hidden, K, EPI_ADD, emit);
+    fold_emitted(ctx, emit, hidden);
+}
+
 // The step's (cos, sin) table of a position encoding: made once per forward pass and shared by
 // every part that rotates alike (by token, or laid out by pair for the projection that rotates
 // its own heads).
@@ -541,7 +598,7 @@ inline std::map<std::string, std::string> tensor_names(const Json& j, std::map<s
 // [heads, heads]); a factor on the mixer's output (output_scale).  With any of them the step runs
 // on the attention_mix kernel, which holds all heads of a query together.
 //
-// Further options of that path: biases of the q, k and v projections (bias); several score maps
+// Further options of that path: biases of the q, k and v projections (bias; before the q/k norm); several score maps
 // per head (score_maps: q has heads x maps x head_dim rows, k kv_heads x maps x head_dim, laid out
 // head by head as [map 1, map 2, ...]; every map is rotated like a head and is an attention of its
 // own over the head's values); and, with two maps, their combination into one head
@@ -618,10 +675,12 @@ public:
                           opt_.values_are_keys || opt_.shared_kv || opt_.unit_norm || !opt_.distance_slopes.empty() ||
                           opt_.element_gate;
         segments_ = opt_.bias || maps_ > 1 || more;
-        if ((opt_.bias || maps_ > 1) && qk_norm_) fail(KIPP_E_CONFIG, "attention: q/k norm with biases or score maps is not supported");
-        if (more && (opt_.bias || maps_ > 1 || opt_.head_mix))
+        if (maps_ > 1 && qk_norm_) fail(KIPP_E_CONFIG, "attention: q/k norm with score maps is not supported");
+        if (more && (maps_ > 1 || opt_.head_mix))
             fail(KIPP_E_CONFIG, "attention: norm_whole, interleaved, chunk, sink, head_gate, values_are_keys, shared_kv, unit_norm, "
-                                "distance_slopes and element_gate do not go with biases, score maps or head_mix");
+                                "distance_slopes and element_gate do not go with score maps or head_mix");
+        if (opt_.bias && (opt_.shared_kv || opt_.values_are_keys))
+            fail(KIPP_E_CONFIG, "attention: biases need k and v projections of the mixer's own");
         if (opt_.unit_norm && !qk_norm_) fail(KIPP_E_CONFIG, "attention: unit_norm needs qk_norm_eps");
         if (opt_.element_gate && opt_.head_gate) fail(KIPP_E_CONFIG, "attention: head_gate and element_gate exclude each other");
         if (!opt_.distance_slopes.empty() && (int)opt_.distance_slopes.size() != heads)
@@ -641,7 +700,7 @@ public:
         v_cols_ = opt_.shared_kv || opt_.values_are_keys ? 0 : vv_dim_;
         g_cols_ = opt_.element_gate ? o_dim_ : opt_.head_gate ? heads : 0;
         proj_cols_ = q_dim_ + k_cols_ + v_cols_ + g_cols_;
-        proj_ld_ = more ? (proj_cols_ + 7) / 8 * 8 : proj_cols_;
+        proj_ld_ = more || opt_.bias ? (proj_cols_ + 7) / 8 * 8 : proj_cols_;
         if (opt_.softcap < 0) fail(KIPP_E_CONFIG, "attention: softcap must not be negative");
         mix_path_ = opt_.head_mix || (window_ > 0 && opt_.keep_first > 0) || v_dim_ != head_dim_ ||
                     opt_.output_scale != 1.0 || segments_ || opt_.softcap > 0;
@@ -776,6 +835,7 @@ public:
         return n;
     }
     bool folds_rms() const override { return Ops::gemm_scale_ok(dtype_, w_qkv_, hidden_, w_qkv_, hidden_); }
+    bool stores_output() const override { return true; }
     void forward(StepContext& ctx, const LayerRun& run, int mixer_slot, const void* h, float* residual) override;
 
 private:
@@ -1016,51 +1076,172 @@ private:
     float *b_in_ = nullptr, *b_down_ = nullptr, *w_row_ = nullptr;
 };
 
-// x += mixer(n) + ffn(n) with n = norm(x): ONE norm whose output both sublayers read.  A block
-// without a feed-forward (ffn null) has the mixer only.
+// What a layer's own embedding of the token adds to the stream: e = the columns [offset, offset + dim) of the
+// token's row of a table all layers share (token_side_table), g = gelu_tanh(W_gate x) * e, y = W_proj g,
+// x += rmsnorm(y).  x is the stream as it is, not normed.  The pass that adds y may also leave the norms of the
+// new stream that the next block starts with.
+class TokenSide : public Part {
+public:
+    explicit TokenSide(const Json& j) {
+        hidden_ = (int)j.get("hidden_size").as_int();
+        vocab_ = (int)j.get("vocab_size").as_int();
+        dim_ = (int)j.get("dim").as_int();
+        cols_ = (int)j.get("table_cols").as_int();
+        offset_ = (int)j.get_int("offset", 0);
+        table_name_ = j.get("table").as_string();
+        names_ = tensor_names(j, {{"gate", "gate"}, {"proj", "proj"}, {"norm", "norm"}});
+        if (hidden_ <= 0 || vocab_ <= 0 || dim_ <= 0) fail(KIPP_E_CONFIG, "token_side: sizes must be positive");
+        if (offset_ < 0 || offset_ + dim_ > cols_) fail(KIPP_E_CONFIG, "token_side: offset and dim must lie inside the table's row");
+        dim_ld_ = (dim_ + 7) / 8 * 8;
+        norm_ = std::make_unique<RMSNorm>(hidden_, j.get("eps").as_double(), names_.at("norm"));
+    }
+    void tensor_specs(const std::string& p, std::vector<TensorSpec>& out) const override {
+        auto add = [&](const char* role, std::vector<int64_t> shape) {
+            TensorSpec s;
+            s.name = p + names_.at(role);
+            s.shape = std::move(shape);
+            out.push_back(s);
+        };
+        add("gate", {dim_, hidden_});
+        add("proj", {hidden_, dim_});
+        norm_->tensor_specs(p, out);
+    }
+    void bind(Binder& b, const std::string& p) override {
+        dtype_ = b.compute_dtype();
+        const size_t es = dtype_size(dtype_);
+        table_ = b.shared(table_name_, dtype_, vocab_, cols_);
+        w_gate_ = b.allocate((size_t)dim_ * hidden_ * es, p + names_.at("gate"));
+        b.load(p + names_.at("gate"), w_gate_, dtype_, hidden_, dim_, hidden_);
+        // rows of W_proj padded to a multiple of 8 elements (zeros beyond the embedding's size)
+        w_proj_ = b.allocate((size_t)hidden_ * dim_ld_ * es, p + names_.at("proj"));
+        cuda_check(cudaMemset(w_proj_, 0, (size_t)hidden_ * dim_ld_ * es), "clearing a padded weight");
+        b.load(p + names_.at("proj"), w_proj_, dtype_, dim_ld_, hidden_, dim_);
+        norm_->bind(b, p);
+    }
+    size_t weight_bytes() const override { return (size_t)2 * dim_ * hidden_ * dtype_size(dtype_) + norm_->weight_bytes(); }
+    // `next`: the norms of the new stream to leave (Join::h), or none
+    void forward(StepContext& ctx, float* x, const Ops::Join& next) {
+        const int T = ctx.tokens();
+        const size_t es = ctx.element();
+        Ops& ops = *ctx.ops;
+        const void* xin = x;
+        if (ctx.dtype != F32) {
+            void* xc = ctx.workspace->buffer("side_input", (size_t)T * hidden_ * es);
+            ops.convert_rows(xc, ctx.dtype, hidden_, x, F32, hidden_, T, hidden_);
+            xin = xc;
+        }
+        float* z = ctx.workspace->get<float>("side_gate_raw", (size_t)T * dim_ld_);
+        ops.gemm(z, F32, dim_ld_, xin, hidden_, w_gate_, hidden_, dtype_, T, dim_, hidden_, EPI_STORE);
+        void* g = ctx.workspace->buffer("side_gate", (size_t)T * dim_ld_ * es);
+        ops.token_side_gate(g, dim_ld_, z, dim_ld_, table_, cols_, offset_, ctx.dtype, ctx.meta->token_ids, T, dim_, vocab_);
+        float* y = ctx.workspace->get<float>("side_output", (size_t)T * hidden_);
+        ops.gemm(y, F32, hidden_, g, dim_ld_, w_proj_, dim_ld_, dtype_, T, hidden_, dim_ld_, EPI_STORE);
+        Ops::Join j = next;
+        j.x = x;
+        j.size = hidden_;
+        join_output(j, 0, y, *norm_->rms_spec());
+        ops.stream_join(j, ctx.dtype, T);
+    }
+    int hidden() const { return hidden_; }
+
+private:
+    int hidden_ = 0, vocab_ = 0, dim_ = 0, dim_ld_ = 0, cols_ = 0, offset_ = 0, dtype_ = BF16;
+    std::string table_name_;
+    std::map<std::string, std::string> names_;
+    std::unique_ptr<RMSNorm> norm_;
+    void *table_ = nullptr, *w_gate_ = nullptr, *w_proj_ = nullptr;
+};
+
+// x += mixer(n) + ffn(n') with n = norm(x) and n' = n (ONE norm whose output both sublayers read) or, with a
+// norm of the feed-forward's own (ffn_norm), n' = ffn_norm(x), both of the same x.  A block without a
+// feed-forward (ffn null) has the mixer only.  Then, with `side`, what the layer's token embedding adds
+// (token_side).  Blocks with ffn_norm or side make their norms in passes over the stream that also add what
+// joins it, across blocks of this kind; their norms must be RMS norms.
 class ParallelBlock : public Block {
 public:
     ParallelBlock(std::unique_ptr<Norm> norm, std::unique_ptr<Mixer> mixer, std::unique_ptr<FeedForward> ffn,
-                  std::vector<std::string> names)
-        : norm_(std::move(norm)), mixer_(std::move(mixer)), ffn_(std::move(ffn)), names_(std::move(names)) {
-        if (names_.size() != 3) fail(KIPP_E_CONFIG, "parallel_block: three name prefixes are needed");
+                  std::vector<std::string> names, std::unique_ptr<Norm> ffn_norm = nullptr, std::unique_ptr<TokenSide> side = nullptr)
+        : norm_(std::move(norm)), mixer_(std::move(mixer)), ffn_(std::move(ffn)), ffn_norm_(std::move(ffn_norm)), side_(std::move(side)),
+          names_(std::move(names)) {
+        if (names_.size() != (ffn_norm_ || side_ ? 5u : 3u))
+            fail(KIPP_E_CONFIG, "parallel_block: three name prefixes are needed (five with a second norm or a token side)");
+        if (ffn_norm_ && !ffn_) fail(KIPP_E_CONFIG, "parallel_block: ffn_norm needs a feed-forward");
+        if ((ffn_norm_ && ffn_norm_->size() != norm_->size()) || (side_ && side_->hidden() != norm_->size()))
+            fail(KIPP_E_CONFIG, "parallel_block: the norms and the token side differ in size");
     }
     void tensor_specs(const std::string& p, std::vector<TensorSpec>& out) const override {
-        norm_->tensor_specs(p + names_[0], out);
-        mixer_->tensor_specs(p + names_[1], out);
-        if (ffn_) ffn_->tensor_specs(p + names_[2], out);
+        each([&](const Part& part, const std::string& name) { part.tensor_specs(p + name, out); });
     }
     void bind(Binder& b, const std::string& p) override {
-        norm_->bind(b, p + names_[0]);
-        mixer_->bind(b, p + names_[1]);
-        if (ffn_) ffn_->bind(b, p + names_[2]);
+        each([&](Part& part, const std::string& name) { part.bind(b, p + name); });
+        if (joins() && (!norm_->rms_spec() || (ffn_norm_ && !ffn_norm_->rms_spec())))
+            fail(KIPP_E_CONFIG, "parallel_block: with a second norm or a token side the norms must be RMS norms");
     }
     size_t weight_bytes() const override {
-        return norm_->weight_bytes() + mixer_->weight_bytes() + (ffn_ ? ffn_->weight_bytes() : 0);
+        size_t n = 0;
+        each([&](const Part& part, const std::string&) { n += part.weight_bytes(); });
+        return n;
     }
-    bool graph_safe() const override { return norm_->graph_safe() && mixer_->graph_safe() && (!ffn_ || ffn_->graph_safe()); }
+    bool graph_safe() const override {
+        bool ok = true;
+        each([&](const Part& part, const std::string&) { ok = ok && part.graph_safe(); });
+        return ok;
+    }
     std::vector<Mixer*> mixers() override { return mixer_->parts(); }
     void forward(StepContext& ctx, const LayerRun& run, float* x) override {
-        const int T = ctx.tokens();
-        // both sublayers read h, and both add to x: h must outlive the mixer, so no part may leave
-        // another norm's input in its place (emit_for stays null)
-        void* h = ctx.workspace->buffer("normed", (size_t)T * norm_->size() * ctx.element());
+        const int T = ctx.tokens(), W = norm_->size();
+        // both sublayers read what is made here, and both add to x: it must outlive the mixer, so no
+        // part may leave another norm's input in its place (emit_for stays null)
+        void* h = ctx.workspace->buffer("normed", (size_t)T * W * ctx.element());
+        void* h2 = ffn_norm_ ? ctx.workspace->buffer("normed_ffn", (size_t)T * W * ctx.element()) : h;
         ctx.input_scale = RowScale{};
         ctx.pending_norm = nullptr;
         ctx.emit_for = nullptr;
         ctx.emitted = false;
-        norm_->forward(ctx, x, h, nullptr, T);
+        const bool ready = ctx.input_ready_for == this;
+        ctx.input_ready_for = nullptr;
+        if (!joins()) {
+            norm_->forward(ctx, x, h, nullptr, T);
+        } else if (!ready) {
+            Ops::Join j;
+            j.x = x;
+            j.size = W;
+            first_norms(j, h, h2);
+            ctx.ops->stream_join(j, ctx.dtype, T);
+        }
         mixer_->forward(ctx, run, 0, h, x);
-        if (ffn_) ffn_->forward(ctx, h, x);
+        if (ffn_) ffn_->forward(ctx, h2, x);
         ctx.emitted = false;
+        if (!side_) return;
+        const ParallelBlock* next = dynamic_cast<const ParallelBlock*>(ctx.following_block);
+        if (next != nullptr && (!next->joins() || next->norm_->size() != W)) next = nullptr;
+        Ops::Join j;
+        if (next != nullptr)
+            next->first_norms(j, h, next->ffn_norm_ ? ctx.workspace->buffer("normed_ffn", (size_t)T * W * ctx.element()) : h);
+        side_->forward(ctx, x, j);
+        ctx.input_ready_for = next;
     }
     Norm* norm() { return norm_.get(); }
+    Norm* ffn_norm() { return ffn_norm_.get(); }
     FeedForward* feed_forward() { return ffn_.get(); }
 
 private:
+    bool joins() const { return ffn_norm_ != nullptr || side_ != nullptr; }
+    void first_norms(Ops::Join& j, void* h, void* h2) const {
+        join_norm(j, 0, h, *norm_->rms_spec());
+        if (ffn_norm_) join_norm(j, 1, h2, *ffn_norm_->rms_spec());
+    }
+    // every part with its name prefix, in the order of names_
+    template <typename F> void each(F&& f) const {
+        Part* parts[5] = {norm_.get(), mixer_.get(), ffn_.get(), ffn_norm_.get(), side_.get()};
+        for (size_t i = 0; i < 5; ++i)
+            if (parts[i] != nullptr) f(*parts[i], names_[i]);
+    }
     std::unique_ptr<Norm> norm_;
     std::unique_ptr<Mixer> mixer_;
     std::unique_ptr<FeedForward> ffn_;
+    std::unique_ptr<Norm> ffn_norm_;
+    std::unique_ptr<TokenSide> side_;
     std::vector<std::string> names_;
 };
 
@@ -1674,9 +1855,16 @@ inline void register_builtin_parts() {
                                                      j.get("buckets").as_int(), j.get("mul_prev").as_int(),
                                                      j.get("mul_cur").as_int(), j.get_string("weight_name", "weight"));
     });
+    r.add_part_kind("token_side_table", [](const Json& j, const BuildContext&) -> std::unique_ptr<Part> {
+        return std::make_unique<TokenSideTable>((int)j.get("vocab_size").as_int(), (int)j.get("cols").as_int(),
+                                                j.get_string("weight_name", "weight"));
+    });
+    r.add_part_kind("token_side", [](const Json& j, const BuildContext&) -> std::unique_ptr<Part> {
+        return std::make_unique<TokenSide>(j);
+    });
     r.add_part_kind("rmsnorm", [](const Json& j, const BuildContext&) -> std::unique_ptr<Part> {
         return std::make_unique<RMSNorm>((int)j.get("size").as_int(), j.get("eps").as_double(),
-                                         j.get_string("weight_name", "weight"));
+                                         j.get_string("weight_name", "weight"), j.get_double("weight_offset", 0.0));
     });
     r.add_part_kind("layernorm", [](const Json& j, const BuildContext&) -> std::unique_ptr<Part> {
         return std::make_unique<LayerNorm>((int)j.get("size").as_int(), j.get("eps").as_double(),
@@ -1730,11 +1918,16 @@ inline void register_builtin_parts() {
         const Registry& reg = Registry::get();
         std::vector<std::string> names;
         for (auto& n : j.get("names").items()) names.push_back(n.as_string());
-        const Json* ff = j.find("ffn");
+        auto given = [&](const char* key) -> const Json* {
+            const Json* p = j.find(key);
+            return p && !p->is_null() ? p : nullptr;
+        };
+        const Json *ff = given("ffn"), *n2 = given("ffn_norm"), *side = given("side");
         return std::make_unique<ParallelBlock>(reg.make_as<Norm>(j.get("norm"), ctx, "a norm"),
                                                reg.make_as<Mixer>(j.get("mixer"), ctx, "a mixer"),
-                                               ff && !ff->is_null() ? reg.make_as<FeedForward>(*ff, ctx, "a feed-forward") : nullptr,
-                                               names);
+                                               ff ? reg.make_as<FeedForward>(*ff, ctx, "a feed-forward") : nullptr, names,
+                                               n2 ? reg.make_as<Norm>(*n2, ctx, "a norm") : nullptr,
+                                               side ? reg.make_as<TokenSide>(*side, ctx, "a token side") : nullptr);
     });
     r.add_part_kind("rotary", [](const Json& j, const BuildContext&) -> std::unique_ptr<Part> {
         const int head_dim = (int)j.get("head_dim").as_int();

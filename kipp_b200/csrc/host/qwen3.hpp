@@ -231,6 +231,7 @@ void register_varunex();                 // varunex.hpp
 void register_zasudra();                 // zasudra.hpp
 void register_zunilorn();                // zunilorn.hpp
 void register_panolorn();                // panolorn.hpp
+void register_nogavik();                 // nogavik.hpp
 
 inline void register_builtin_architectures() {
     Registry::get().add_architecture("Qwen3ForCausalLM", Architecture{qwen3::normalize, qwen3::plan});
@@ -239,6 +240,7 @@ inline void register_builtin_architectures() {
     register_zasudra();
     register_zunilorn();
     register_panolorn();
+    register_nogavik();
 }
 
 }  // namespace kipp

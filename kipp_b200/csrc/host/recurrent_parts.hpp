@@ -7,7 +7,10 @@
 //                 token, held stable by a running maximum, with a normalizer vector beside the matrix
 //   wkv           time mixing with a decay per head, key channel and token and a bonus for the current
 //                 token; every projection reads its own mix of the token's input and the one before
-//   parallel      the sum of several mixers that read the same input
+//   state_space   the selective state space layer in its matrix-state form, with a short convolution
+//   gated_delta   the delta rule with a decay per head, key channel and token and a write rate per head,
+//                 with short convolutions on queries, keys and values
+//   parallel      the sum of several mixers that read the same input, or of their normed outputs
 //   polynorm_mlp  W_down act(W_up h), act = c0 N(z) + c1 N(z^2) + c2 N(z^3) + c3
 //
 // Every constant (sizes, decays, scales, gates, eps) and every tensor name is a parameter of the
@@ -367,7 +370,9 @@ private:
 // ---------------------------------------------------------------------------------------------
 // Several mixers side by side: each reads the same input and adds its (scaled) output to the
 // residual stream; each has its own cache or state (mixer slot = its index).  The scale of a
-// branch is that mixer's own output_scale.
+// branch is that mixer's own output_scale.  With `out_norm` ({size, eps, offset}) every branch has an RMS
+// norm over its output (weight `norm` of the branch) and the stream gets out_scale times the sum of
+// the normed outputs, in one pass.
 class ParallelMixer : public Mixer {
 public:
     ParallelMixer(const Json& j, const BuildContext& ctx) {
@@ -375,18 +380,30 @@ public:
             prefixes_.push_back(b.get_string("prefix", ""));
             branches_.push_back(Registry::get().make_as<Mixer>(b.get("part"), ctx, "a mixer"));
         }
+        out_scale_ = (float)j.get_double("out_scale", 1.0);
+        if (const Json* n = j.find("out_norm"); n && !n->is_null()) {
+            size_ = (int)n->get("size").as_int();
+            for (auto& b : j.get("branches").items())
+                out_norms_.push_back(std::make_unique<RMSNorm>(size_, n->get("eps").as_double(), b.get("norm").as_string(),
+                                                               n->get_double("offset", 0.0)));
+        } else if (out_scale_ != 1.f) {
+            fail(KIPP_E_CONFIG, "parallel: out_scale goes with out_norm (a branch has an output_scale of its own)");
+        }
         if (branches_.empty()) fail(KIPP_E_CONFIG, "parallel: at least one branch is needed");
         if (branches_.size() > 16) fail(KIPP_E_CONFIG, "parallel: at most 16 branches");
     }
     void tensor_specs(const std::string& p, std::vector<TensorSpec>& out) const override {
         for (size_t i = 0; i < branches_.size(); ++i) branches_[i]->tensor_specs(p + prefixes_[i], out);
+        for (auto& n : out_norms_) n->tensor_specs(p, out);
     }
     void bind(Binder& b, const std::string& p) override {
         for (size_t i = 0; i < branches_.size(); ++i) branches_[i]->bind(b, p + prefixes_[i]);
+        for (auto& n : out_norms_) n->bind(b, p);
     }
     size_t weight_bytes() const override {
         size_t n = 0;
         for (auto& m : branches_) n += m->weight_bytes();
+        for (auto& m : out_norms_) n += m->weight_bytes();
         return n;
     }
     bool graph_safe() const override {
@@ -408,6 +425,10 @@ public:
         // only the last residual add may leave the next norm's deferred form: the stream is
         // complete only then
         const RmsNormSpec* emit_for = ctx.emit_for;
+        if (!out_norms_.empty()) {
+            normed_outputs(ctx, run, mixer_slot, h, residual);
+            return;
+        }
         for (size_t i = 0; i < branches_.size(); ++i) {
             ctx.emit_for = i + 1 == branches_.size() ? emit_for : nullptr;
             branches_[i]->forward(ctx, run, mixer_slot + (int)i, h, residual);
@@ -415,8 +436,33 @@ public:
     }
 
 private:
+    // every branch's output in a buffer of its own, then the pass that norms and adds them (two at a time)
+    void normed_outputs(StepContext& ctx, const LayerRun& run, int mixer_slot, const void* h, float* residual) {
+        const size_t n = (size_t)ctx.tokens() * size_;
+        ctx.emit_for = nullptr;
+        std::vector<float*> y;
+        for (size_t i = 0; i < branches_.size(); ++i) {
+            y.push_back(ctx.workspace->get<float>("branch_output_" + std::to_string(i), n));
+            const bool stores = branches_[i]->stores_output();
+            if (!stores) cuda_check(cudaMemsetAsync(y[i], 0, n * sizeof(float), ctx.stream), "clearing a branch's output");
+            ctx.store_output = stores;
+            branches_[i]->forward(ctx, run, mixer_slot + (int)i, h, y[i]);
+            ctx.store_output = false;
+        }
+        for (size_t i = 0; i < branches_.size(); i += 2) {
+            Ops::Join j;
+            j.x = residual;
+            j.size = size_;
+            j.mult = out_scale_;
+            for (size_t b = i; b < std::min(i + 2, branches_.size()); ++b) join_output(j, (int)(b - i), y[b], *out_norms_[b]->rms_spec());
+            ctx.ops->stream_join(j, ctx.dtype, ctx.tokens());
+        }
+    }
     std::vector<std::string> prefixes_;
     std::vector<std::unique_ptr<Mixer>> branches_;
+    std::vector<std::unique_ptr<RMSNorm>> out_norms_;
+    int size_ = 0;
+    float out_scale_ = 1.f;
 };
 
 // ---------------------------------------------------------------------------------------------
@@ -697,12 +743,13 @@ public:
                ((size_t)channels_ * (taps_ + 1) + 3 * (size_t)heads_ + inner_) * 4;
     }
     bool folds_rms() const override { return Ops::gemm_scale_ok(dtype_, w_in_, hidden_, w_in_, hidden_); }
+    bool stores_output() const override { return true; }
     void forward(StepContext& ctx, const LayerRun& run, int mixer_slot, const void* h, float* residual) override {
         const int T = ctx.tokens();
         const size_t es = ctx.element();
         Ops& ops = *ctx.ops;
         const StepMeta& m = *ctx.meta;
-        NormFold fold_in, fold_out;
+        NormFold fold_in;
         float* state = static_cast<float*>(ctx.state_view(run, mixer_slot, nullptr));
         void* proj = ctx.workspace->buffer("state_space_proj", (size_t)T * proj_ld_ * es);
         ops.gemm(proj, ctx.dtype, proj_ld_, h, hidden_, w_in_, hidden_, dtype_, T, proj_cols_, hidden_, EPI_STORE,
@@ -712,9 +759,7 @@ public:
         ops.ssd_scan(gated, inner_ld_, proj, proj_ld_, ctx.dtype, 0, inner_, inner_ + channels_, conv_, conv_b_, taps_, dt_bias_,
                      a_log_, d_, norm_, norm_groups_, state, state_floats(), m.q_start, m.entry_of_token, m.slots,
                      m.shape.entries, T, heads_, groups_, state_, v_dim_, eps_);
-        const NormFold* emit = fold_emit(ctx, fold_out, hidden_);
-        ops.gemm(residual, F32, hidden_, gated, inner_ld_, w_o_, inner_ld_, dtype_, T, hidden_, inner_ld_, EPI_ADD, emit);
-        fold_emitted(ctx, emit, hidden_);
+        output_product(ctx, residual, gated, inner_ld_, w_o_, inner_ld_, dtype_, hidden_, inner_ld_);
     }
 
 private:
@@ -726,7 +771,173 @@ private:
     float *conv_ = nullptr, *conv_b_ = nullptr, *dt_bias_ = nullptr, *a_log_ = nullptr, *d_ = nullptr, *norm_ = nullptr;
 };
 
+// The gated delta rule (recurrent.cu, kind 5).  q, k = W_q h, W_k h [kv_heads, dim] and v = W_v h [heads, v_dim]
+// pass a causal convolution per channel (no bias) and silu; q and k become unit vectors per head,
+// x / sqrt(sum x^2 + 1e-6), and q is multiplied by query_scale (default dim^-1/2); head h uses q/k head
+// h / (heads / kv_heads).  beta = sigmoid(W_b h) per head; the decay per head and key channel is
+// g = exp(-exp(A_log_h) softplus(W_a2 (W_a1 h) + dt_bias)).  Per head S <- diag(g) S, u = beta (v - S^T k),
+// S <- S + k u^T, o = S^T q.  Each head's o divided by its root mean square (eps inside the root), times a
+// weight of v_dim that all heads share, times gate(W_g2 (W_g1 h)), through W_o.  Per request slot: S in
+// float32 and the last taps - 1 inputs of every convolved channel.  Everything behind the projections is float32.
+class GatedDeltaMixer : public Mixer {
+public:
+    GatedDeltaMixer(const Json& j, const BuildContext&) {
+        hidden_ = (int)j.get("hidden_size").as_int();
+        heads_ = (int)j.get("num_heads").as_int();
+        kv_heads_ = (int)j.get_int("num_kv_heads", heads_);
+        dim_ = (int)j.get("head_dim").as_int();
+        v_dim_ = (int)j.get_int("value_dim", dim_);
+        taps_ = (int)j.get("conv").as_int();
+        a_rank_ = (int)j.get_int("decay_rank", 0);    // 0: the widths of the bottlenecks are read from their tensors
+        g_rank_ = (int)j.get_int("gate_rank", 0);
+        eps_ = (float)j.get("eps").as_double();
+        q_scale_ = (float)j.get_double("query_scale", 1.0 / std::sqrt((double)dim_));
+        out_scale_ = (float)j.get_double("output_scale", 1.0);
+        gate_ = gate_code(j.get_string("gate", "sigmoid"));
+        names_ = tensor_names(j, {{"q", "q"}, {"k", "k"}, {"v", "v"}, {"q_conv", "q.conv"}, {"k_conv", "k.conv"}, {"v_conv", "v.conv"},
+                                  {"b", "b"}, {"a_log", "A_log"}, {"a1", "a1"}, {"a2", "a2"}, {"dt_bias", "dt_bias"}, {"g1", "g1"},
+                                  {"g2", "g2"}, {"norm", "norm"}, {"o", "o"}});
+        if (hidden_ <= 0 || heads_ <= 0 || kv_heads_ <= 0 || dim_ <= 0 || v_dim_ <= 0 || taps_ <= 0 || a_rank_ < 0 || g_rank_ < 0)
+            fail(KIPP_E_CONFIG, "gated_delta: sizes must be positive");
+        if (heads_ % kv_heads_) fail(KIPP_E_CONFIG, "gated_delta: num_heads must be a multiple of num_kv_heads");
+        if (gate_ == 0) fail(KIPP_E_CONFIG, "gated_delta: the gate is silu or sigmoid");
+        qk_ = kv_heads_ * dim_;
+        vv_ = heads_ * v_dim_;
+        channels_ = 2 * qk_ + vv_;
+        vv_ld_ = pad8(vv_);
+        set_ranks(a_rank_, g_rank_);
+    }
+    static int pad8(int n) { return (n + 7) / 8 * 8; }
+    // Rows of the fused projection: q, k, v; the two bottlenecks, each from a multiple of 8 on and padded to one (rows of
+    // zeros: a bottleneck's columns are the next product's input as they lie); the write rates.
+    void set_ranks(int a_rank, int g_rank) {
+        a_rank_ = a_rank;
+        g_rank_ = g_rank;
+        a_ld_ = pad8(a_rank);
+        g_ld_ = pad8(g_rank);
+        a_off_ = pad8(channels_);
+        g_off_ = a_off_ + a_ld_;
+        b_off_ = g_off_ + g_ld_;
+        cols_ = b_off_ + heads_;
+        ld_ = pad8(cols_);
+    }
+    void tensor_specs(const std::string& p, std::vector<TensorSpec>& out) const override {
+        auto add = [&](const char* role, std::vector<int64_t> shape, const char* init = "normal") {
+            TensorSpec s;
+            s.name = p + names_.at(role);
+            s.shape = std::move(shape);
+            s.init = init;
+            out.push_back(s);
+        };
+        const int a = a_rank_ > 0 ? a_rank_ : -1, g = g_rank_ > 0 ? g_rank_ : -1;
+        add("q", {qk_, hidden_});
+        add("q_conv", {qk_, taps_});
+        add("k", {qk_, hidden_});
+        add("k_conv", {qk_, taps_});
+        add("v", {vv_, hidden_});
+        add("v_conv", {vv_, taps_});
+        add("b", {heads_, hidden_});
+        add("a_log", {heads_});
+        add("a1", {a, hidden_});
+        add("a2", {heads_ * dim_, a});
+        add("dt_bias", {heads_ * dim_});
+        add("g1", {g, hidden_});
+        add("g2", {vv_, g});
+        add("norm", {v_dim_}, "near_one");
+        add("o", {hidden_, vv_});
+    }
+    long long state_floats() const { return (long long)heads_ * dim_ * v_dim_ + (long long)(taps_ - 1) * channels_; }
+    std::optional<StateSpec> state_spec() const override { return StateSpec{{state_floats()}, F32}; }
+    void bind(Binder& b, const std::string& p) override {
+        dtype_ = b.compute_dtype();
+        const size_t es = dtype_size(dtype_);
+        auto rank = [&](const char* first, const char* second, int given) {
+            if (given > 0) return given;
+            const std::vector<int64_t> s1 = b.stored_shape(p + names_.at(first)), s2 = b.stored_shape(p + names_.at(second));
+            if (s1.size() != 2 || s2.size() != 2 || s1[0] <= 0 || s1[0] != s2[1])
+                fail(KIPP_E_WEIGHTS, "gated_delta: " + p + names_.at(first) + " and " + p + names_.at(second) +
+                                         " do not agree on the width of the bottleneck");
+            return (int)s1[0];
+        };
+        const int a_rank = rank("a1", "a2", a_rank_);
+        set_ranks(a_rank, rank("g1", "g2", g_rank_));
+        w_in_ = b.allocate((size_t)cols_ * hidden_ * es, p + "qkv, a1, g1, b");
+        cuda_check(cudaMemset(w_in_, 0, (size_t)cols_ * hidden_ * es), "clearing a padded weight");
+        auto put = [&](const char* role, int row, int rows) {
+            b.load(p + names_.at(role), static_cast<char*>(w_in_) + (size_t)row * hidden_ * es, dtype_, hidden_, rows, hidden_);
+        };
+        put("q", 0, qk_);
+        put("k", qk_, qk_);
+        put("v", 2 * qk_, vv_);
+        put("a1", a_off_, a_rank_);
+        put("g1", g_off_, g_rank_);
+        put("b", b_off_, heads_);
+        auto padded = [&](const char* role, int rows, int cols, int ld) {
+            void* w = b.allocate((size_t)rows * ld * es, p + names_.at(role));
+            cuda_check(cudaMemset(w, 0, (size_t)rows * ld * es), "clearing a padded weight");
+            b.load(p + names_.at(role), w, dtype_, ld, rows, cols);
+            return w;
+        };
+        w_a2_ = padded("a2", heads_ * dim_, a_rank_, a_ld_);
+        w_g2_ = padded("g2", vv_, g_rank_, g_ld_);
+        w_o_ = padded("o", hidden_, vv_, vv_ld_);
+        conv_ = static_cast<float*>(b.allocate((size_t)channels_ * taps_ * sizeof(float), p + "convolutions"));
+        b.load(p + names_.at("q_conv"), conv_, F32, taps_, qk_, taps_);
+        b.load(p + names_.at("k_conv"), conv_ + (size_t)qk_ * taps_, F32, taps_, qk_, taps_);
+        b.load(p + names_.at("v_conv"), conv_ + (size_t)2 * qk_ * taps_, F32, taps_, vv_, taps_);
+        dt_bias_ = load_f32(b, p + names_.at("dt_bias"), (int64_t)heads_ * dim_);
+        a_log_ = load_f32(b, p + names_.at("a_log"), heads_);
+        norm_ = load_f32(b, p + names_.at("norm"), v_dim_);
+        if (!Ops::gated_delta_ok(dim_, v_dim_))
+            fail(KIPP_E_UNSUPPORTED, format("gated_delta: the scan kernel does not take heads of %d x %d", dim_, v_dim_));
+        if (taps_ > Ops::ssd_max_taps()) fail(KIPP_E_UNSUPPORTED, format("gated_delta: at most %d taps", Ops::ssd_max_taps()));
+        if (Ops::gated_delta_state_floats(heads_, kv_heads_, dim_, v_dim_, taps_) != state_floats())
+            fail(KIPP_E_STATE, "gated_delta: the kernel library lays the slot out otherwise");
+    }
+    size_t weight_bytes() const override {
+        return ((size_t)cols_ * hidden_ + (size_t)heads_ * dim_ * a_rank_ + (size_t)vv_ * g_rank_ + (size_t)hidden_ * vv_) *
+                   dtype_size(dtype_) +
+               ((size_t)channels_ * taps_ + (size_t)heads_ * (dim_ + 1) + v_dim_) * 4;
+    }
+    bool folds_rms() const override { return Ops::gemm_scale_ok(dtype_, w_in_, hidden_, w_in_, hidden_); }
+    bool stores_output() const override { return true; }
+    void forward(StepContext& ctx, const LayerRun& run, int mixer_slot, const void* h, float* residual) override {
+        const int T = ctx.tokens();
+        const size_t es = ctx.element();
+        Ops& ops = *ctx.ops;
+        const StepMeta& m = *ctx.meta;
+        NormFold fold_in;
+        float* state = static_cast<float*>(ctx.state_view(run, mixer_slot, nullptr));
+        void* proj = ctx.workspace->buffer("gated_delta_proj", (size_t)T * ld_ * es);
+        ops.gemm(proj, ctx.dtype, ld_, h, hidden_, w_in_, hidden_, dtype_, T, cols_, hidden_, EPI_STORE, fold_input(ctx, fold_in));
+        // the second products of the bottlenecks stay float32: softplus, exponentials and the gate's sigmoid read them
+        float* a_raw = ctx.workspace->get<float>("gated_delta_decay", (size_t)T * heads_ * dim_);
+        ops.gemm(a_raw, F32, heads_ * dim_, static_cast<const char*>(proj) + (size_t)a_off_ * es, ld_, w_a2_, a_ld_, dtype_, T,
+                 heads_ * dim_, a_ld_, EPI_STORE);
+        float* g_raw = ctx.workspace->get<float>("gated_delta_gate", (size_t)T * vv_);
+        ops.gemm(g_raw, F32, vv_, static_cast<const char*>(proj) + (size_t)g_off_ * es, ld_, w_g2_, g_ld_, dtype_, T, vv_, g_ld_,
+                 EPI_STORE);
+        void* gated = ctx.workspace->buffer("gated_delta_out", (size_t)T * vv_ld_ * es);
+        if (vv_ld_ != vv_) cuda_check(cudaMemsetAsync(gated, 0, (size_t)T * vv_ld_ * es, ctx.stream), "clearing the padding");
+        ops.gated_delta_scan(gated, vv_ld_, proj, ld_, ctx.dtype, 0, b_off_, conv_, taps_, a_raw, heads_ * dim_, dt_bias_, a_log_, g_raw,
+                             vv_, gate_, norm_, state, state_floats(), m.q_start, m.entry_of_token, m.slots, m.shape.entries, T, heads_,
+                             kv_heads_, dim_, v_dim_, q_scale_, eps_, out_scale_);
+        output_product(ctx, residual, gated, vv_ld_, w_o_, vv_ld_, dtype_, hidden_, vv_ld_);
+    }
+
+private:
+    int hidden_ = 0, heads_ = 0, kv_heads_ = 0, dim_ = 0, v_dim_ = 0, taps_ = 1, a_rank_ = 0, g_rank_ = 0, a_ld_ = 0, g_ld_ = 0,
+        qk_ = 0, vv_ = 0, vv_ld_ = 0, channels_ = 0, a_off_ = 0, g_off_ = 0, b_off_ = 0, cols_ = 0, ld_ = 0, gate_ = 2, dtype_ = BF16;
+    float eps_ = 0.f, q_scale_ = 1.f, out_scale_ = 1.f;
+    std::map<std::string, std::string> names_;
+    void *w_in_ = nullptr, *w_a2_ = nullptr, *w_g2_ = nullptr, *w_o_ = nullptr;
+    float *conv_ = nullptr, *dt_bias_ = nullptr, *a_log_ = nullptr, *norm_ = nullptr;
+};
+
 inline void register_recurrent_parts(Registry& r) {
+    r.add_part_kind("gated_delta", [](const Json& j, const BuildContext& ctx) -> std::unique_ptr<Part> {
+        return std::make_unique<GatedDeltaMixer>(j, ctx);
+    });
     r.add_part_kind("state_space", [](const Json& j, const BuildContext& ctx) -> std::unique_ptr<Part> {
         return std::make_unique<StateSpaceMixer>(j, ctx);
     });

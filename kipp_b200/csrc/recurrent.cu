@@ -15,6 +15,11 @@
 //                    pass a short causal convolution and silu first; dt = softplus(dt_raw + bias); the
 //                    heads of a group share B and C; then the gate silu(z), a root-mean-square division
 //                    in equal parts of the row, a weight)
+//   gated delta     S <- diag(g_t) S_{t-1}, u_t = beta_t (v_t - S^T k_t), S_t = S + k_t u_t^T, o_t = S_t^T q_t
+//                    (the delta rule with a decay per head, key channel and token, g = exp(-exp(A_h)
+//                    softplus(a_raw + bias)), and a write rate per head and token; q, k and v pass a short
+//                    causal convolution and silu first, q and k are unit vectors; the heads of a group share
+//                    q and k; the weight after the root-mean-square division is shared by all heads)
 //
 // S is [key dim, value dim].  Retention rotates q and k by the step's (cos, sin)
 // table (pair (i, i + rot/2), the first `rot` dims) and scales k afterwards; its
@@ -86,12 +91,17 @@ struct ScanArgs {
     const float* conv_w; const float* conv_b;
     const float* dt_bias; const float* a_log; const float* d_skip;
     const int* entry_of_token;
+    // the convolved channels and where a slot keeps their last inputs (floats behind its start)
+    int channels; long long kept_off;
+    // gated delta rule: a_raw and g_raw float32, [T, heads * dim] and [T, heads * v_dim]
+    const float* a_raw; long long ld_a; const float* g_raw; long long ld_g; int b_off;
 };
-enum { RETENTION = 0, DELTA_RULE = 1, GATED_MEMORY = 2, WKV = 3, SSD = 4 };
+enum { RETENTION = 0, DELTA_RULE = 1, GATED_MEMORY = 2, WKV = 3, SSD = 4, GATED_DELTA = 5 };
 // vectors per token besides v, extra floats after them, extra value columns
 template <int KIND> struct Rec {
-    static constexpr int NV = KIND == DELTA_RULE ? 5 : KIND == WKV ? 3 : 2;     // wkv: r, k, w
-    static constexpr int XG = KIND == GATED_MEMORY || KIND == WKV || KIND == SSD ? 4 : 0;   // (i, f, 0, 0), wkv's (sum u k r, 0, 0, 0) or the state space's (decay, dt, 0, 0), after the vectors
+    static constexpr int NV = KIND == DELTA_RULE ? 5 : KIND == WKV || KIND == GATED_DELTA ? 3 : 2;     // wkv: r, k, w; gated delta: q, k, g
+    // after the vectors: (i, f, 0, 0), wkv's (sum u k r, 0, 0, 0), the state space's (decay, dt, 0, 0) or the gated delta rule's (beta, q . k, 0, 0)
+    static constexpr int XG = KIND == GATED_MEMORY || KIND == WKV || KIND == SSD || KIND == GATED_DELTA ? 4 : 0;
     static constexpr int XV = KIND == GATED_MEMORY ? 4 : 0;     // value columns (1, 0, 0, 0) after v
 };
 __device__ __forceinline__ float log_sigmoid(float x) { return fminf(x, 0.f) - log1pf(expf(-fabsf(x))); }
@@ -251,7 +261,7 @@ recurrent_scan_kernel(const ScanArgs a, const float* __restrict__ vec, float* __
     float S[CHUNK];
 #pragma unroll
     for (int i = 0; i < CHUNK; ++i) S[i] = (live && row_of(i) < D) ? S_slot[(size_t)row_of(i) * V + col] : 0.f;
-    const float decay = DELTA || KIND == WKV ? 0.f : a.decay[h];
+    const float decay = KIND == RETENTION ? a.decay[h] : 0.f;
 
     load_batch(smem, smem + TB * nvd, recs, rec, nvd, min(TB, n_tok), slice, V, async, VS * P);
     int buf = 0;
@@ -302,6 +312,55 @@ recurrent_scan_kernel(const ScanArgs a, const float* __restrict__ vec, float* __
                 for (int x = P / 2; x > 0; x >>= 1) us += __shfl_xor_sync(0xffffffffu, us, x);
             }
             float o = 0.f;
+            if (KIND == GATED_DELTA) {
+                // the decayed state meets k and q in one pass and both sums travel together; the token's own
+                // write then joins the output as (q . k) u
+                float kr[CHUNK], us4[4] = {0.f, 0.f, 0.f, 0.f}, os4[4] = {0.f, 0.f, 0.f, 0.f};
+                if (VEC) {
+#pragma unroll
+                    for (int g = 0; g < CHUNK / 4; ++g) {
+                        const int r = 4 * (p + P * g);
+                        if (r < D) {
+                            const float4 q4 = *reinterpret_cast<const float4*>(tok + r);
+                            const float4 k4 = *reinterpret_cast<const float4*>(tok + D + r);
+                            const float4 g4 = *reinterpret_cast<const float4*>(tok + 2 * D + r);
+                            const float qq[4] = {q4.x, q4.y, q4.z, q4.w}, kk[4] = {k4.x, k4.y, k4.z, k4.w}, gg[4] = {g4.x, g4.y, g4.z, g4.w};
+#pragma unroll
+                            for (int j = 0; j < 4; ++j) {
+                                const float s = S[4 * g + j] * gg[j];
+                                S[4 * g + j] = s;
+                                kr[4 * g + j] = kk[j];
+                                us4[j] = fmaf(kk[j], s, us4[j]);
+                                os4[j] = fmaf(qq[j], s, os4[j]);
+                            }
+                        }
+                    }
+                } else {
+#pragma unroll
+                    for (int i = 0; i < CHUNK; ++i)
+                        if (p + P * i < D) {
+                            const float s = S[i] * base[2 * D + P * i];
+                            S[i] = s;
+                            kr[i] = base[D + P * i];
+                            us4[i & 3] = fmaf(kr[i], s, us4[i & 3]);
+                            os4[i & 3] = fmaf(base[P * i], s, os4[i & 3]);
+                        }
+                }
+                us = (us4[0] + us4[1]) + (us4[2] + us4[3]);
+                o = (os4[0] + os4[1]) + (os4[2] + os4[3]);
+#pragma unroll
+                for (int x = P / 2; x > 0; x >>= 1) {
+                    us += __shfl_xor_sync(0xffffffffu, us, x);
+                    o += __shfl_xor_sync(0xffffffffu, o, x);
+                }
+                const float u = tok[NV * D] * (v - us);
+#pragma unroll
+                for (int i = 0; i < CHUNK; ++i)
+                    if (row_of(i) < D) S[i] = fmaf(kr[i], u, S[i]);
+                o = fmaf(tok[NV * D + 1], u, o);
+                if (live && p == 0) o_raw[(size_t)(row0 + t0 + tt) * (a.heads * V) + h * V + col] = o;
+                continue;
+            }
             const float tv = take * v;                  // (gated memory, state space: the input's weight on this column's value)
             if (VEC && KIND == SSD) {
                 // the state space layer's heads are tall (128 rows and more): a group's four rows are a short chain
@@ -399,18 +458,18 @@ recurrent_finish_kernel(const ScanArgs a, const float* __restrict__ o_raw, int t
     for (int c = lane; c < V; c += 32) {
         const int hc = h * V + c;
         float y = o[c] * den * inv;
-        if (a.norm_w != nullptr) y *= a.norm_w[hc];
+        if (a.norm_w != nullptr) y *= a.norm_w[KIND == GATED_DELTA ? c : hc];
         if (a.gate != 0) {
-            const float g = to_f32(proj[row * a.ld_proj + a.g_off + hc]);
+            const float g = KIND == GATED_DELTA ? a.g_raw[row * a.ld_g + hc] : to_f32(proj[row * a.ld_proj + a.g_off + hc]);
             y *= a.gate == 1 ? g * sigmoidf_(g) : sigmoidf_(g);
         }
         out[row * a.ld_out + hc] = from_f32<T>(y * a.out_scale);
     }
 }
 
-// The state space layer's causal convolution: a thread per (token, channel) sums taps inputs (the
-// step's own rows, and before the portion's first token the rows the slot keeps, zeros at a
-// sequence's start), adds the bias and applies silu; the result stays float32, [tokens, channels].
+// The causal convolution of the state space layer and of the gated delta rule: a thread per (token, channel) sums
+// taps inputs (the step's own rows, and before the portion's first token the rows the slot keeps, zeros at a
+// sequence's start), adds the bias (if any) and applies silu; the result stays float32, [tokens, channels].
 constexpr int MAX_TAPS = 16;
 template <typename T>
 __global__ void __launch_bounds__(256)
@@ -418,13 +477,13 @@ ssd_conv_kernel(const ScanArgs a, float* __restrict__ conv_out) {
     pdl_launch_dependents();
     pdl_wait();
     const int row = blockIdx.x, taps = a.taps;
-    const int channels = a.heads * a.v_dim + 2 * a.groups * a.dim;
+    const int channels = a.channels;
     const int c = blockIdx.y * blockDim.x + threadIdx.x;
     if (c >= channels) return;
     const int e = a.entry_of_token[row], first = a.q_start[e];
     const T* proj = static_cast<const T*>(a.proj);
-    const float* kept = a.state + (size_t)a.slots[e] * (size_t)a.slot_stride + (size_t)a.heads * a.dim * a.v_dim;   // [taps - 1][channels]
-    float acc = a.conv_b[c];
+    const float* kept = a.state + (size_t)a.slots[e] * (size_t)a.slot_stride + a.kept_off;      // [taps - 1][channels]
+    float acc = a.conv_b != nullptr ? a.conv_b[c] : 0.f;
     for (int j = 0; j < taps; ++j) {
         const int r = row - (taps - 1 - j);                         // the row that meets tap j
         const float in = r >= first ? to_f32(proj[(size_t)r * a.ld_proj + a.xbc_off + c])
@@ -465,6 +524,52 @@ ssd_prepare_kernel(const ScanArgs a, const float* __restrict__ conv_out, float* 
         dst[2 * D + 1] = dt;
         dst[2 * D + 2] = 0.f;
         dst[2 * D + 3] = 0.f;
+    }
+}
+
+// The gated delta rule's token vectors.  A warp per (token, head) makes the unit vectors of its group's q and k
+// (q also times q_scale), the decay of every key channel and the write rate: the record
+// [q, k, g, (beta, q . k, 0, 0), v].
+template <typename T>
+__global__ void __launch_bounds__(128)
+gated_delta_prepare_kernel(const ScanArgs a, const float* __restrict__ conv_out, float* __restrict__ vec, int tokens) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int lane = threadIdx.x & 31;
+    const long long wg = ((long long)blockIdx.x * blockDim.x + threadIdx.x) >> 5;
+    if (wg >= (long long)tokens * a.heads) return;
+    const int row = (int)(wg / a.heads), h = (int)(wg % a.heads);
+    const int D = a.dim, V = a.v_dim;
+    const int g = h / (a.heads / a.groups);
+    const float* qv = conv_out + (size_t)row * a.channels + g * D;
+    const float* kv = qv + a.groups * D;
+    const float* vv = conv_out + (size_t)row * a.channels + 2 * a.groups * D + h * V;
+    const int rec = 3 * D + 4 + V;
+    float* dst = vec + ((size_t)h * tokens + row) * rec;
+    float qq = 0.f, kk = 0.f, qk = 0.f;
+    for (int d = lane; d < D; d += 32) {
+        const float q = qv[d], k = kv[d];
+        qq = fmaf(q, q, qq);
+        kk = fmaf(k, k, kk);
+        qk = fmaf(q, k, qk);
+    }
+    const float iq = a.q_scale / sqrtf(warp_sum(qq) + 1e-6f), ik = 1.0f / sqrtf(warp_sum(kk) + 1e-6f);
+    qk = warp_sum(qk) * iq * ik;
+    const float rate = expf(a.a_log[h]);
+    const float* ar = a.a_raw + (size_t)row * a.ld_a + h * D;
+    for (int d = lane; d < D; d += 32) {
+        const float raw = ar[d] + a.dt_bias[h * D + d];
+        const float sp = fmaxf(raw, 0.f) + log1pf(expf(-fabsf(raw)));       // softplus, exact at both ends
+        dst[d] = qv[d] * iq;
+        dst[D + d] = kv[d] * ik;
+        dst[2 * D + d] = expf(-rate * sp);
+    }
+    for (int c = lane; c < V; c += 32) dst[3 * D + 4 + c] = vv[c];
+    if (lane == 0) {
+        dst[3 * D] = sigmoidf_(to_f32(static_cast<const T*>(a.proj)[(size_t)row * a.ld_proj + a.b_off + h]));
+        dst[3 * D + 1] = qk;
+        dst[3 * D + 2] = 0.f;
+        dst[3 * D + 3] = 0.f;
     }
 }
 
@@ -522,11 +627,11 @@ ssd_conv_keep_kernel(const ScanArgs a) {
     pdl_launch_dependents();
     pdl_wait();
     const int e = blockIdx.x, first = a.q_start[e], n = a.q_start[e + 1] - first, keep = a.taps - 1;
-    const int channels = a.heads * a.v_dim + 2 * a.groups * a.dim;
+    const int channels = a.channels;
     const int c = blockIdx.y * blockDim.x + threadIdx.x;
     if (n <= 0 || c >= channels) return;
     const T* proj = static_cast<const T*>(a.proj);
-    float* kept = a.state + (size_t)a.slots[e] * (size_t)a.slot_stride + (size_t)a.heads * a.dim * a.v_dim;
+    float* kept = a.state + (size_t)a.slots[e] * (size_t)a.slot_stride + a.kept_off;
     float rows[MAX_TAPS - 1];
 #pragma unroll
     for (int r = 0; r < MAX_TAPS - 1; ++r) {
@@ -541,14 +646,25 @@ ssd_conv_keep_kernel(const ScanArgs a) {
     }
 }
 
+// (P below 8 comes with at most 8 rows per thread, see launch_scan; rows that do not go by fours are rare, so two
+// sizes of the unrolled loop serve them)
 template <typename T, int DELTA, int P, bool VEC>
 int launch_scan_rows(const ScanArgs& b, const float* vec, float* o_raw, int slices, int tokens, dim3 grid, size_t smem,
                      cudaStream_t stream) {
     const int chunk = (b.dim + P - 1) / P;
-    if (chunk <= 8) return kipp_launch(recurrent_scan_kernel<T, DELTA, P, 8, VEC>, grid, dim3(VS * P), smem, stream, 1, b, vec, o_raw, slices, tokens);
-    if (chunk <= 16) return kipp_launch(recurrent_scan_kernel<T, DELTA, P, 16, VEC>, grid, dim3(VS * P), smem, stream, 1, b, vec, o_raw, slices, tokens);
-    if (chunk <= 24) return kipp_launch(recurrent_scan_kernel<T, DELTA, P, 24, VEC>, grid, dim3(VS * P), smem, stream, 1, b, vec, o_raw, slices, tokens);
-    return kipp_launch(recurrent_scan_kernel<T, DELTA, P, 32, VEC>, grid, dim3(VS * P), smem, stream, 1, b, vec, o_raw, slices, tokens);
+#define KIPP_SCAN(C) return kipp_launch(recurrent_scan_kernel<T, DELTA, P, C, VEC>, grid, dim3(VS * P), smem, stream, 1, b, vec, o_raw, slices, tokens)
+    if constexpr (P < 8) {
+        if (chunk > 8) return KIPP_ERR_ARG;
+        KIPP_SCAN(8);
+    } else {
+        if (chunk <= 8) KIPP_SCAN(8);
+        if constexpr (VEC) {
+            if (chunk <= 16) KIPP_SCAN(16);
+            if (chunk <= 24) KIPP_SCAN(24);
+        }
+        KIPP_SCAN(32);
+    }
+#undef KIPP_SCAN
 }
 template <typename T, int DELTA, int P>
 int launch_scan_chunk(const ScanArgs& b, const float* vec, float* o_raw, int slices, int tokens, dim3 grid, size_t smem,
@@ -560,7 +676,7 @@ int launch_scan_chunk(const ScanArgs& b, const float* vec, float* o_raw, int sli
 }
 
 // scratch: float32 [heads][tokens][NV * dim + v_dim] for the records, then [tokens][heads * v_dim] for raw o
-// conv_out: float32 [tokens, channels] for the state space layer's convolved rows (null for the other kinds)
+// conv_out: float32 [tokens, channels] for the convolved rows of the state space layer and the gated delta rule (null for the other kinds)
 template <typename T, int DELTA>
 int launch_scan(const ScanArgs& a, int entries, int tokens, float* scratch, cudaStream_t stream, float* conv_out = nullptr) {
     const int D = a.dim, V = a.v_dim + Rec<DELTA>::XV;
@@ -570,7 +686,7 @@ int launch_scan(const ScanArgs& a, int entries, int tokens, float* scratch, cuda
     int P = 1;
     while (P < 8 && (D + P - 1) / P > 8) P *= 2;
     if ((D + P - 1) / P > MAX_CHUNK) P = 16;
-    if (DELTA == SSD && D > 64 && KIPP_SSD_WIDE) P = 16;
+    if ((DELTA == SSD || DELTA == GATED_DELTA) && D > 64 && KIPP_SSD_WIDE) P = 16;
     if ((D + P - 1) / P > MAX_CHUNK || scratch == nullptr) return KIPP_ERR_ARG;
     const size_t per_token = ((size_t)NV * D + XG + VS) * sizeof(float);
     int batch = (int)std::min<size_t>(32, (20 * 1024) / per_token);       // two buffers of at most 20 KB
@@ -582,13 +698,15 @@ int launch_scan(const ScanArgs& a, int entries, int tokens, float* scratch, cuda
     const long long warps = (long long)tokens * a.heads;
     const dim3 wgrid((unsigned)((warps + 3) / 4));
     int rc = 0;
-    const int channels = DELTA == SSD ? a.heads * a.v_dim + 2 * a.groups * a.dim : 0;
-    if (DELTA == SSD) {
+    constexpr bool CONV = DELTA == SSD || DELTA == GATED_DELTA;
+    const int channels = a.channels;
+    if constexpr (CONV) {
         if (conv_out == nullptr) return KIPP_ERR_ARG;
         rc = kipp_launch(ssd_conv_kernel<T>, dim3((unsigned)tokens, (unsigned)((channels + 255) / 256)), dim3(256), 0, stream, 1, b,
                          conv_out);
         if (rc) return rc;
-        rc = kipp_launch(ssd_prepare_kernel<T>, wgrid, dim3(128), 0, stream, 1, b, (const float*)conv_out, vec, tokens);
+        rc = kipp_launch(DELTA == SSD ? ssd_prepare_kernel<T> : gated_delta_prepare_kernel<T>, wgrid, dim3(128), 0, stream, 1, b,
+                         (const float*)conv_out, vec, tokens);
     } else {
         rc = kipp_launch(recurrent_prepare_kernel<T, DELTA>, wgrid, dim3(128), 0, stream, 1, b, vec, tokens);
     }
@@ -604,17 +722,18 @@ int launch_scan(const ScanArgs& a, int entries, int tokens, float* scratch, cuda
     default: rc = launch_scan_chunk<T, DELTA, 16>(b, vec, o_raw, slices, tokens, grid, smem, stream); break;
     }
     if (rc) return rc;
-    if (DELTA == SSD) {
+    if constexpr (DELTA == SSD) {
         const long long parts = (long long)tokens * b.norm_groups;
         if (parts > 0x7fffffffLL) return KIPP_ERR_ARG;
         const int per_part = a.heads * a.v_dim / b.norm_groups;
         rc = kipp_launch(ssd_finish_kernel<T>, dim3((unsigned)parts), dim3(per_part >= 128 ? 128 : (per_part + 31) / 32 * 32), 0,
                          stream, 1, b, (const float*)conv_out, (const float*)o_raw);
-        if (rc || b.taps <= 1) return rc;
-        return kipp_launch(ssd_conv_keep_kernel<T>, dim3((unsigned)entries, (unsigned)((channels + 255) / 256)), dim3(256), 0,
-                           stream, 1, b);
+    } else {
+        rc = kipp_launch(recurrent_finish_kernel<T, DELTA>, wgrid, dim3(128), 0, stream, 1, b, (const float*)o_raw, tokens);
     }
-    return kipp_launch(recurrent_finish_kernel<T, DELTA>, wgrid, dim3(128), 0, stream, 1, b, (const float*)o_raw, tokens);
+    if (rc || !CONV || b.taps <= 1) return rc;
+    return kipp_launch(ssd_conv_keep_kernel<T>, dim3((unsigned)entries, (unsigned)((channels + 255) / 256)), dim3(256), 0, stream,
+                       1, b);
 }
 
 template <typename T>
@@ -661,13 +780,13 @@ __global__ void tanh_rows_kernel(T* __restrict__ out, long long ld_out, const T*
 
 // Whether the scan kernels take a head of these sizes.
 extern "C" int kipp_recurrent_scan_ok(int dim, int v_dim, int kind) {
-    if (dim <= 0 || v_dim <= 0 || dim > 16 * MAX_CHUNK || kind < 0 || kind > 4) return 0;
-    return (((kind == DELTA_RULE ? 5 : kind == WKV ? 3 : 2) * (size_t)dim + 4 + VS) * sizeof(float)) <= 20 * 1024 ? 1 : 0;
+    if (dim <= 0 || v_dim <= 0 || dim > 16 * MAX_CHUNK || kind < 0 || kind > GATED_DELTA) return 0;
+    return (((kind == DELTA_RULE ? 5 : kind == WKV || kind == GATED_DELTA ? 3 : 2) * (size_t)dim + 4 + VS) * sizeof(float)) <= 20 * 1024 ? 1 : 0;
 }
 // float32 values of scratch a scan of `tokens` tokens needs.
 extern "C" long long kipp_recurrent_scratch_floats(int tokens, int heads, int dim, int v_dim, int kind) {
-    const long long x = kind == GATED_MEMORY ? 4 : 0, g = kind == WKV || kind == SSD ? 4 : 0;
-    return (long long)tokens * heads * ((kind == DELTA_RULE ? 5 : kind == WKV ? 3 : 2) * (long long)dim + x + g + 2 * ((long long)v_dim + x));
+    const long long x = kind == GATED_MEMORY ? 4 : 0, g = kind == WKV || kind == SSD || kind == GATED_DELTA ? 4 : 0;
+    return (long long)tokens * heads * ((kind == DELTA_RULE ? 5 : kind == WKV || kind == GATED_DELTA ? 3 : 2) * (long long)dim + x + g + 2 * ((long long)v_dim + x));
 }
 // float32 values of state one request slot of the gated memory holds: S with n's column and its
 // padding, then one running maximum per head and slice of value columns.
@@ -792,8 +911,46 @@ extern "C" int kipp_ssd_scan(void* out, long long ld_out, const void* proj, long
     a.conv_w = conv_w; a.conv_b = conv_b; a.dt_bias = dt_bias; a.a_log = a_log; a.d_skip = d_skip; a.norm_w = norm_w;
     a.state = state; a.slot_stride = slot_stride; a.q_start = q_start; a.entry_of_token = entry_of_token; a.slots = slots;
     a.heads = heads; a.dim = dim; a.v_dim = v_dim; a.eps = eps; a.k_scale = 1.f; a.out_scale = 1.f;
+    a.channels = heads * v_dim + 2 * groups * dim; a.kept_off = (long long)heads * dim * v_dim;
     if (dtype == KIPP_DT_F32) return launch_scan<float, SSD>(a, entries, tokens, scratch, (cudaStream_t)stream, conv_out);
     if (dtype == KIPP_DT_BF16) return launch_scan<bf16, SSD>(a, entries, tokens, scratch, (cudaStream_t)stream, conv_out);
+    return KIPP_ERR_DTYPE;
+}
+
+// float32 values of state one request slot of the gated delta rule holds: S [heads, dim, v_dim], then the last
+// taps - 1 inputs of the 2 * kv_heads * dim + heads * v_dim convolved channels.
+extern "C" long long kipp_gated_delta_state_floats(int heads, int kv_heads, int dim, int v_dim, int taps) {
+    return (long long)heads * dim * v_dim + (long long)(taps > 1 ? taps - 1 : 0) * (2LL * kv_heads * dim + (long long)heads * v_dim);
+}
+
+// The gated delta rule (see the head of this file).  proj [T, ...] holds the channels to convolve [q: kv_heads * dim |
+// k: kv_heads * dim | v: heads * v_dim] at qkv_off and the write rates' pre-activations [heads] at b_off; conv_w
+// [channels, taps] (the last tap meets the current token); a_raw [T, heads * dim] and g_raw [T, heads * v_dim]
+// float32 are the pre-activations of the decay and of the output's gate (1 silu, 2 sigmoid); dt_bias [heads * dim],
+// a_log [heads], norm_w [v_dim] float32.  A slot is kipp_gated_delta_state_floats floats.  conv_out: float32
+// [tokens, channels] of scratch.  At most 16 taps.
+extern "C" int kipp_gated_delta_scan(void* out, long long ld_out, const void* proj, long long ld_proj, int dtype, int qkv_off,
+                                     int b_off, const float* conv_w, int taps, const float* a_raw, long long ld_a,
+                                     const float* dt_bias, const float* a_log, const float* g_raw, long long ld_g, int gate,
+                                     const float* norm_w, float* state, long long slot_stride, const int* q_start,
+                                     const int* entry_of_token, const int* slots, int entries, int tokens, int heads, int kv_heads,
+                                     int dim, int v_dim, float q_scale, float eps, float out_scale, float* scratch, float* conv_out,
+                                     void* stream) {
+    if (entries <= 0 || tokens <= 0) return 0;
+    if (!kipp_recurrent_scan_ok(dim, v_dim, GATED_DELTA) || heads <= 0 || kv_heads <= 0 || heads % kv_heads || taps < 1 ||
+        taps > MAX_TAPS || conv_w == nullptr || a_raw == nullptr || g_raw == nullptr || dt_bias == nullptr || a_log == nullptr ||
+        norm_w == nullptr || entry_of_token == nullptr || gate < 1 || gate > 2 || ld_a < (long long)heads * dim ||
+        ld_g < (long long)heads * v_dim || slot_stride < kipp_gated_delta_state_floats(heads, kv_heads, dim, v_dim, taps))
+        return KIPP_ERR_ARG;
+    ScanArgs a = {};
+    a.out = out; a.ld_out = ld_out; a.proj = proj; a.ld_proj = ld_proj;
+    a.xbc_off = qkv_off; a.b_off = b_off; a.conv_w = conv_w; a.taps = taps; a.groups = kv_heads;
+    a.a_raw = a_raw; a.ld_a = ld_a; a.dt_bias = dt_bias; a.a_log = a_log; a.g_raw = g_raw; a.ld_g = ld_g; a.gate = gate; a.norm_w = norm_w;
+    a.state = state; a.slot_stride = slot_stride; a.q_start = q_start; a.entry_of_token = entry_of_token; a.slots = slots;
+    a.heads = heads; a.dim = dim; a.v_dim = v_dim; a.q_scale = q_scale; a.eps = eps; a.k_scale = 1.f; a.out_scale = out_scale;
+    a.channels = 2 * kv_heads * dim + heads * v_dim; a.kept_off = (long long)heads * dim * v_dim;
+    if (dtype == KIPP_DT_F32) return launch_scan<float, GATED_DELTA>(a, entries, tokens, scratch, (cudaStream_t)stream, conv_out);
+    if (dtype == KIPP_DT_BF16) return launch_scan<bf16, GATED_DELTA>(a, entries, tokens, scratch, (cudaStream_t)stream, conv_out);
     return KIPP_ERR_DTYPE;
 }
 
