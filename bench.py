@@ -221,6 +221,23 @@ def panolorn_of(size: str, vocab: int = 32000) -> dict:
             "layers": [{"type": "attention", "mixer": att, "mlp": mlps[i % 2]} for i in range(layers)]}
 
 
+def nogavik_of(size: str, vocab: int = 32000) -> dict:
+    """The design's mixers in turn (the state space layer of zunilorn_of; attention over a cached latent, as wide
+    as varunex_of's; attention with values of twice a head's size beside the gated delta rule with square
+    states; a latent attention that reads that layer's latent), each beside a dense feed-forward with the
+    square of relu, an embedding of 128 per layer and token."""
+    width, heads, kv, dim, ff, layers = DESIGN_SIZES[size]
+    mlp = {"kind": "dense", "ff": ff}
+    ssm = {"heads": 2 * width // 64, "groups": 8, "vdim": 64, "state": 128, "conv": 4, "norm_groups": 8}
+    latent = {"heads": heads, "dim": dim, "rot_dim": dim // 2, "vdim": dim, "kv_rank": 4 * dim, "q_rank": width // 2,
+              "rot": {"base": 1e6, "dims": dim // 2}, "scale": (dim + dim // 2) ** -0.5}
+    par = {"left": {"heads": heads // 2, "kv_heads": kv // 2, "dim": dim, "vdim": 2 * dim, "scale": dim ** -0.5},
+           "right": {"heads": heads // 2, "kv_heads": heads // 2, "dim": dim, "vdim": dim, "conv": 4, "decay_rank": dim, "gate_rank": dim}}
+    order = [("mamba2", ssm), ("latent_attention", latent), ("parallel", par), ("latent_attention", dict(latent, kv_from=1))]
+    return {"architecture": "Nogavik", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "token_side": {"dim": 128},
+            "layers": [{"type": t, "mixer": m, "mlp": mlp} for t, m in (order[i % 4] for i in range(layers))]}
+
+
 def qwen3_of(size: str, vocab: int = 32000) -> dict:
     width, heads, kv, dim, ff, layers = DESIGN_SIZES[size]
     return dict(architectures=["Qwen3ForCausalLM"], model_type="qwen3", vocab_size=vocab, hidden_size=width,
@@ -242,7 +259,8 @@ def compare_designs(args) -> int:
     families = {"venizen": [("venizen", venizen_of)], "varunex": [("varunex", varunex_of), ("venizen", venizen_of)],
                 "zasudra": [("zasudra", zasudra_of), ("venizen", venizen_of)],
                 "zunilorn": [("zunilorn", zunilorn_of), ("zasudra", zasudra_of)],
-                "panolorn": [("panolorn", panolorn_of), ("zasudra", zasudra_of)]}
+                "panolorn": [("panolorn", panolorn_of), ("zasudra", zasudra_of)],
+                "nogavik": [("nogavik", nogavik_of), ("zunilorn", zunilorn_of), ("varunex", varunex_of)]}
     designs = families[args.design_family] + [("qwen3", qwen3_of)]
     out = {"metric": "prefill and decode tokens/s, " + " and ".join(d.capitalize() for d, _ in designs[:-1]) +
                      " beside Qwen3 at equal layer sizes", "dtype": "bf16",
@@ -329,9 +347,11 @@ def main() -> int:
                     help="instead of the default workload: a design (--design-family) beside Qwen3 at equal layer sizes, "
                          f"a list of {','.join(DESIGN_SIZES)} (prefill and decode tokens/s, time per kernel)")
     ap.add_argument("--designs-prompt", type=int, default=2048, help="prompt and decode context of --designs")
-    ap.add_argument("--design-family", default="venizen", choices=["venizen", "varunex", "zasudra", "zunilorn", "panolorn"],
+    ap.add_argument("--design-family", default="venizen",
+                    choices=["venizen", "varunex", "zasudra", "zunilorn", "panolorn", "nogavik"],
                     help="the design --designs measures: venizen, or varunex or zasudra (with Venizen, their closest "
-                         "relative, beside it), or zunilorn or panolorn (with Zasudra beside it)")
+                         "relative, beside it), or zunilorn or panolorn (with Zasudra beside it), or nogavik (with Zunilorn and "
+                         "Varunex beside it)")
     args = ap.parse_args()
     if args.impl == "reference":
         return reference_arm(args)

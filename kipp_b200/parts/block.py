@@ -2,6 +2,7 @@
 from __future__ import annotations
 
 from .base import Block, FeedForward, Mixer, Norm
+from .embedding import TokenSide
 
 
 class PreNormBlock(Block):
@@ -25,18 +26,23 @@ class PreNormBlock(Block):
 
 class ParallelBlock(Block):
     """x += mixer(n) + ffn(n) with n = norm(x): ONE norm whose output both
-    sublayers read.  ``ffn`` None: the mixer only.  The part itself:
-    csrc/host/parts.hpp."""
+    sublayers read, or (``ffn_norm``) one each, of the same x.  ``ffn`` None: the
+    mixer only.  ``side``: a ``TokenSide`` behind them.  ``names``: prefixes of norm,
+    mixer and feed-forward and, where given, of ``ffn_norm`` and ``side``.  The part
+    itself: csrc/host/parts.hpp."""
     kind = "parallel_block"
 
-    def __init__(self, norm: Norm, mixer: Mixer, ffn: FeedForward, names: tuple[str, str, str] = ("norm.", "mix.", "mlp.")):
+    def __init__(self, norm: Norm, mixer: Mixer, ffn: FeedForward | None, names: tuple = ("norm.", "mix.", "mlp."), *,
+                 ffn_norm: Norm | None = None, side: TokenSide | None = None):
+        self.parts = (norm, mixer, ffn, ffn_norm, side)
         self.norm, self.mixer, self.ffn = norm, mixer, ffn
-        self.names = tuple(names)
+        self.names = tuple(names) if len(names) == 5 or (ffn_norm is None and side is None) else tuple(names) + ("", "side.")
 
     def params(self, prefix, ctx) -> dict:
-        parts = (self.norm, self.mixer, self.ffn)
-        described = [None if p is None else p.describe(prefix + n, ctx) for p, n in zip(parts, self.names)]
-        return {"names": list(self.names), "norm": described[0], "mixer": described[1], "ffn": described[2]}
+        roles = ("norm", "mixer", "ffn", "ffn_norm", "side")
+        names = self.names + ("",) * (5 - len(self.names))
+        described = {r: None if p is None else p.describe(prefix + n, ctx) for r, p, n in zip(roles, self.parts, names)}
+        return {"names": list(self.names), **described}
 
 
 class SandwichNormBlock(Block):

@@ -24,6 +24,33 @@ class TokenEmbedding(EmbeddingStage):
                 "scale": self.scale}
 
 
+class TokenSideTable(EmbeddingStage):
+    """A second table [vocab, cols] that layers read by token, each its own columns (``TokenSide``)."""
+    kind = "token_side_table"
+
+    def __init__(self, vocab_size: int, cols: int, weight_name: str = "weight"):
+        self.vocab_size, self.cols, self.weight_name = vocab_size, cols, weight_name
+
+    def params(self, prefix, ctx) -> dict:
+        return {"vocab_size": self.vocab_size, "cols": self.cols, "weight_name": self.weight_name}
+
+
+class TokenSide(Part):
+    """What a layer's own embedding e of the token adds to the stream: x += rmsnorm(W_proj (gelu(W_gate x) * e))
+    with e the columns [offset, offset + dim) of the token's row of ``table`` (a ``TokenSideTable`` of
+    ``table_cols`` columns)."""
+    kind = "token_side"
+
+    def __init__(self, vocab_size: int, hidden_size: int, dim: int, table: str, table_cols: int, offset: int, eps: float,
+                 names: Optional[dict] = None):
+        self.vocab_size, self.hidden_size, self.dim, self.table, self.table_cols = vocab_size, hidden_size, dim, table, table_cols
+        self.offset, self.eps, self.names = offset, float(eps), dict(names or {})
+
+    def params(self, prefix, ctx) -> dict:
+        return {"vocab_size": self.vocab_size, "hidden_size": self.hidden_size, "dim": self.dim, "table": self.table,
+                "table_cols": self.table_cols, "offset": self.offset, "eps": self.eps, "names": self.names}
+
+
 class OutputHead(Part):
     """``tied_to`` names the checkpoint tensor (an embedding matrix) that stands
     in when the checkpoint has no head of its own."""

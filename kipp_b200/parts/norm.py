@@ -9,13 +9,15 @@ from .base import Norm
 class RMSNorm(Norm):
     kind = "rmsnorm"
 
-    def __init__(self, size: int, eps: float, weight_name: str = "weight"):
+    def __init__(self, size: int, eps: float, weight_name: str = "weight", weight_offset: float = 0.0):
+        """``weight_offset`` 1: the checkpoint stores the weight's distance from one."""
         self.size = size
         self.eps = float(eps)
         self.weight_name = weight_name
+        self.weight_offset = float(weight_offset)
 
     def params(self, prefix, ctx) -> dict:
-        return {"size": self.size, "eps": self.eps, "weight_name": self.weight_name}
+        return {"size": self.size, "eps": self.eps, "weight_name": self.weight_name, "weight_offset": self.weight_offset}
 
 
 class LayerNorm(Norm):
