@@ -53,7 +53,7 @@
 // A second form of the kernel (X, kipp_attn_prefill_tc_ex) takes what the attention_mix kernels take
 // without a mix of the heads: blocks of positions as the mask, capped scores, a number per head taken
 // off per position of distance, a sink in the denominator, a gate per head or per element, a factor on
-// the output, and heads of any multiple of 8 up to 128 whose values may have a size of their own, up to 256 (a
+// the output, and heads of any multiple of 8 up to 192 whose values may have a size of their own, up to 256 (a
 // tile of 64 columns that a head does not fill is filled with zeros by the TMA unit: the maps end at
 // the head).  The cap is c tanh(x / c) = c - 2 c / (1 + e^(2x / c)), an exponential and a reciprocal per
 // score in float32.  The weights keep float32 precision through the 16-bit product: p = hi + lo with
@@ -287,7 +287,8 @@ struct Params {
     float out_scale;
 };
 
-// D, DV: columns of the query / key tiles (64 or 128) and of the value tile (64, 128, and in the X form 192 or 256)
+// D, DV: columns of the query / key tiles (64, 128, and in the X form 192) and of the value tile (64, 128, and in the X
+// form 192 or 256)
 template <int D, int DV> struct Cfg {
     static constexpr int HALVES = D / 64, V_HALVES = DV / 64;
     static constexpr int Q_BYTES = BM * D * 2;
@@ -296,7 +297,7 @@ template <int D, int DV> struct Cfg {
     static constexpr int TMEM_COLS = DV > 128 ? 512 : 256;      // two score buffers (64 each) + O (DV), power of two
     // a CTA with all of the tensor memory has its SM for itself: its shared memory leaves no room for another,
     // which would only stand waiting for tensor memory
-    static constexpr int CTAS = DV > 128 ? 1 : 2;
+    static constexpr int CTAS = DV > 128 || D > 128 ? 1 : 2;
     // 100,480 bytes at head_dim 128: two CTAs (plus the 1 KB the system keeps per CTA) fit in 227 KB
     static constexpr size_t NEED = Q_BYTES + 2 * K_BYTES + 2 * V_BYTES + XCHG_BYTES + 144;   // 16 barriers, 2 words
     static constexpr size_t SMEM = CTAS == 1 && NEED < 116 * 1024 ? 116 * 1024 : NEED;
@@ -845,7 +846,7 @@ extern "C" int kipp_attn_prefill_tc_page_ok(int page_size) {
 // `extras` (or null) with v_dim and out_scale: the X form (blocks, cap, slopes, sink, gate; see the head of this
 // file).  Of the options of MixExtras it takes neither score maps nor values that lie in their key rows.
 extern "C" int kipp_attn_prefill_tc_ex_supported(int head_dim, int v_dim, int n_q, int n_kv) {
-    return head_dim >= 16 && head_dim <= 128 && head_dim % 8 == 0 && v_dim >= 16 && v_dim <= 256 && v_dim % 8 == 0 && n_kv > 0 &&
+    return head_dim >= 16 && head_dim <= 192 && head_dim % 8 == 0 && v_dim >= 16 && v_dim <= 256 && v_dim % 8 == 0 && n_kv > 0 &&
            n_q % n_kv == 0;
 }
 static int prefill_tc(void* out, const void* q, int tokens, const void* k_pages, const void* v_pages, int n_pages,
@@ -903,6 +904,11 @@ static int prefill_tc(void* out, const void* q, int tokens, const void* k_pages,
     p.slopes = ex->slopes; p.sink = ex->sink;
     p.gate = static_cast<const bf16*>(ex->gate) + (ex->gate != nullptr ? ex->gate_off : 0);
     p.ld_gate = ex->ld_gate; p.gate_dims = ex->gate_dims;
+    if (head_dim > 128)
+        return v_dim <= 64    ? launch<192, 64, true>(mk, mv, mk4, mv4, mq, mo, p, items, s)
+               : v_dim <= 128 ? launch<192, 128, true>(mk, mv, mk4, mv4, mq, mo, p, items, s)
+               : v_dim <= 192 ? launch<192, 192, true>(mk, mv, mk4, mv4, mq, mo, p, items, s)
+                              : launch<192, 256, true>(mk, mv, mk4, mv4, mq, mo, p, items, s);
     if (v_dim > 192)
         return head_dim <= 64 ? launch<64, 256, true>(mk, mv, mk4, mv4, mq, mo, p, items, s)
                               : launch<128, 256, true>(mk, mv, mk4, mv4, mq, mo, p, items, s);

@@ -21,6 +21,9 @@
 // 32-bit, or where rows do not start on 16-byte boundaries, few tokens by a kernel that reads the
 // weights once and more tokens in tiles on the CUDA cores.  (Products with a latent: keys absorbed into queries, values expanded after the
 // weighted sum.)
+//
+// kipp_latent_expand: the keys and values of every head out of cached latents, for prompt kernels that read them as
+// keys and values of heads of their own: see the kernel.
 #include "common.cuh"
 #include <math.h>
 
@@ -358,6 +361,146 @@ head_matmul_mma_kernel(bf16* __restrict__ C, const bf16* __restrict__ A, const b
     }
 }
 
+// The keys and values of every head from the latents a step's entries have cached (bfloat16).  A cached row holds a
+// token's latent c [rank] and a key part [rot] all heads share; head h's key is [W_uk,h c | shared part], its value
+// W_uv,h c.  They go to a pool of their own in pages of 64 tokens, keys [page][head][64][dim + rot] and values
+// [page][head][64][v_dim], where token t of entry e lies in page e * pages_per_entry + t / 64 (that table is written too);
+// rows of a page beyond the entry's last token are zeros.  A block of 8 warps (2 x 4) takes 128 tokens x 128
+// features on mma.sync, K in steps of 32 through three stages of asynchronous copies; the tile leaves through shared
+// memory in 16-byte pieces.  One more block per tile copies the shared key part into every head's keys.
+constexpr int EM = 128, EN = 128, EK = 32, ELD = EK + 8, E_STAGES = 3, E_THREADS = 256, E_PAGE = 64;
+constexpr size_t E_SMEM = (size_t)E_STAGES * (EM + EN) * ELD * 2;
+static_assert(E_SMEM >= (size_t)EM * (EN + 8) * 2, "the result tile fits where the stages were");
+struct ExpandArgs {
+    const bf16* pages;                       // [page][page_size][row] latents
+    const int* block_table; int table_width, page_size, row;
+    const int* q_start; const int* context_len;
+    const bf16* w_k; const bf16* w_v;        // [heads * dim, rank], [heads * v_dim, rank]
+    int rank, dim, rot, v_dim, heads;
+    bf16* k_out; bf16* v_out; int* table_out;
+    int pages_per_entry, k_tiles, v_tiles;
+    int* status;
+};
+__device__ __forceinline__ void ldmatrix4(uint32_t* r, uint32_t addr) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
+                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
+}
+__global__ void __launch_bounds__(E_THREADS)
+latent_expand_kernel(const ExpandArgs a) {
+    extern __shared__ __align__(16) bf16 tile_mem[];
+    pdl_launch_dependents();
+    pdl_wait();
+    const int e = blockIdx.z, t0 = blockIdx.y * EM, tid = threadIdx.x;
+    const int len = a.context_len[e] + a.q_start[e + 1] - a.q_start[e];
+    const int rows_end = (len + E_PAGE - 1) / E_PAGE * E_PAGE;          // rows to write: whole pages
+    const int ft = blockIdx.x;
+    if (ft == a.k_tiles + a.v_tiles && blockIdx.y == 0)
+        for (int j = tid; j < a.pages_per_entry; j += E_THREADS) a.table_out[(size_t)e * a.pages_per_entry + j] = e * a.pages_per_entry + j;
+    if (t0 >= rows_end) return;
+    const int* table = a.block_table + (size_t)e * a.table_width;
+    const int k_row = a.dim + a.rot;
+    // the cached row of token t, or null where the entry has no such token
+    auto cached = [&](int t) -> const bf16* {
+        if (t >= len) return nullptr;
+        const int slot = t / a.page_size, page = slot < a.table_width ? table[slot] : -1;
+        if (page < 0) {
+            atomicExch(a.status, 3);                                    // a needed key is not mapped
+            return nullptr;
+        }
+        return a.pages + ((size_t)page * a.page_size + t % a.page_size) * a.row;
+    };
+    auto out_row = [&](bf16* base, int t, int h, int width) {
+        return base + ((((size_t)e * a.pages_per_entry + t / E_PAGE) * a.heads + h) * E_PAGE + t % E_PAGE) * width;
+    };
+    if (ft == a.k_tiles + a.v_tiles) {                                  // the shared key part
+        const int chunks = a.rot / 8;
+        for (int i = tid; i < EM * chunks; i += E_THREADS) {
+            const int t = t0 + i / chunks, c = i % chunks;
+            if (t >= rows_end) break;
+            const bf16* src = cached(t);
+            const uint4 v = src != nullptr ? *reinterpret_cast<const uint4*>(src + a.rank + c * 8) : make_uint4(0u, 0u, 0u, 0u);
+            for (int h = 0; h < a.heads; ++h) *reinterpret_cast<uint4*>(out_row(a.k_out, t, h, k_row) + a.dim + c * 8) = v;
+        }
+        return;
+    }
+    const bool keys = ft < a.k_tiles;
+    const int per_head = keys ? a.dim : a.v_dim, features = a.heads * per_head, n0 = (keys ? ft : ft - a.k_tiles) * EN;
+    const bf16* w = keys ? a.w_k : a.w_v;
+    // 128 rows x 4 chunks of 8 elements per operand and stage: two of each per thread, rows lr and lr + 64
+    const int lr = tid >> 2, lc = (tid & 3) * 8;
+    const bf16* a_src[2];
+    const bf16* w_src[2];
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+        a_src[i] = cached(t0 + lr + 64 * i);
+        w_src[i] = n0 + lr + 64 * i < features ? w + (size_t)(n0 + lr + 64 * i) * a.rank : nullptr;
+    }
+    auto fetch = [&](int k0, int stage) {
+        bf16* as = tile_mem + (size_t)stage * (EM + EN) * ELD;
+        bf16* ws = as + EM * ELD;
+        const bool in = k0 + lc < a.rank;
+#pragma unroll
+        for (int i = 0; i < 2; ++i) {
+            const bool oa = in && a_src[i] != nullptr, ow = in && w_src[i] != nullptr;
+            cp_async16(smem_address(as + (lr + 64 * i) * ELD + lc), oa ? a_src[i] + k0 + lc : a.pages, oa ? 16 : 0);
+            cp_async16(smem_address(ws + (lr + 64 * i) * ELD + lc), ow ? w_src[i] + k0 + lc : w, ow ? 16 : 0);
+        }
+    };
+    const int lane = tid & 31, warp = tid >> 5, wm = (warp >> 2) * 64, wn = (warp & 3) * 32, gid = lane >> 2, tig = lane & 3;
+    float acc[4][4][4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) acc[i][j][0] = acc[i][j][1] = acc[i][j][2] = acc[i][j][3] = 0.f;
+    const int steps = (a.rank + EK - 1) / EK;
+#pragma unroll
+    for (int s = 0; s < E_STAGES - 1; ++s) {
+        if (s < steps) fetch(s * EK, s);
+        cp_async_commit();
+    }
+    for (int s = 0; s < steps; ++s) {
+        cp_async_wait<E_STAGES - 2>();
+        __syncthreads();
+        if (s + E_STAGES - 1 < steps) fetch((s + E_STAGES - 1) * EK, (s + E_STAGES - 1) % E_STAGES);
+        cp_async_commit();
+        const bf16* as = tile_mem + (size_t)(s % E_STAGES) * (EM + EN) * ELD;
+        const bf16* ws = as + EM * ELD;
+#pragma unroll
+        for (int ks = 0; ks < EK; ks += 16) {
+            uint32_t af[4][4], bf[2][4];
+#pragma unroll
+            for (int i = 0; i < 4; ++i) ldmatrix4(af[i], smem_address(as + (wm + i * 16 + (lane & 15)) * ELD + ks + (lane >> 4) * 8));
+            // two groups of 8 features per load: rows (lane & 7) + 8 (lane >> 4), k half by bit 3 of the lane
+#pragma unroll
+            for (int j = 0; j < 2; ++j)
+                ldmatrix4(bf[j], smem_address(ws + (wn + j * 16 + (lane & 7) + (lane >> 4) * 8) * ELD + ks + ((lane >> 3) & 1) * 8));
+#pragma unroll
+            for (int i = 0; i < 4; ++i)
+#pragma unroll
+                for (int j = 0; j < 4; ++j) mma_bf16_16816(acc[i][j], af[i], bf[j >> 1][2 * (j & 1)], bf[j >> 1][2 * (j & 1) + 1]);
+        }
+    }
+    cp_async_wait<0>();
+    __syncthreads();
+    constexpr int CLD = EN + 8;
+    bf16* ct = tile_mem;
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j)
+#pragma unroll
+            for (int half = 0; half < 2; ++half)
+                *reinterpret_cast<__nv_bfloat162*>(ct + (wm + i * 16 + gid + 8 * half) * CLD + wn + j * 8 + tig * 2) =
+                    __floats2bfloat162_rn(acc[i][j][2 * half], acc[i][j][2 * half + 1]);
+    __syncthreads();
+    for (int i = tid; i < EM * (EN / 8); i += E_THREADS) {
+        const int r = i / (EN / 8), n = n0 + i % (EN / 8) * 8, t = t0 + r;
+        if (t >= rows_end || n >= features) continue;                   // (heads are multiples of 8: a piece lies in one head)
+        bf16* dst = keys ? out_row(a.k_out, t, n / per_head, k_row) : out_row(a.v_out, t, n / per_head, a.v_dim);
+        *reinterpret_cast<uint4*>(dst + n % per_head) = *reinterpret_cast<const uint4*>(ct + r * CLD + i % (EN / 8) * 8);
+    }
+}
+
 // out[h][n][k] = in[h][k][n]: the matrices of every head transposed (at bind time).
 template <typename T>
 __global__ void transpose_heads_kernel(T* __restrict__ out, const T* __restrict__ in, int rows, int cols) {
@@ -460,6 +603,42 @@ extern "C" int kipp_head_matmul(void* C, const void* A, const void* W, int dtype
                                 long long lda, long long a_head, long long w_head, long long ldc, long long c_head,
                                 void* stream) {
     return kipp_head_matmul_gated(C, A, W, dtype, M, N, K, heads, lda, a_head, w_head, ldc, c_head, nullptr, 0, stream);
+}
+
+// Whether kipp_latent_expand takes these sizes: every row and head goes by 16-byte pieces.
+extern "C" int kipp_latent_expand_ok(int rank, int dim, int rot, int v_dim, int heads) {
+    return rank > 0 && dim > 0 && rot >= 0 && v_dim > 0 && heads > 0 && rank % 8 == 0 && dim % 8 == 0 && rot % 8 == 0 && v_dim % 8 == 0;
+}
+extern "C" int kipp_latent_expand_page() { return E_PAGE; }
+
+// See latent_expand_kernel.  pages_per_entry pages of kipp_latent_expand_page() tokens hold the longest context the
+// block table can name.
+extern "C" int kipp_latent_expand(const void* pages, const int* block_table, int table_width, int page_size, int row,
+                                  const int* q_start, const int* context_len, int entries, const void* w_k, const void* w_v,
+                                  int rank, int dim, int rot, int v_dim, int heads, void* k_out, void* v_out, int* table_out,
+                                  int pages_per_entry, int* status, void* stream) {
+    if (entries <= 0) return 0;
+    if (!kipp_latent_expand_ok(rank, dim, rot, v_dim, heads) || row != rank + rot || page_size <= 0 || table_width <= 0 ||
+        (long long)pages_per_entry * E_PAGE < (long long)table_width * page_size || entries > 65535)
+        return KIPP_ERR_ARG;
+    if ((((uintptr_t)pages | (uintptr_t)w_k | (uintptr_t)w_v | (uintptr_t)k_out | (uintptr_t)v_out) & 15) != 0) return -3;
+    ExpandArgs a = {};
+    a.pages = (const bf16*)pages; a.block_table = block_table; a.table_width = table_width; a.page_size = page_size; a.row = row;
+    a.q_start = q_start; a.context_len = context_len; a.w_k = (const bf16*)w_k; a.w_v = (const bf16*)w_v;
+    a.rank = rank; a.dim = dim; a.rot = rot; a.v_dim = v_dim; a.heads = heads;
+    a.k_out = (bf16*)k_out; a.v_out = (bf16*)v_out; a.table_out = table_out; a.pages_per_entry = pages_per_entry; a.status = status;
+    a.k_tiles = (heads * dim + EN - 1) / EN;
+    a.v_tiles = (heads * v_dim + EN - 1) / EN;
+    static bool configured = false;
+    if (!configured) {
+        const cudaError_t e = cudaFuncSetAttribute(latent_expand_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)E_SMEM);
+        if (e != cudaSuccess) { cudaGetLastError(); return (int)e; }
+        configured = true;
+    }
+    const int tiles = (pages_per_entry * E_PAGE + EM - 1) / EM;
+    if (tiles > 65535) return KIPP_ERR_ARG;
+    return kipp_launch(latent_expand_kernel, dim3((unsigned)(a.k_tiles + a.v_tiles + 1), (unsigned)tiles, (unsigned)entries),
+                       dim3(E_THREADS), E_SMEM, (cudaStream_t)stream, 1, a);
 }
 
 // out[h] = in[h]^T for `heads` row-major matrices of [rows, cols] in `dtype`.

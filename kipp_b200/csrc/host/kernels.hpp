@@ -328,14 +328,8 @@ public:
         if (dtype == BF16 && mix_tensor_core && prefill_tensor_core && separate && tokens > MIX_MMA_MIN_TOKENS && wide_tiles != nullptr &&
             n_wide_tiles > 0 && tokens >= WIDE_TILE_MIN_ROWS * n_wide_tiles && aligned &&
             attention_tc_ex_supported(*extras, head_dim, v_dim, n_q, n_kv, cache.page_size)) {
-            using Ft = int (*)(void*, const void*, int, const void*, const void*, int, const int*, const int*, const int*, int, int,
-                               const int*, int, int, int, int, int, float, int, float, const void*, int*, void*);
-            static Ft tc = kernel_symbol<Ft>("attention_tc", "kipp_attn_prefill_tc_ex");
-            run(tc(out, q, tokens, cache.k_pages, cache.v_pages, cache.n_pages, q_start, context_len, cache.block_table,
-                   cache.table_width, cache.page_size, wide_tiles, n_wide_tiles, n_q, n_kv, head_dim, v_dim, scale, window, out_scale,
-                   extras, status, stream),
-                "attn_prefill_tc");
-            ++mix_tc_launches;
+            attention_prompt_tc(out, q, cache, tokens, n_q, n_kv, head_dim, v_dim, scale, window, out_scale, q_start, context_len, *extras,
+                                wide_tiles, n_wide_tiles);
             return;
         }
         // (single tokens of many requests are the group kernel's below)
@@ -388,6 +382,66 @@ public:
               cache.table_width, cache.page_size, tokens, n_q, n_kv, head_dim, v_dim, scale, window, keep_first,
               out_scale, runs, partial, extras, status, stream),
             "attention_mix", runs > 1 ? 2 : 1);
+    }
+
+    // The tcgen05 prompt kernel with the options of `extras` (attention_tc_ex_supported): a block per head and 128 tokens.
+    void attention_prompt_tc(void* out, const void* q, const PagedCacheView& cache, int tokens, int n_q, int n_kv, int head_dim,
+                             int v_dim, float scale, int window, float out_scale, const int* q_start, const int* context_len,
+                             const AttentionExtras& extras, const int* wide_tiles, int n_wide_tiles) {
+        using Ft = int (*)(void*, const void*, int, const void*, const void*, int, const int*, const int*, const int*, int, int,
+                           const int*, int, int, int, int, int, float, int, float, const void*, int*, void*);
+        static Ft tc = kernel_symbol<Ft>("attention_tc", "kipp_attn_prefill_tc_ex");
+        run(tc(out, q, tokens, cache.k_pages, cache.v_pages, cache.n_pages, q_start, context_len, cache.block_table,
+               cache.table_width, cache.page_size, wide_tiles, n_wide_tiles, n_q, n_kv, head_dim, v_dim, scale, window, out_scale,
+               &extras, status, stream),
+            "attn_prefill_tc");
+        ++mix_tc_launches;
+    }
+
+    // The keys and values of every head out of the latents the step's entries have cached, in pages of their own
+    // (head_ops.cu): the view of those pages, or none where the kernels do not take the sizes or the pages would pass
+    // EXPAND_MAX_BYTES.  Which it is depends on the step's shape only.
+    static constexpr long long EXPAND_MAX_BYTES = 1LL << 30;
+    static bool latent_expand_ok(int dtype, int rank, int dim, int rot, int v_dim, int heads) {
+        using Fn = int (*)(int, int, int, int, int);
+        static Fn f = kernel_symbol<Fn>("head_ops", "kipp_latent_expand_ok");
+        return dtype == BF16 && f(rank, dim, rot, v_dim, heads) != 0;
+    }
+    bool latent_prompt_ok(const AttentionExtras& extras, const PagedCacheView& cache, int tokens, int entries, int n_wide_tiles,
+                          int rank, int dim, int rot, int v_dim, int heads) {
+        if (!mix_tensor_core || !prefill_tensor_core || tokens <= MIX_MMA_MIN_TOKENS || n_wide_tiles <= 0 ||
+            tokens < WIDE_TILE_MIN_ROWS * n_wide_tiles)
+            return false;
+        const long long per = expand_pages(cache), bytes = (long long)entries * per * expand_page() * heads * (dim + rot + v_dim) * 2;
+        return bytes <= EXPAND_MAX_BYTES && attention_tc_ex_supported(extras, dim + rot, v_dim, heads, heads, expand_page());
+    }
+    static int expand_page() {
+        using Fn = int (*)();
+        static Fn f = kernel_symbol<Fn>("head_ops", "kipp_latent_expand_page");
+        return f();
+    }
+    static int expand_pages(const PagedCacheView& cache) {
+        return (int)(((long long)cache.table_width * cache.page_size + expand_page() - 1) / expand_page());
+    }
+    PagedCacheView latent_expand(const PagedCacheView& cache, const int* q_start, const int* context_len, int entries, const void* w_k,
+                                 const void* w_v, int rank, int dim, int rot, int v_dim, int heads) {
+        using Fn = int (*)(const void*, const int*, int, int, int, const int*, const int*, int, const void*, const void*, int, int, int,
+                           int, int, void*, void*, int*, int, int*, void*);
+        static Fn f = kernel_symbol<Fn>("head_ops", "kipp_latent_expand");
+        PagedCacheView v;
+        v.page_size = expand_page();
+        v.table_width = expand_pages(cache);
+        v.n_pages = entries * v.table_width;
+        const size_t rows = (size_t)v.n_pages * v.page_size * heads;
+        v.k_pages = workspace->buffer("latent_keys", rows * (dim + rot) * 2);
+        v.v_pages = workspace->buffer("latent_values", rows * v_dim * 2);
+        int* table = workspace->get<int>("latent_table", (size_t)v.n_pages);
+        v.block_table = table;
+        run(f(cache.k_pages, cache.block_table, cache.table_width, cache.page_size, rank + rot, q_start, context_len, entries, w_k, w_v,
+              rank, dim, rot, v_dim, heads, v.k_pages, v.v_pages, table, v.table_width, status, stream),
+            "latent_expand");
+        ++latent_expansions;
+        return v;
     }
 
     // Bias, per-head norm, rotation of a part of the head and the way to an activation buffer or
@@ -1133,6 +1187,7 @@ public:
     long long mix_mma_launches = 0;         // launches of the tensor-core kernel of the mixed-head attention
     long long group_launches = 0;           // launches of the tensor-core kernel for groups of heads (few tokens)
     long long mix_tc_launches = 0;          // launches of the tcgen05 prompt kernel with the options of that attention
+    long long latent_expansions = 0;        // prompts whose heads' keys and values were made from cached latents
     long long shared_key_launches = 0;      // launches of the tensor-core kernel for one shared key row per token
     long long glu_epilogues = 0;            // gated activations with limits that ran inside a tensor-core product
 };

@@ -16,7 +16,10 @@
 // no value pages.  The products with W_uk and W_uv are moved to the query's side of the sums:
 // q_lat = W_uk^T q_plain (per head) meets c directly, score = q_lat . c + q_rot . k_rot, the
 // weighted sum runs over c itself, and W_uv expands it afterwards.  A step's cost then does not
-// grow with heads x context, and prompts, portions and decoded tokens take the same path.
+// grow with heads x context.  Prompt-sized steps on the tensor cores take the other order (prompt()): the keys
+// and values of every head are made from the cached latents of the step's entries first, into pages of their
+// own, and the tcgen05 prompt kernel reads them as those of any other attention: with many queries per key
+// that is a third of the work.
 // Every size, eps, scale and tensor name is a parameter of the plan.
 #pragma once
 #include "recurrent_parts.hpp"
@@ -54,7 +57,7 @@ public:
         qh_ = dim_ + rot_;
         row_ = kv_rank_ + rot_;
         kv_cols_ = shared_kv_ ? 0 : row_;
-        g_off_ = q_rank_ + kv_cols_;
+        g_off_ = pad8(q_rank_ + kv_cols_);            // (the prompt kernel reads the gate's columns 16 bytes at a time)
         g_cols_ = element_gate_ ? heads_ * v_dim_ : gate_ ? heads_ : 0;
         cols1_ = g_off_ + g_cols_;
         ld1_ = pad8(cols1_);
@@ -94,6 +97,7 @@ public:
         const size_t es = dtype_size(dtype_);
         // one matrix for the two down projections and the gate
         w_in_ = b.allocate((size_t)cols1_ * hidden_ * es, p + "dq_dkv_g");
+        cuda_check(cudaMemset(w_in_, 0, (size_t)cols1_ * hidden_ * es), "clearing a padded weight");
         char* base = static_cast<char*>(w_in_);
         b.load(p + names_.at("dq"), base, dtype_, hidden_, q_rank_, hidden_);
         if (kv_cols_) b.load(p + names_.at("dkv"), base + (size_t)q_rank_ * hidden_ * es, dtype_, hidden_, row_, hidden_);
@@ -103,10 +107,10 @@ public:
         cuda_check(cudaMemset(w_uq_, 0, (size_t)heads_ * qh_ * q_rank_ld_ * es), "clearing a padded weight");
         b.load(p + names_.at("uq"), w_uq_, dtype_, q_rank_ld_, (int64_t)heads_ * qh_, q_rank_);
         // W_uk of every head transposed to [kv_rank, dim]: it multiplies the plain part of the query
-        void* uk = b.allocate((size_t)heads_ * dim_ * kv_rank_ * es, p + names_.at("uk"));
-        b.load(p + names_.at("uk"), uk, dtype_, kv_rank_, (int64_t)heads_ * dim_, kv_rank_);
+        w_uk_ = b.allocate((size_t)heads_ * dim_ * kv_rank_ * es, p + names_.at("uk"));
+        b.load(p + names_.at("uk"), w_uk_, dtype_, kv_rank_, (int64_t)heads_ * dim_, kv_rank_);
         w_uk_t_ = b.allocate((size_t)heads_ * dim_ * kv_rank_ * es, p + names_.at("uk") + " transposed");
-        b.ops().transpose_heads(w_uk_t_, uk, dtype_, heads_, dim_, kv_rank_);
+        b.ops().transpose_heads(w_uk_t_, w_uk_, dtype_, heads_, dim_, kv_rank_);
         w_uv_ = b.allocate((size_t)heads_ * v_dim_ * kv_rank_ * es, p + names_.at("uv"));
         b.load(p + names_.at("uv"), w_uv_, dtype_, kv_rank_, (int64_t)heads_ * v_dim_, kv_rank_);
         ldo_ = pad8(heads_ * v_dim_);
@@ -124,6 +128,11 @@ public:
     }
     bool folds_rms() const override { return Ops::gemm_scale_ok(dtype_, w_in_, hidden_, w_in_, hidden_); }
     bool stores_output() const override { return true; }
+    // (the tiles of the prompt kernel)
+    std::shared_ptr<WorkPlanner> planner(const DeviceInfo&, bool) override {
+        planner_ = std::make_shared<MixTilePlanner>(Ops::attention_mix_tile());
+        return planner_;
+    }
     void forward(StepContext& ctx, const LayerRun& run, int mixer_slot, const void* h, float* residual) override {
         const int T = ctx.tokens();
         const size_t es = ctx.element();
@@ -154,6 +163,15 @@ public:
         // -- the queries: up projection, the plain part through W_uk^T, the rotated part turned
         void* q = ctx.workspace->buffer("latent_q_up", (size_t)T * ldq_ * es);
         ops.gemm(q, ctx.dtype, ldq_, cq, q_rank_ld_, w_uq_, q_rank_ld_, dtype_, T, heads_ * qh_, q_rank_ld_, EPI_STORE);
+        AttentionExtras extras;
+        extras.sink = sink_;
+        if (g_cols_) { extras.gate = proj; extras.ld_gate = ld1_; extras.gate_off = g_off_; extras.gate_dims = element_gate_ ? 1 : 0; }
+        const int *tiles = nullptr, n_tiles = planner_tiles(m, &tiles);
+        if (Ops::latent_expand_ok(ctx.dtype, kv_rank_, dim_, rot_, v_dim_, heads_) &&
+            ops.latent_prompt_ok(extras, cache, T, m.shape.entries, n_tiles, kv_rank_, dim_, rot_, v_dim_, heads_)) {
+            prompt(ctx, cache, q, cos_sin, extras, tiles, n_tiles, residual);
+            return;
+        }
         void* ql = ctx.workspace->buffer("q", (size_t)T * heads_ * row_ * es);
         ops.head_matmul(ql, (long long)heads_ * row_, row_, q, ldq_, qh_, w_uk_t_, (long long)kv_rank_ * dim_, ctx.dtype, T,
                         kv_rank_, dim_, heads_);
@@ -165,10 +183,8 @@ public:
             ops.head_segments(q, ldq_, ctx.dtype, &r, 1, nullptr, 0, 0, 0, m.positions, m.entry_of_token, T, 0, eps_);
         }
         // -- scores against [c, k_rot], the weighted sum of c, the gate
-        AttentionExtras extras;
-        extras.sink = sink_;
         extras.values_in_keys = 1;
-        if (gate_) { extras.gate = proj; extras.ld_gate = ld1_; extras.gate_off = g_off_; }
+        if (element_gate_) { extras.gate = nullptr; extras.gate_dims = 0; }      // (it belongs to the values: W_uv's product has it)
         void* lat = ctx.workspace->buffer("latent_out", (size_t)T * heads_ * kv_rank_ * es);
         ops.attention_mix(lat, ql, cache, ctx.dtype, nullptr, m.positions, m.entry_of_token, T, heads_, 1, row_, kv_rank_,
                           scale_, window_, 0, out_scale_, nullptr, 0, m.q_start, m.context_len, &extras);
@@ -182,13 +198,44 @@ public:
     }
 
 private:
+    int planner_tiles(const StepMeta& m, const int** tiles) const {
+        if (!planner_) return 0;
+        auto it = m.work.find(planner_->key());
+        if (it == m.work.end()) return 0;
+        *tiles = it->second[1];
+        return m.work_sizes.at(planner_->key())[1] / 2;
+    }
+    // q: the up projection's rows [T, heads, dim | rot]
+    void prompt(StepContext& ctx, const PagedCacheView& cache, const void* q, const float* cos_sin, const AttentionExtras& extras,
+                const int* tiles, int n_tiles, float* residual) {
+        const int T = ctx.tokens();
+        Ops& ops = *ctx.ops;
+        const StepMeta& m = *ctx.meta;
+        const PagedCacheView kv = ops.latent_expand(cache, m.q_start, m.context_len, m.shape.entries, w_uk_, w_uv_, kv_rank_, dim_, rot_,
+                                                    v_dim_, heads_);
+        const void* qr = q;
+        if (rot_ > 0) {
+            HeadSegment r;
+            r.src_off = 0; r.heads = heads_; r.dim = qh_; r.src_stride = qh_; r.rot_off = dim_; r.rot = rot_; r.cos_sin = cos_sin;
+            r.interleaved = interleaved_ ? 1 : 0;
+            void* dst = ctx.workspace->buffer("q", (size_t)T * heads_ * qh_ * ctx.element());
+            r.target = 0; r.dst = dst; r.ld_dst = (long long)heads_ * qh_; r.dst_off = 0; r.dst_stride = qh_;
+            ops.head_segments(q, ldq_, ctx.dtype, &r, 1, nullptr, 0, 0, 0, m.positions, m.entry_of_token, T, 0, eps_);
+            qr = dst;
+        }
+        void* attn = ctx.workspace->buffer("attn_out", (size_t)T * ldo_ * ctx.element());
+        ops.attention_prompt_tc(attn, qr, kv, T, heads_, heads_, qh_, v_dim_, scale_, window_, out_scale_, m.q_start, m.context_len, extras,
+                                tiles, n_tiles);
+        output_product(ctx, residual, attn, ldo_, w_o_, ldo_, dtype_, hidden_, ldo_);
+    }
     int hidden_ = 0, heads_ = 0, dim_ = 0, rot_ = 0, v_dim_ = 0, kv_rank_ = 0, q_rank_ = 0, window_ = 0;
     int qh_ = 0, row_ = 0, kv_cols_ = 0, g_cols_ = 0, g_off_ = 0, cols1_ = 0, ld1_ = 0, q_rank_ld_ = 0, ldq_ = 0, ldo_ = 0, gate_ = 0, dtype_ = BF16;
     bool sink_on_ = false, element_gate_ = false, interleaved_ = false, shared_kv_ = false;
     float eps_ = 0.f, scale_ = 1.f, out_scale_ = 1.f;
     std::unique_ptr<PositionEncoding> position_;
+    std::shared_ptr<MixTilePlanner> planner_;
     std::map<std::string, std::string> names_;
-    void *w_in_ = nullptr, *w_uq_ = nullptr, *w_uk_t_ = nullptr, *w_uv_ = nullptr, *w_o_ = nullptr;
+    void *w_in_ = nullptr, *w_uq_ = nullptr, *w_uk_ = nullptr, *w_uk_t_ = nullptr, *w_uv_ = nullptr, *w_o_ = nullptr;
     float *dq_norm_ = nullptr, *dkv_norm_ = nullptr, *sink_ = nullptr;
 };
 

@@ -93,6 +93,12 @@ def test_latent_attention_alone(name, layer, dtype):
     h = h_dev.double().cpu()
     want = P.latent_attention(m, w, p, h, eps, P.latent_keys(m, w, p, h, eps))
     close(_in_portions(eng, layer, "mixer", h_dev, (70, 1, 79)), want, dtype, f"{name} layer {layer}")
+    counters = eng.info()["counters"]
+    # in bfloat16, where rows go by 16 bytes, prompts make the heads' keys and values first; a token does not
+    wide = dtype == "bfloat16" and name != "D"
+    assert counters["latent_expansions"] == counters["mix_tc_launches"] == (2 if wide else 0)
+    if dtype == "bfloat16" and name == "C":
+        assert counters["shared_key_launches"] == 1
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
