@@ -33,6 +33,20 @@ inline float* load_f32(Binder& b, const std::string& name, int64_t n) {
     b.load(name, d, F32, n, 1, n);
     return d;
 }
+// The convolutions of runs of channels, stored [channels, taps] each, one after another as [taps, channels]: what the
+// kernels read (neighbouring channels lie side by side).
+inline float* load_taps(Binder& b, const std::vector<std::pair<std::string, int>>& runs, int channels, int taps) {
+    const size_t bytes = (size_t)channels * taps * sizeof(float);
+    float* stored = static_cast<float*>(b.allocate(bytes, "convolutions"));
+    float* turned = static_cast<float*>(b.allocate(bytes, "convolutions by tap"));
+    int at = 0;
+    for (auto& r : runs) {
+        b.load(r.first, stored + (size_t)at * taps, F32, taps, r.second, taps);
+        at += r.second;
+    }
+    b.ops().transpose_heads(turned, stored, F32, 1, channels, taps);
+    return turned;
+}
 inline int gate_code(const std::string& g) {
     if (g == "none") return 0;
     if (g == "silu") return 1;
@@ -725,7 +739,7 @@ public:
         w_o_ = b.allocate((size_t)hidden_ * inner_ld_ * es, p + names_.at("o"));
         cuda_check(cudaMemset(w_o_, 0, (size_t)hidden_ * inner_ld_ * es), "clearing a padded weight");
         b.load(p + names_.at("o"), w_o_, dtype_, inner_ld_, hidden_, inner_);
-        conv_ = load_f32(b, p + names_.at("conv"), (int64_t)channels_ * taps_);
+        conv_ = load_taps(b, {{p + names_.at("conv"), channels_}}, channels_, taps_);
         conv_b_ = load_f32(b, p + names_.at("conv_bias"), channels_);
         dt_bias_ = load_f32(b, p + names_.at("dt_bias"), heads_);
         a_log_ = load_f32(b, p + names_.at("a_log"), heads_);
@@ -881,10 +895,8 @@ public:
         w_a2_ = padded("a2", heads_ * dim_, a_rank_, a_ld_);
         w_g2_ = padded("g2", vv_, g_rank_, g_ld_);
         w_o_ = padded("o", hidden_, vv_, vv_ld_);
-        conv_ = static_cast<float*>(b.allocate((size_t)channels_ * taps_ * sizeof(float), p + "convolutions"));
-        b.load(p + names_.at("q_conv"), conv_, F32, taps_, qk_, taps_);
-        b.load(p + names_.at("k_conv"), conv_ + (size_t)qk_ * taps_, F32, taps_, qk_, taps_);
-        b.load(p + names_.at("v_conv"), conv_ + (size_t)2 * qk_ * taps_, F32, taps_, vv_, taps_);
+        conv_ = load_taps(b, {{p + names_.at("q_conv"), qk_}, {p + names_.at("k_conv"), qk_}, {p + names_.at("v_conv"), vv_}}, channels_,
+                          taps_);
         dt_bias_ = load_f32(b, p + names_.at("dt_bias"), (int64_t)heads_ * dim_);
         a_log_ = load_f32(b, p + names_.at("a_log"), heads_);
         norm_ = load_f32(b, p + names_.at("norm"), v_dim_);

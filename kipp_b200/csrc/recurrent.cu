@@ -75,7 +75,7 @@ struct ScanArgs {
     const float* cos_sin; int rot;         // retention: [T, rot / 2, 2] or null
     float* state;                          // [slots, heads, dim, v_dim]
     const int* q_start; const int* slots;
-    int heads, dim, v_dim, batch;
+    int heads, dim, v_dim, batch, entries;
     float k_scale, eps, out_scale;
     int gate;                              // 0 none, 1 silu, 2 sigmoid
     // gated memory: columns of the two gates in proj, their biases [heads], the cap, the scale of q
@@ -316,36 +316,15 @@ recurrent_scan_kernel(const ScanArgs a, const float* __restrict__ vec, float* __
                 // the decayed state meets k and q in one pass and both sums travel together; the token's own
                 // write then joins the output as (q . k) u
                 float kr[CHUNK], us4[4] = {0.f, 0.f, 0.f, 0.f}, os4[4] = {0.f, 0.f, 0.f, 0.f};
-                if (VEC) {
 #pragma unroll
-                    for (int g = 0; g < CHUNK / 4; ++g) {
-                        const int r = 4 * (p + P * g);
-                        if (r < D) {
-                            const float4 q4 = *reinterpret_cast<const float4*>(tok + r);
-                            const float4 k4 = *reinterpret_cast<const float4*>(tok + D + r);
-                            const float4 g4 = *reinterpret_cast<const float4*>(tok + 2 * D + r);
-                            const float qq[4] = {q4.x, q4.y, q4.z, q4.w}, kk[4] = {k4.x, k4.y, k4.z, k4.w}, gg[4] = {g4.x, g4.y, g4.z, g4.w};
-#pragma unroll
-                            for (int j = 0; j < 4; ++j) {
-                                const float s = S[4 * g + j] * gg[j];
-                                S[4 * g + j] = s;
-                                kr[4 * g + j] = kk[j];
-                                us4[j] = fmaf(kk[j], s, us4[j]);
-                                os4[j] = fmaf(qq[j], s, os4[j]);
-                            }
-                        }
+                for (int i = 0; i < CHUNK; ++i)
+                    if (row_of(i) < D) {
+                        const float s = S[i] * tok[2 * D + row_of(i)];
+                        S[i] = s;
+                        kr[i] = tok[D + row_of(i)];
+                        us4[i & 3] = fmaf(kr[i], s, us4[i & 3]);
+                        os4[i & 3] = fmaf(tok[row_of(i)], s, os4[i & 3]);
                     }
-                } else {
-#pragma unroll
-                    for (int i = 0; i < CHUNK; ++i)
-                        if (p + P * i < D) {
-                            const float s = S[i] * base[2 * D + P * i];
-                            S[i] = s;
-                            kr[i] = base[D + P * i];
-                            us4[i & 3] = fmaf(kr[i], s, us4[i & 3]);
-                            os4[i & 3] = fmaf(base[P * i], s, os4[i & 3]);
-                        }
-                }
                 us = (us4[0] + us4[1]) + (us4[2] + us4[3]);
                 o = (os4[0] + os4[1]) + (os4[2] + os4[3]);
 #pragma unroll
@@ -488,7 +467,7 @@ ssd_conv_kernel(const ScanArgs a, float* __restrict__ conv_out) {
         const int r = row - (taps - 1 - j);                         // the row that meets tap j
         const float in = r >= first ? to_f32(proj[(size_t)r * a.ld_proj + a.xbc_off + c])
                                     : kept[(size_t)(taps - 1 + r - first) * channels + c];
-        acc = fmaf(a.conv_w[(size_t)c * taps + j], in, acc);
+        acc = fmaf(a.conv_w[(size_t)j * channels + c], in, acc);
     }
     conv_out[(size_t)row * channels + c] = acc / (1.0f + expf(-acc));
 }
@@ -525,6 +504,20 @@ ssd_prepare_kernel(const ScanArgs a, const float* __restrict__ conv_out, float* 
         dst[2 * D + 2] = 0.f;
         dst[2 * D + 3] = 0.f;
     }
+}
+
+// Decay and step size of every (token, head), where the convolution's kernel does not form them.
+template <typename T>
+__global__ void __launch_bounds__(128)
+ssd_dt_kernel(const ScanArgs a, float2* __restrict__ dts, int tokens) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i >= (long long)tokens * a.heads) return;
+    const int h = (int)(i % a.heads);
+    const float raw = to_f32(static_cast<const T*>(a.proj)[(size_t)(i / a.heads) * a.ld_proj + a.dt_off + h]) + a.dt_bias[h];
+    const float dt = fmaxf(raw, 0.f) + log1pf(expf(-fabsf(raw)));
+    dts[i] = make_float2(expf(-expf(a.a_log[h]) * dt), dt);
 }
 
 // The gated delta rule's token vectors.  A warp per (token, head) makes the unit vectors of its group's q and k
@@ -648,11 +641,400 @@ ssd_conv_keep_kernel(const ScanArgs a) {
 
 // (P below 8 comes with at most 8 rows per thread, see launch_scan; rows that do not go by fours are rare, so two
 // sizes of the unrolled loop serve them)
+// The launch of a kernel whose blocks walk tokens: many tokens per entry make its blocks long-running, and those want
+// to be spread over the SMs.
+template <typename... KArgs, typename... Args>
+int launch_walk(const ScanArgs& a, int tokens, void (*kernel)(KArgs...), dim3 grid, dim3 block, size_t smem, cudaStream_t stream,
+                Args&&... args) {
+    if (tokens >= 8 * a.entries) return kipp_launch_spread(kernel, grid, block, smem, stream, static_cast<Args&&>(args)...);
+    return kipp_launch(kernel, grid, block, smem, stream, 1, static_cast<Args&&>(args)...);
+}
+
+// ---------------------------------------------------------------------------
+// The two recurrences whose scans are built for heads that go by fours (other sizes take the template above).  Both
+// walk an entry's tokens in order with S in registers; what a token needs of shared memory is fetched into registers
+// while the token before is worked on, so that only the recurrence itself is a chain.  The order of every sum
+// depends on the sizes only.
+//
+// State space: a thread owns 4 columns x R rows (P threads per group of columns, rows in groups of four dealt out in
+// turn), so that a token's C and B serve four columns per load; the four outputs' sums over P lanes meet in P's
+// logarithm plus one shuffles (every exchange also halves the columns a lane is responsible for).  C, B and x come
+// straight out of the convolved rows, decay and step size from dts [tokens][heads].
+// Rows go through the arithmetic in pairs (float32 pairs in one instruction).
+constexpr int SCAN_COLS = 4;
+__device__ __forceinline__ float2 mul2(float2 a, float2 b) {
+    float2 d;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(reinterpret_cast<unsigned long long&>(d))
+        : "l"(reinterpret_cast<const unsigned long long&>(a)), "l"(reinterpret_cast<const unsigned long long&>(b)));
+    return d;
+}
+__device__ __forceinline__ float2 fma2(float2 a, float2 b, float2 c) {
+    float2 d;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(reinterpret_cast<unsigned long long&>(d))
+        : "l"(reinterpret_cast<const unsigned long long&>(a)), "l"(reinterpret_cast<const unsigned long long&>(b)),
+          "l"(reinterpret_cast<const unsigned long long&>(c)));
+    return d;
+}
+__device__ __forceinline__ float2 both(float v) { return make_float2(v, v); }
+struct TokenBatch {                          // two buffers of `tokens` tokens of `floats` floats
+    int tokens, floats;
+};
+__host__ __device__ inline TokenBatch token_batch(int floats) {
+    TokenBatch b;
+    b.floats = floats;
+    b.tokens = floats * 4 * 32 <= 22 * 1024 ? 32 : (22 * 1024) / (floats * 4);
+    if (b.tokens < 1) b.tokens = 1;
+    return b;
+}
+// EXACT: the P threads' rows are the head's, none too many.
+template <int P, int R, int WARPS, bool EXACT>
+__global__ void __launch_bounds__(32 * WARPS)
+ssd_scan_kernel(const ScanArgs a, const float* __restrict__ conv, const float2* __restrict__ dts, float* __restrict__ o_raw, int v_slices) {
+    extern __shared__ __align__(16) float smem[];
+    constexpr int COLS = SCAN_COLS * 32 * WARPS / P, THREADS = 32 * WARPS;
+    const int D = a.dim, V = a.v_dim;
+    const TokenBatch tb = token_batch(2 * D + COLS + 4);
+    pdl_launch_dependents();
+    pdl_wait();
+    const int tid = threadIdx.x, p = tid % P, slice = blockIdx.x % v_slices, eh = blockIdx.x / v_slices;
+    const int e = eh / a.heads, h = eh % a.heads, g = h / (a.heads / a.groups);
+    const int row0 = a.q_start[e], n_tok = a.q_start[e + 1] - row0;
+    const int cl = tid / P * SCAN_COLS, col = slice * COLS + cl;
+    const bool live = col < V;                                      // (V is a multiple of 4: a group is whole or absent)
+    float* S_slot = a.state + (size_t)a.slots[e] * (size_t)a.slot_stride + (size_t)h * D * V;
+    const int inner = a.heads * V;
+    const float* b_at = conv + inner + (size_t)g * D;
+    const float* c_at = conv + inner + (size_t)(a.groups + g) * D;
+    // a token in a buffer: C [D], B [D], x [COLS], (decay, step size, -, -)
+    auto fetch = [&](int t0, float* buf) {
+        // (a warp takes whole tokens: nothing to divide)
+        const int nb = min(tb.tokens, n_tok - t0), d4 = D / 4, per = 2 * d4 + COLS / 4;
+        for (int t = tid >> 5; t < nb; t += WARPS) {
+            const size_t at = (size_t)(row0 + t0 + t) * a.channels;
+            const uint32_t to = smem_address(buf + (size_t)t * tb.floats);
+            for (int c = tid & 31; c < per; c += 32) {
+                const int x = slice * COLS + 4 * (c - 2 * d4);
+                const bool ok = c < 2 * d4 || x < V;
+                const float* src = c < d4 ? c_at + 4 * c : c < 2 * d4 ? b_at + 4 * (c - d4) : conv + (ok ? h * V + x : 0);
+                cp_async16(to + 16 * c, src + at, ok ? 16 : 0);
+            }
+        }
+        for (int t = tid; t < nb; t += THREADS)
+            *reinterpret_cast<float2*>(buf + (size_t)t * tb.floats + 2 * D + COLS) = dts[(size_t)(row0 + t0 + t) * a.heads + h];
+        cp_async_commit();
+    };
+    // row i of this thread: 4 (p + P (i / 4)) + i % 4; S[i / 2][c] holds rows i and i + 1 of column c
+    float2 S[R / 2][SCAN_COLS];
+#pragma unroll
+    for (int i = 0; i < R; ++i) {
+        const int r = 4 * (p + P * (i >> 2)) + (i & 3);
+        const float4 s4 = live && r < D ? *reinterpret_cast<const float4*>(S_slot + (size_t)r * V + col) : make_float4(0.f, 0.f, 0.f, 0.f);
+        const float e[4] = {s4.x, s4.y, s4.z, s4.w};
+#pragma unroll
+        for (int c = 0; c < SCAN_COLS; ++c) (i & 1 ? S[i >> 1][c].y : S[i >> 1][c].x) = e[c];
+    }
+    float2 cv[R / 2], bv[R / 2], keep, tx[SCAN_COLS];
+    auto take = [&](const float* tok) {
+#pragma unroll
+        for (int q = 0; q < R / 4; ++q) {
+            const int r = 4 * (p + P * q);
+            float4 c4 = make_float4(0.f, 0.f, 0.f, 0.f), b4 = c4;
+            if (EXACT || r < D) {
+                c4 = *reinterpret_cast<const float4*>(tok + r);
+                b4 = *reinterpret_cast<const float4*>(tok + D + r);
+            }
+            cv[2 * q] = make_float2(c4.x, c4.y); cv[2 * q + 1] = make_float2(c4.z, c4.w);
+            bv[2 * q] = make_float2(b4.x, b4.y); bv[2 * q + 1] = make_float2(b4.z, b4.w);
+        }
+        const float4 x4 = *reinterpret_cast<const float4*>(tok + 2 * D + cl);
+        const float2 kd = *reinterpret_cast<const float2*>(tok + 2 * D + COLS);
+        keep = both(kd.x);
+        tx[0] = both(kd.y * x4.x); tx[1] = both(kd.y * x4.y); tx[2] = both(kd.y * x4.z); tx[3] = both(kd.y * x4.w);
+    };
+    fetch(0, smem);
+    int buf = 0;
+    for (int t0 = 0; t0 < n_tok; t0 += tb.tokens, buf ^= 1) {
+        const int nb = min(tb.tokens, n_tok - t0);
+        if (t0 + tb.tokens < n_tok) fetch(t0 + tb.tokens, smem + (size_t)(buf ^ 1) * tb.tokens * tb.floats);
+        else cp_async_commit();
+        cp_async_wait<1>();
+        __syncthreads();
+        const float* toks = smem + (size_t)buf * tb.tokens * tb.floats;
+        take(toks);
+        // a token's sums travel while the next token is worked on: the chain of shuffles is nobody's wait
+        float last[SCAN_COLS] = {0.f, 0.f, 0.f, 0.f};
+        float* out = o_raw + (size_t)(row0 + t0) * inner + h * V + col + 2 * (p & 1) + (p >> 1);      // lanes p < 4
+        auto meet = [&](const float* o) {
+            // lane p of a group of P ends up with column 2 (p & 1) + (p >> 1 & 1)
+            const bool odd = p & 1, second = p & 2;
+            float k0 = odd ? o[2] : o[0], k1 = odd ? o[3] : o[1];
+            k0 += __shfl_xor_sync(0xffffffffu, odd ? o[0] : o[2], 1);
+            k1 += __shfl_xor_sync(0xffffffffu, odd ? o[1] : o[3], 1);
+            float y = (second ? k1 : k0) + __shfl_xor_sync(0xffffffffu, second ? k0 : k1, 2);
+#pragma unroll
+            for (int x = 4; x < P; x <<= 1) y += __shfl_xor_sync(0xffffffffu, y, x);
+            return y;
+        };
+        const bool writes = live && p < SCAN_COLS;
+        for (int t = 0; t < nb; ++t) {
+            float2 o[SCAN_COLS];
+            const float y = meet(last);
+#pragma unroll
+            for (int i = 0; i < R / 2; ++i)
+#pragma unroll
+                for (int c = 0; c < SCAN_COLS; ++c) {
+                    S[i][c] = fma2(bv[i], tx[c], mul2(keep, S[i][c]));
+                    o[c] = i == 0 ? mul2(cv[i], S[i][c]) : fma2(cv[i], S[i][c], o[c]);
+                }
+            take(toks + (size_t)min(t + 1, nb - 1) * tb.floats);
+            if (writes && t > 0) {
+                *out = y;
+                out += inner;
+            }
+#pragma unroll
+            for (int c = 0; c < SCAN_COLS; ++c) last[c] = o[c].x + o[c].y;
+        }
+        const float y = meet(last);
+        if (writes) *out = y;
+        __syncthreads();                    // the buffer is free for the batch after the next
+    }
+#pragma unroll
+    for (int i = 0; i < R; ++i) {
+        const int r = 4 * (p + P * (i >> 2)) + (i & 3);
+        auto at = [&](int c) { return i & 1 ? S[i >> 1][c].y : S[i >> 1][c].x; };
+        if (live && r < D) *reinterpret_cast<float4*>(S_slot + (size_t)r * V + col) = make_float4(at(0), at(1), at(2), at(3));
+    }
+}
+
+// The gated delta rule: a thread owns R rows of one column.  The decayed state meets k and q in one pass and both
+// sums travel through the same shuffles; the token's own write then joins the output as (q . k) u.
+template <int P, int R, int WARPS, bool EXACT>
+__global__ void __launch_bounds__(32 * WARPS)
+gated_delta_scan_kernel(const ScanArgs a, const float* __restrict__ vec, float* __restrict__ o_raw, int v_slices, int tokens) {
+    extern __shared__ __align__(16) float smem[];
+    constexpr int COLS = 32 * WARPS / P;
+    const int D = a.dim, V = a.v_dim, nvd = 3 * D + 4, rec = nvd + V;
+    const TokenBatch tb = token_batch(nvd + COLS);
+    pdl_launch_dependents();
+    pdl_wait();
+    const int tid = threadIdx.x, p = tid % P, slice = blockIdx.x % v_slices, eh = blockIdx.x / v_slices;
+    const int e = eh / a.heads, h = eh % a.heads;
+    const int row0 = a.q_start[e], n_tok = a.q_start[e + 1] - row0;
+    const int cl = tid / P, col = slice * COLS + cl;
+    const bool live = col < V;
+    float* S_slot = a.state + (size_t)a.slots[e] * (size_t)a.slot_stride + (size_t)h * D * V;
+    const float* recs = vec + ((size_t)h * tokens + row0) * rec;
+    auto fetch = [&](int t0, float* buf) {
+        const int nb = min(tb.tokens, n_tok - t0), n4 = nvd / 4, per = n4 + COLS / 4;
+        for (int t = tid >> 5; t < nb; t += WARPS) {
+            const float* src = recs + (size_t)(t0 + t) * rec;
+            const uint32_t to = smem_address(buf + (size_t)t * tb.floats);
+            for (int c = tid & 31; c < per; c += 32) {
+                const int x = slice * COLS + 4 * (c - n4);
+                const bool ok = c < n4 || x < V;                    // (V is a multiple of 4 here)
+                cp_async16(to + 16 * c, src + (c < n4 ? 4 * c : ok ? nvd + x : 0), ok ? 16 : 0);
+            }
+        }
+        cp_async_commit();
+    };
+    float2 S[R / 2];                        // pairs of neighbouring rows
+#pragma unroll
+    for (int i = 0; i < R; ++i) {
+        const int r = 4 * (p + P * (i >> 2)) + (i & 3);
+        (i & 1 ? S[i >> 1].y : S[i >> 1].x) = live && r < D ? S_slot[(size_t)r * V + col] : 0.f;
+    }
+    struct Token { float2 q[R / 2], k[R / 2], g[R / 2]; float beta, qk, v; };
+    auto take = [&](const float* tok, Token& n) {
+#pragma unroll
+        for (int q = 0; q < R / 4; ++q) {
+            const int r = 4 * (p + P * q);
+            float4 q4 = make_float4(0.f, 0.f, 0.f, 0.f), k4 = q4, g4 = q4;
+            if (EXACT || r < D) {
+                q4 = *reinterpret_cast<const float4*>(tok + r);
+                k4 = *reinterpret_cast<const float4*>(tok + D + r);
+                g4 = *reinterpret_cast<const float4*>(tok + 2 * D + r);
+            }
+            n.q[2 * q] = make_float2(q4.x, q4.y); n.q[2 * q + 1] = make_float2(q4.z, q4.w);
+            n.k[2 * q] = make_float2(k4.x, k4.y); n.k[2 * q + 1] = make_float2(k4.z, k4.w);
+            n.g[2 * q] = make_float2(g4.x, g4.y); n.g[2 * q + 1] = make_float2(g4.z, g4.w);
+        }
+        n.beta = tok[3 * D];
+        n.qk = tok[3 * D + 1];
+        n.v = tok[nvd + cl];
+    };
+    fetch(0, smem);
+    int buf = 0;
+    for (int t0 = 0; t0 < n_tok; t0 += tb.tokens, buf ^= 1) {
+        const int nb = min(tb.tokens, n_tok - t0);
+        if (t0 + tb.tokens < n_tok) fetch(t0 + tb.tokens, smem + (size_t)(buf ^ 1) * tb.tokens * tb.floats);
+        else cp_async_commit();
+        cp_async_wait<1>();
+        __syncthreads();
+        const float* toks = smem + (size_t)buf * tb.tokens * tb.floats;
+        float* out = o_raw + (size_t)(row0 + t0) * (a.heads * V) + h * V + col;
+        const bool writes = live && p == 0;
+        Token even, odd;
+        // one token from `now`; `next` is fetched meanwhile (the last token of a batch fetches itself again)
+        auto step = [&](int t, const Token& now, Token& next) {
+            // (two sums per product, so that no chain is longer than a quarter of the rows)
+            float2 us[2], os[2];
+#pragma unroll
+            for (int i = 0; i < R / 2; ++i) {
+                S[i] = mul2(S[i], now.g[i]);
+                us[i & 1] = i < 2 ? mul2(now.k[i], S[i]) : fma2(now.k[i], S[i], us[i & 1]);
+            }
+            float uy = (us[0].x + us[0].y) + (us[1].x + us[1].y);
+#pragma unroll
+            for (int x = P / 2; x > 0; x >>= 1) uy += __shfl_xor_sync(0xffffffffu, uy, x);
+#pragma unroll
+            for (int i = 0; i < R / 2; ++i) os[i & 1] = i < 2 ? mul2(now.q[i], S[i]) : fma2(now.q[i], S[i], os[i & 1]);
+            float oy = (os[0].x + os[0].y) + (os[1].x + os[1].y);
+#pragma unroll
+            for (int x = P / 2; x > 0; x >>= 1) oy += __shfl_xor_sync(0xffffffffu, oy, x);
+            take(toks + (size_t)min(t + 1, nb - 1) * tb.floats, next);
+            const float u = now.beta * (now.v - uy);
+            const float2 u2 = both(u);
+#pragma unroll
+            for (int i = 0; i < R / 2; ++i) S[i] = fma2(now.k[i], u2, S[i]);
+            if (writes) *out = fmaf(now.qk, u, oy);
+            out += a.heads * V;
+        };
+        take(toks, even);
+        int t = 0;
+        for (; t + 1 < nb; t += 2) {
+            step(t, even, odd);
+            step(t + 1, odd, even);
+        }
+        if (t < nb) step(t, even, odd);
+        __syncthreads();                    // the buffer is free for the batch after the next
+    }
+#pragma unroll
+    for (int i = 0; i < R; ++i) {
+        const int r = 4 * (p + P * (i >> 2)) + (i & 3);
+        if (live && r < D) S_slot[(size_t)r * V + col] = i & 1 ? S[i >> 1].y : S[i >> 1].x;
+    }
+}
+
+// The convolution for channels that go by eights (four in 32-bit) and up to 4 taps: a thread takes 16 bytes of
+// channels over a run of CONV_RUN tokens and reads every input once (the last taps - 1 stay in registers; they come
+// anew where a run or an entry starts).  The order of a channel's sum is ssd_conv_kernel's.  The last row of
+// blocks forms the state space layer's decays and step sizes, dts [tokens][heads] (null: none).
+constexpr int CONV_RUN = 8, CONV_THREADS = 128;
+template <typename T, int TAPS>
+__global__ void __launch_bounds__(CONV_THREADS)
+conv_run_kernel(const ScanArgs a, float* __restrict__ conv_out, float2* __restrict__ dts, int tokens) {
+    constexpr int VEC = 16 / (int)sizeof(T);
+    pdl_launch_dependents();
+    pdl_wait();
+    const int r0 = blockIdx.x * CONV_RUN, r1 = min(tokens, r0 + CONV_RUN);
+    const T* proj = static_cast<const T*>(a.proj);
+    if (dts != nullptr && blockIdx.y == gridDim.y - 1) {
+        for (int i = threadIdx.x; i < (r1 - r0) * a.heads; i += CONV_THREADS) {
+            const int row = r0 + i / a.heads, h = i % a.heads;
+            const float raw = to_f32(proj[(size_t)row * a.ld_proj + a.dt_off + h]) + a.dt_bias[h];
+            const float dt = fmaxf(raw, 0.f) + log1pf(expf(-fabsf(raw)));       // softplus, exact at both ends
+            dts[(size_t)row * a.heads + h] = make_float2(expf(-expf(a.a_log[h]) * dt), dt);
+        }
+        return;
+    }
+    const int c = (blockIdx.y * CONV_THREADS + threadIdx.x) * VEC;
+    if (c >= a.channels) return;
+    float w[VEC][TAPS], bias[VEC], in[TAPS][VEC];              // in[TAPS - 1]: the current token's
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) {
+        bias[i] = a.conv_b != nullptr ? a.conv_b[c + i] : 0.f;
+#pragma unroll
+        for (int j = 0; j < TAPS; ++j) w[i][j] = a.conv_w[(size_t)j * a.channels + c + i];
+    }
+    auto load = [&](int row, float* to) {
+        const uint4 raw = *reinterpret_cast<const uint4*>(proj + (size_t)row * a.ld_proj + a.xbc_off + c);
+        const T* e = reinterpret_cast<const T*>(&raw);
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) to[i] = to_f32(e[i]);
+    };
+    int end = r0;                                              // where the entry of the run's next token ends
+    for (int row = r0; row < r1; ++row) {
+        if (row == end || row == r0) {
+            const int e = a.entry_of_token[row], first = a.q_start[e];
+            end = a.q_start[e + 1];
+            const float* kept = a.state + (size_t)a.slots[e] * (size_t)a.slot_stride + a.kept_off;     // [TAPS - 1][channels]
+#pragma unroll
+            for (int j = 0; j < TAPS - 1; ++j) {
+                const int r = row - (TAPS - 1 - j);
+                if (r >= first) {
+                    load(r, in[j]);
+                } else {
+#pragma unroll
+                    for (int i = 0; i < VEC; ++i) in[j][i] = kept[(size_t)(TAPS - 1 + r - first) * a.channels + c + i];
+                }
+            }
+        }
+        load(row, in[TAPS - 1]);
+        float y[VEC];
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) {
+            float acc = bias[i];
+#pragma unroll
+            for (int j = 0; j < TAPS; ++j) acc = fmaf(w[i][j], in[j][i], acc);
+            y[i] = acc / (1.0f + expf(-acc));
+#pragma unroll
+            for (int j = 0; j < TAPS - 1; ++j) in[j][i] = in[j + 1][i];
+        }
+#pragma unroll
+        for (int i = 0; i < VEC; i += 4)
+            *reinterpret_cast<float4*>(conv_out + (size_t)row * a.channels + c + i) = make_float4(y[i], y[i + 1], y[i + 2], y[i + 3]);
+    }
+}
+template <typename T>
+int launch_conv(const ScanArgs& a, float* conv_out, float2* dts, int tokens, bool run, cudaStream_t stream) {
+    if (!run)
+        return kipp_launch(ssd_conv_kernel<T>, dim3((unsigned)tokens, (unsigned)((a.channels + 255) / 256)), dim3(256), 0, stream, 1, a,
+                           conv_out);
+    constexpr int VEC = 16 / (int)sizeof(T);
+    const dim3 grid((unsigned)((tokens + CONV_RUN - 1) / CONV_RUN),
+                    (unsigned)((a.channels / VEC + CONV_THREADS - 1) / CONV_THREADS + (dts != nullptr ? 1 : 0)));
+    auto go = [&](auto kernel) { return kipp_launch(kernel, grid, dim3(CONV_THREADS), 0, stream, 1, a, conv_out, dts, tokens); };
+    switch (a.taps) {
+    case 1: return go(conv_run_kernel<T, 1>);
+    case 2: return go(conv_run_kernel<T, 2>);
+    case 3: return go(conv_run_kernel<T, 3>);
+    default: return go(conv_run_kernel<T, 4>);
+    }
+}
+template <typename T> bool conv_run_ok(const ScanArgs& a) {
+    constexpr int VEC = 16 / (int)sizeof(T);
+    return a.taps <= 4 && a.channels % VEC == 0 && a.ld_proj % VEC == 0 && a.xbc_off % VEC == 0 && ((uintptr_t)a.proj & 15) == 0;
+}
+// Whether the scans built for heads that go by fours take this one.
+inline bool scan_by_fours(const ScanArgs& a) {
+    return a.dim % 4 == 0 && a.v_dim % 4 == 0 && a.dim <= 256 && a.slot_stride % 4 == 0 && ((uintptr_t)a.state & 15) == 0;
+}
+// (32 columns a block)
+template <int P, int R>
+int launch_ssd_scan(const ScanArgs& a, const float* conv, const float2* dts, float* o_raw, int entries, int tokens, cudaStream_t stream) {
+    constexpr int WARPS = P / 4, COLS = SCAN_COLS * 32 * WARPS / P;
+    const TokenBatch tb = token_batch(2 * a.dim + COLS + 4);
+    const int slices = (a.v_dim + COLS - 1) / COLS;
+    return launch_walk(a, tokens, a.dim == P * R ? ssd_scan_kernel<P, R, WARPS, true> : ssd_scan_kernel<P, R, WARPS, false>,
+                       dim3((unsigned)(entries * a.heads * slices)), dim3(32 * WARPS), (size_t)2 * tb.tokens * tb.floats * sizeof(float),
+                       stream, a, conv, dts, o_raw, slices);
+}
+// (8 columns a block: the more blocks, the fewer warps share an SM, and a token's chain is what this scan is bound by)
+template <int P, int R>
+int launch_gated_delta_scan(const ScanArgs& a, const float* vec, float* o_raw, int entries, int tokens, cudaStream_t stream) {
+    constexpr int WARPS = P / 4, COLS = 32 * WARPS / P;
+    const TokenBatch tb = token_batch(3 * a.dim + 4 + COLS);
+    const int slices = (a.v_dim + COLS - 1) / COLS;
+    return launch_walk(a, tokens, a.dim == P * R ? gated_delta_scan_kernel<P, R, WARPS, true> : gated_delta_scan_kernel<P, R, WARPS, false>,
+                       dim3((unsigned)(entries * a.heads * slices)), dim3(32 * WARPS), (size_t)2 * tb.tokens * tb.floats * sizeof(float),
+                       stream, a, vec, o_raw, slices, tokens);
+}
+
 template <typename T, int DELTA, int P, bool VEC>
 int launch_scan_rows(const ScanArgs& b, const float* vec, float* o_raw, int slices, int tokens, dim3 grid, size_t smem,
                      cudaStream_t stream) {
     const int chunk = (b.dim + P - 1) / P;
-#define KIPP_SCAN(C) return kipp_launch(recurrent_scan_kernel<T, DELTA, P, C, VEC>, grid, dim3(VS * P), smem, stream, 1, b, vec, o_raw, slices, tokens)
+#define KIPP_SCAN(C) return launch_walk(b, tokens, recurrent_scan_kernel<T, DELTA, P, C, VEC>, grid, dim3(VS * P), smem, stream, b, vec, o_raw, slices, tokens)
     if constexpr (P < 8) {
         if (chunk > 8) return KIPP_ERR_ARG;
         KIPP_SCAN(8);
@@ -693,20 +1075,47 @@ int launch_scan(const ScanArgs& a, int entries, int tokens, float* scratch, cuda
     if (batch < 1) return KIPP_ERR_ARG;
     ScanArgs b = a;
     b.batch = batch;
+    b.entries = entries;
     float* vec = scratch;
     float* o_raw = scratch + (size_t)tokens * a.heads * (NV * D + XG + V);
     const long long warps = (long long)tokens * a.heads;
     const dim3 wgrid((unsigned)((warps + 3) / 4));
     int rc = 0;
     constexpr bool CONV = DELTA == SSD || DELTA == GATED_DELTA;
+    bool scanned = false;
     const int channels = a.channels;
     if constexpr (CONV) {
         if (conv_out == nullptr) return KIPP_ERR_ARG;
-        rc = kipp_launch(ssd_conv_kernel<T>, dim3((unsigned)tokens, (unsigned)((channels + 255) / 256)), dim3(256), 0, stream, 1, b,
-                         conv_out);
+        const bool by_fours = scan_by_fours(b) && ((uintptr_t)conv_out & 15) == 0 && ((uintptr_t)scratch & 15) == 0;
+        // the state space layer's scan reads the convolved rows themselves; decays and step sizes lie where the
+        // records would
+        const bool direct = DELTA == SSD && by_fours && channels % 4 == 0, run = conv_run_ok<T>(b) && (DELTA != SSD || direct);
+        float2* dts = direct ? reinterpret_cast<float2*>(vec) : nullptr;
+        rc = launch_conv<T>(b, conv_out, run ? dts : nullptr, tokens, run, stream);
         if (rc) return rc;
-        rc = kipp_launch(DELTA == SSD ? ssd_prepare_kernel<T> : gated_delta_prepare_kernel<T>, wgrid, dim3(128), 0, stream, 1, b,
-                         (const float*)conv_out, vec, tokens);
+        if (DELTA == SSD && direct && !run) {
+            rc = kipp_launch(ssd_dt_kernel<T>, dim3((unsigned)(((long long)tokens * a.heads + 127) / 128)), dim3(128), 0, stream, 1, b, dts,
+                             tokens);
+        } else if (!direct) {
+            rc = kipp_launch(DELTA == SSD ? ssd_prepare_kernel<T> : gated_delta_prepare_kernel<T>, wgrid, dim3(128), 0, stream, 1, b,
+                             (const float*)conv_out, vec, tokens);
+        }
+        if (rc) return rc;
+        if (by_fours && (DELTA != SSD || direct)) {
+            if constexpr (DELTA == SSD) {
+                const float* cv = conv_out;
+                if (D <= 32) rc = launch_ssd_scan<8, 4>(b, cv, dts, o_raw, entries, tokens, stream);
+                else if (D <= 64) rc = launch_ssd_scan<16, 4>(b, cv, dts, o_raw, entries, tokens, stream);
+                else if (D <= 128) rc = launch_ssd_scan<32, 4>(b, cv, dts, o_raw, entries, tokens, stream);
+                else rc = launch_ssd_scan<32, 8>(b, cv, dts, o_raw, entries, tokens, stream);
+            } else {
+                if (D <= 32) rc = launch_gated_delta_scan<8, 4>(b, vec, o_raw, entries, tokens, stream);
+                else if (D <= 64) rc = launch_gated_delta_scan<16, 4>(b, vec, o_raw, entries, tokens, stream);
+                else if (D <= 128) rc = launch_gated_delta_scan<32, 4>(b, vec, o_raw, entries, tokens, stream);
+                else rc = launch_gated_delta_scan<32, 8>(b, vec, o_raw, entries, tokens, stream);
+            }
+            scanned = true;
+        }
     } else {
         rc = kipp_launch(recurrent_prepare_kernel<T, DELTA>, wgrid, dim3(128), 0, stream, 1, b, vec, tokens);
     }
@@ -714,7 +1123,7 @@ int launch_scan(const ScanArgs& a, int entries, int tokens, float* scratch, cuda
     const int slices = (V + VS - 1) / VS;
     const dim3 grid((unsigned)(entries * a.heads * slices));
     const size_t smem = 2 * per_token * batch;
-    switch (P) {
+    if (!scanned) switch (P) {
     case 1: rc = launch_scan_chunk<T, DELTA, 1>(b, vec, o_raw, slices, tokens, grid, smem, stream); break;
     case 2: rc = launch_scan_chunk<T, DELTA, 2>(b, vec, o_raw, slices, tokens, grid, smem, stream); break;
     case 4: rc = launch_scan_chunk<T, DELTA, 4>(b, vec, o_raw, slices, tokens, grid, smem, stream); break;
@@ -888,7 +1297,7 @@ extern "C" long long kipp_ssd_state_floats(int heads, int groups, int dim, int v
 }
 
 // The state space layer (see the head of this file).  proj [T, ...] holds z [heads * v_dim] at z_off, the
-// channels to convolve [x | B | C] at xbc_off and dt [heads] at dt_off; conv_w [channels, taps] (the last
+// channels to convolve [x | B | C] at xbc_off and dt [heads] at dt_off; conv_w [taps, channels] (the last
 // tap meets the current token), conv_b [channels], dt_bias, a_log, d_skip [heads], norm_w [heads * v_dim]
 // (or null) float32; `dim` is the size of B and C (the state's rows).  A slot is kipp_ssd_state_floats floats.
 // conv_out: float32 [tokens, channels] of scratch for the convolved rows.  At most 16 taps.
@@ -925,7 +1334,7 @@ extern "C" long long kipp_gated_delta_state_floats(int heads, int kv_heads, int 
 
 // The gated delta rule (see the head of this file).  proj [T, ...] holds the channels to convolve [q: kv_heads * dim |
 // k: kv_heads * dim | v: heads * v_dim] at qkv_off and the write rates' pre-activations [heads] at b_off; conv_w
-// [channels, taps] (the last tap meets the current token); a_raw [T, heads * dim] and g_raw [T, heads * v_dim]
+// [taps, channels] (the last tap meets the current token); a_raw [T, heads * dim] and g_raw [T, heads * v_dim]
 // float32 are the pre-activations of the decay and of the output's gate (1 silu, 2 sigmoid); dt_bias [heads * dim],
 // a_log [heads], norm_w [v_dim] float32.  A slot is kipp_gated_delta_state_floats floats.  conv_out: float32
 // [tokens, channels] of scratch.  At most 16 taps.
