@@ -1553,6 +1553,7 @@ inline std::string Engine::info_json() {
     counters.set("mix_tc_launches", ops_.mix_tc_launches);
     counters.set("group_launches", ops_.group_launches);
     counters.set("latent_expansions", ops_.latent_expansions);
+    counters.set("token_side_launches", ops_.token_side_launches);
     counters.set("shared_key_launches", ops_.shared_key_launches);
     counters.set("glu_epilogues", ops_.glu_epilogues);
     j.set("counters", std::move(counters));

@@ -621,6 +621,22 @@ public:
         static Fn f = kernel_symbol<Fn>("elementwise", "kipp_stream_join");
         run(f(&j, dtype, rows, stream), "stream_join");
     }
+    // The same of a step of few tokens straight from the stream, g = gelu_tanh(W_gate x) * table[ids[t], off ...], in one
+    // kernel (token_side.cu); up to this many tokens it is the faster way.
+    static constexpr int SIDE_FEW_TOKENS = 64;
+    static bool token_side_few_ok(int dtype, int tokens, int width) {
+        using Fn = int (*)(int);
+        static Fn f = kernel_symbol<Fn>("token_side", "kipp_token_side_few_ok");
+        return dtype == BF16 && tokens <= SIDE_FEW_TOKENS && f(width) != 0;
+    }
+    void token_side_few(void* g, long long ld_g, const float* x, const void* w_gate, const void* table, long long ld_table, int off,
+                        const int* ids, int tokens, int width, int dim, int vocab) {
+        using Fn = int (*)(void*, long long, const float*, const void*, const void*, long long, int, const int*, int, int, int, int,
+                           void*);
+        static Fn f = kernel_symbol<Fn>("token_side", "kipp_token_side_few");
+        run(f(g, ld_g, x, w_gate, table, ld_table, off, ids, tokens, width, dim, vocab, stream), "token_side_few");
+        ++token_side_launches;
+    }
     // g[t, k] = gelu_tanh(z[t, k]) * table[ids[t], off + k] in the compute type, zeros from dim up to ld_g
     void token_side_gate(void* g, long long ld_g, const float* z, long long ld_z, const void* table, long long ld_table, int off,
                          int dtype, const int* ids, int tokens, int dim, int vocab) {
@@ -811,7 +827,7 @@ public:
         run(f(out, ld_out, proj, ld_proj, dtype, z_off, xbc_off, dt_off, conv_w, conv_b, taps, dt_bias, a_log, d_skip, norm_w,
               norm_groups, state, slot_stride, q_start, entry_of_token, slots, entries, tokens, heads, groups, dim, v_dim, eps,
               scratch, conv_out, stream),
-            "ssd_scan", taps > 1 ? 5 : 4);
+            "ssd_scan", tokens == entries ? 2 : taps > 1 ? 4 : 3);
     }
 
     // The gated delta rule (recurrent.cu, kind 5): convolution, unit keys, decays, the recurrence, norm and gate.
@@ -839,7 +855,7 @@ public:
         run(f(out, ld_out, proj, ld_proj, dtype, qkv_off, b_off, conv_w, taps, a_raw, ld_a, dt_bias, a_log, g_raw, ld_g, gate, norm_w,
               state, slot_stride, q_start, entry_of_token, slots, entries, tokens, heads, kv_heads, dim, v_dim, q_scale, eps, out_scale,
               scratch, conv_out, stream),
-            "gated_delta_scan", taps > 1 ? 5 : 4);
+            "gated_delta_scan", tokens == entries ? 1 : taps > 1 ? 5 : 4);
     }
 
     // Routing by scores (moe.cu): softmax over all `outputs` (sigmoid: of each), the choice by score + correction,
@@ -1187,6 +1203,7 @@ public:
     long long mix_mma_launches = 0;         // launches of the tensor-core kernel of the mixed-head attention
     long long group_launches = 0;           // launches of the tensor-core kernel for groups of heads (few tokens)
     long long mix_tc_launches = 0;          // launches of the tcgen05 prompt kernel with the options of that attention
+    long long token_side_launches = 0;      // gates of token sides that ran as one kernel
     long long latent_expansions = 0;        // prompts whose heads' keys and values were made from cached latents
     long long shared_key_launches = 0;      // launches of the tensor-core kernel for one shared key row per token
     long long glu_epilogues = 0;            // gated activations with limits that ran inside a tensor-core product

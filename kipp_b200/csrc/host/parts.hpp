@@ -1124,16 +1124,20 @@ public:
         const int T = ctx.tokens();
         const size_t es = ctx.element();
         Ops& ops = *ctx.ops;
-        const void* xin = x;
-        if (ctx.dtype != F32) {
-            void* xc = ctx.workspace->buffer("side_input", (size_t)T * hidden_ * es);
-            ops.convert_rows(xc, ctx.dtype, hidden_, x, F32, hidden_, T, hidden_);
-            xin = xc;
-        }
-        float* z = ctx.workspace->get<float>("side_gate_raw", (size_t)T * dim_ld_);
-        ops.gemm(z, F32, dim_ld_, xin, hidden_, w_gate_, hidden_, dtype_, T, dim_, hidden_, EPI_STORE);
         void* g = ctx.workspace->buffer("side_gate", (size_t)T * dim_ld_ * es);
-        ops.token_side_gate(g, dim_ld_, z, dim_ld_, table_, cols_, offset_, ctx.dtype, ctx.meta->token_ids, T, dim_, vocab_);
+        if (Ops::token_side_few_ok(ctx.dtype, T, hidden_)) {
+            ops.token_side_few(g, dim_ld_, x, w_gate_, table_, cols_, offset_, ctx.meta->token_ids, T, hidden_, dim_, vocab_);
+        } else {
+            const void* xin = x;
+            if (ctx.dtype != F32) {
+                void* xc = ctx.workspace->buffer("side_input", (size_t)T * hidden_ * es);
+                ops.convert_rows(xc, ctx.dtype, hidden_, x, F32, hidden_, T, hidden_);
+                xin = xc;
+            }
+            float* z = ctx.workspace->get<float>("side_gate_raw", (size_t)T * dim_ld_);
+            ops.gemm(z, F32, dim_ld_, xin, hidden_, w_gate_, hidden_, dtype_, T, dim_, hidden_, EPI_STORE);
+            ops.token_side_gate(g, dim_ld_, z, dim_ld_, table_, cols_, offset_, ctx.dtype, ctx.meta->token_ids, T, dim_, vocab_);
+        }
         float* y = ctx.workspace->get<float>("side_output", (size_t)T * hidden_);
         ops.gemm(y, F32, hidden_, g, dim_ld_, w_proj_, dim_ld_, dtype_, T, hidden_, dim_ld_, EPI_STORE);
         Ops::Join j = next;

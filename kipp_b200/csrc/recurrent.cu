@@ -568,12 +568,22 @@ gated_delta_prepare_kernel(const ScanArgs a, const float* __restrict__ conv_out,
 
 // After the scan: y = (o + D_h x) * silu(z), divided by the root mean square of its part of the row
 // (norm_groups equal parts of heads * v_dim), times the weight.  A block per (token, part).
+// keep: every entry brought one token, and the blocks of its row also move its kept inputs on.
 template <typename T>
-__global__ void __launch_bounds__(128)
-ssd_finish_kernel(const ScanArgs a, const float* __restrict__ conv_out, const float* __restrict__ o_raw) {
+__global__ void __launch_bounds__(256)
+ssd_finish_kernel(const ScanArgs a, const float* __restrict__ conv_out, const float* __restrict__ o_raw, int keep) {
     __shared__ float scratch[32];
     pdl_launch_dependents();
     pdl_wait();
+    if (keep) {
+        const int e = blockIdx.x / a.norm_groups;               // (row e is entry e's)
+        float* kept = a.state + (size_t)a.slots[e] * (size_t)a.slot_stride + a.kept_off;
+        const T* in = static_cast<const T*>(a.proj) + (size_t)e * a.ld_proj + a.xbc_off;
+        for (int c = (blockIdx.x % a.norm_groups) * blockDim.x + threadIdx.x; c < a.channels; c += a.norm_groups * blockDim.x) {
+            for (int j = 0; j + 2 < a.taps; ++j) kept[(size_t)j * a.channels + c] = kept[(size_t)(j + 1) * a.channels + c];
+            kept[(size_t)(a.taps - 2) * a.channels + c] = to_f32(in[c]);
+        }
+    }
     const size_t row = blockIdx.x / a.norm_groups;
     const int part = blockIdx.x % a.norm_groups, V = a.v_dim, inner = a.heads * V, n = inner / a.norm_groups;
     const int channels = inner + 2 * a.groups * a.dim;
@@ -1030,6 +1040,179 @@ int launch_gated_delta_scan(const ScanArgs& a, const float* vec, float* o_raw, i
                        stream, a, vec, o_raw, slices, tokens);
 }
 
+// ---------------------------------------------------------------------------
+// Steps in which every entry brings ONE token: what the scans do in three or four launches, with lanes over the
+// columns of S, so that the state, which is what such a step moves, is read and written in whole lines.  A thread owns
+// the rows rg, rg + RG, ... of one column (RG row groups); the groups' sums meet in shared memory in order.  The state's
+// loads are on their way while the convolution runs.
+// One convolved channel of an entry's only token: silu of the sum over the kept inputs and the new one.  `keep`: the
+// kept inputs move on (the caller owns the channel).
+template <typename T>
+__device__ __forceinline__ float conv_one(const ScanArgs& a, const T* __restrict__ proj, float* __restrict__ kept, int c, bool keep) {
+    const int taps = a.taps;
+    float acc = a.conv_b != nullptr ? a.conv_b[c] : 0.f;
+    const float in = to_f32(proj[a.xbc_off + c]);
+    for (int j = 0; j < taps - 1; ++j) {
+        const float old = kept[(size_t)j * a.channels + c];
+        acc = fmaf(a.conv_w[(size_t)j * a.channels + c], old, acc);
+        if (keep && j > 0) kept[(size_t)(j - 1) * a.channels + c] = old;
+    }
+    acc = fmaf(a.conv_w[(size_t)(taps - 1) * a.channels + c], in, acc);
+    if (keep && taps > 1) kept[(size_t)(taps - 2) * a.channels + c] = in;
+    return acc / (1.0f + expf(-acc));
+}
+struct TokenShape {
+    int cols, groups, rows;                  // threads along a row of S, row groups, rows per thread
+};
+inline TokenShape token_shape(int dim, int v_dim) {
+    TokenShape t;
+    t.cols = (v_dim + 31) / 32 * 32;
+    t.groups = t.cols > 512 ? 1 : 512 / t.cols;
+    if (t.groups > dim) t.groups = dim;
+    if (t.groups > 16) t.groups = 16;
+    t.rows = (dim + t.groups - 1) / t.groups;
+    return t;
+}
+constexpr int TOKEN_ROWS = 32;
+inline bool token_kernel_ok(const ScanArgs& a, int tokens) {
+    const TokenShape t = token_shape(a.dim, a.v_dim);
+    return tokens == a.entries && t.cols <= 512 && t.rows <= TOKEN_ROWS && a.dim <= 512;
+}
+
+// The gated delta rule: a block per (entry, q/k head) does the whole layer behind the projections for the heads of its
+// group: convolution (and the kept inputs), unit vectors, decays, the recurrence, norm and gate.
+template <typename T, int MR>
+__global__ void __launch_bounds__(512, MR <= 16 ? 2 : 1)
+gated_delta_token_kernel(const ScanArgs a, int cols, int groups) {
+    extern __shared__ __align__(16) float smem[];
+    __shared__ float scratch[32];
+    const int D = a.dim, V = a.v_dim, per = a.heads / a.groups;
+    float *qs = smem, *ks = qs + D, *gs = ks + D, *vs = gs + D, *red = vs + V;           // red: [2][groups][cols]
+    pdl_launch_dependents();
+    pdl_wait();
+    const int e = blockIdx.x / a.groups, kvh = blockIdx.x % a.groups, tid = threadIdx.x;
+    const int row = a.q_start[e], col = tid % cols, rg = tid / cols;
+    const T* proj = static_cast<const T*>(a.proj) + (size_t)row * a.ld_proj;
+    float* slot = a.state + (size_t)a.slots[e] * (size_t)a.slot_stride;
+    float* kept = slot + a.kept_off;
+    const bool live = col < V;
+    for (int hh = 0; hh < per; ++hh) {
+        const int h = kvh * per + hh;
+        float* S_slot = slot + (size_t)h * D * V;
+        float S[MR];
+#pragma unroll
+        for (int i = 0; i < MR; ++i) {
+            const int r = rg + groups * i;
+            S[i] = live && r < D ? S_slot[(size_t)r * V + col] : 0.f;
+        }
+        if (hh == 0)
+            for (int c = tid; c < 2 * D; c += blockDim.x) {
+                const int ch = c < D ? kvh * D + c : (a.groups + kvh) * D + c - D;
+                smem[c] = conv_one(a, proj, kept, ch, true);
+            }
+        for (int c = tid; c < V; c += blockDim.x) vs[c] = conv_one(a, proj, kept, 2 * a.groups * D + h * V + c, true);
+        const float rate = expf(a.a_log[h]);
+        for (int d = tid; d < D; d += blockDim.x) {
+            const float raw = a.a_raw[(size_t)row * a.ld_a + h * D + d] + a.dt_bias[h * D + d];
+            const float sp = fmaxf(raw, 0.f) + log1pf(expf(-fabsf(raw)));       // softplus, exact at both ends
+            gs[d] = expf(-rate * sp);
+        }
+        const float beta = sigmoidf_(to_f32(proj[a.b_off + h]));
+        __syncthreads();
+        // every warp forms the three sums over the key channels itself
+        float qq = 0.f, kk = 0.f, qk = 0.f;
+        for (int d = tid & 31; d < D; d += 32) {
+            qq = fmaf(qs[d], qs[d], qq);
+            kk = fmaf(ks[d], ks[d], kk);
+            qk = fmaf(qs[d], ks[d], qk);
+        }
+        const float iq = a.q_scale / sqrtf(warp_sum(qq) + 1e-6f), ik = 1.0f / sqrtf(warp_sum(kk) + 1e-6f);
+        qk = warp_sum(qk) * iq * ik;
+        float us = 0.f, os = 0.f;
+#pragma unroll
+        for (int i = 0; i < MR; ++i) {
+            const int r = rg + groups * i;
+            if (r < D) {
+                S[i] *= gs[r];
+                us = fmaf(ks[r] * ik, S[i], us);
+                os = fmaf(qs[r] * iq, S[i], os);
+            }
+        }
+        red[rg * cols + col] = us;
+        red[(groups + rg) * cols + col] = os;
+        __syncthreads();
+        us = os = 0.f;
+        for (int g = 0; g < groups; ++g) {
+            us += red[g * cols + col];
+            os += red[(groups + g) * cols + col];
+        }
+        const float u = live ? beta * (vs[col] - us) : 0.f;
+#pragma unroll
+        for (int i = 0; i < MR; ++i) {
+            const int r = rg + groups * i;
+            if (live && r < D) S_slot[(size_t)r * V + col] = fmaf(ks[r] * ik, u, S[i]);
+        }
+        const float o = live ? fmaf(qk, u, os) : 0.f;
+        const float inv = 1.0f / sqrtf(block_sum(rg == 0 ? o * o : 0.f, scratch) / (float)V + a.eps);
+        if (rg == 0 && live) {
+            const float g = a.g_raw[(size_t)row * a.ld_g + h * V + col];
+            const float y = o * inv * a.norm_w[col] * (a.gate == 1 ? g * sigmoidf_(g) : sigmoidf_(g));
+            static_cast<T*>(a.out)[(size_t)row * a.ld_out + h * V + col] = from_f32<T>(y * a.out_scale);
+        }
+        __syncthreads();                    // the head's values and sums may be overwritten
+    }
+}
+
+// The state space layer: a block per (entry, head) convolves its head's x and its group's B and C and updates the
+// state; x and the output go where ssd_finish_kernel reads them (it also moves the kept inputs on then).
+template <typename T, int MR>
+__global__ void __launch_bounds__(512, MR <= 16 ? 2 : 1)
+ssd_token_kernel(const ScanArgs a, float* __restrict__ conv_out, float* __restrict__ o_raw, int cols, int groups) {
+    extern __shared__ __align__(16) float smem[];
+    const int D = a.dim, V = a.v_dim;
+    float *bs = smem, *cs = bs + D, *xs = cs + D, *red = xs + V;                          // red: [groups][cols]
+    pdl_launch_dependents();
+    pdl_wait();
+    const int e = blockIdx.x / a.heads, h = blockIdx.x % a.heads, tid = threadIdx.x, g = h / (a.heads / a.groups);
+    const int row = a.q_start[e], col = tid % cols, rg = tid / cols, inner = a.heads * V;
+    const T* proj = static_cast<const T*>(a.proj) + (size_t)row * a.ld_proj;
+    float* slot = a.state + (size_t)a.slots[e] * (size_t)a.slot_stride;
+    float* S_slot = slot + (size_t)h * D * V;
+    const bool live = col < V;
+    float S[MR];
+#pragma unroll
+    for (int i = 0; i < MR; ++i) {
+        const int r = rg + groups * i;
+        S[i] = live && r < D ? S_slot[(size_t)r * V + col] : 0.f;
+    }
+    for (int c = tid; c < 2 * D + V; c += blockDim.x) {
+        const int ch = c < D ? inner + g * D + c : c < 2 * D ? inner + (a.groups + g) * D + c - D : h * V + c - 2 * D;
+        const float v = conv_one(a, proj, slot + a.kept_off, ch, false);
+        smem[c] = v;
+        if (c >= 2 * D) conv_out[(size_t)row * a.channels + ch] = v;
+    }
+    const float raw = to_f32(proj[a.dt_off + h]) + a.dt_bias[h];
+    const float dt = fmaxf(raw, 0.f) + log1pf(expf(-fabsf(raw)));               // softplus, exact at both ends
+    const float keep = expf(-expf(a.a_log[h]) * dt);
+    __syncthreads();
+    const float tx = live ? dt * xs[col] : 0.f;
+    float o = 0.f;
+#pragma unroll
+    for (int i = 0; i < MR; ++i) {
+        const int r = rg + groups * i;
+        if (live && r < D) {
+            const float s = fmaf(bs[r], tx, keep * S[i]);
+            o = fmaf(cs[r], s, o);
+            S_slot[(size_t)r * V + col] = s;
+        }
+    }
+    red[rg * cols + col] = o;
+    __syncthreads();
+    if (rg > 0 || !live) return;
+    for (int q = 1; q < groups; ++q) o += red[q * cols + col];
+    o_raw[(size_t)row * inner + h * V + col] = o;
+}
+
 template <typename T, int DELTA, int P, bool VEC>
 int launch_scan_rows(const ScanArgs& b, const float* vec, float* o_raw, int slices, int tokens, dim3 grid, size_t smem,
                      cudaStream_t stream) {
@@ -1083,9 +1266,29 @@ int launch_scan(const ScanArgs& a, int entries, int tokens, float* scratch, cuda
     int rc = 0;
     constexpr bool CONV = DELTA == SSD || DELTA == GATED_DELTA;
     bool scanned = false;
-    const int channels = a.channels;
+    const bool one_token = CONV && token_kernel_ok(b, tokens);
     if constexpr (CONV) {
         if (conv_out == nullptr) return KIPP_ERR_ARG;
+        if (one_token) {
+            const TokenShape t = token_shape(D, V);
+            const dim3 block((unsigned)(t.cols * t.groups));
+            if constexpr (DELTA == GATED_DELTA) {
+                const size_t bytes = ((size_t)3 * D + V + 2 * (size_t)t.groups * t.cols) * sizeof(float);
+                return kipp_launch(t.rows <= 8    ? gated_delta_token_kernel<T, 8>
+                                   : t.rows <= 16 ? gated_delta_token_kernel<T, 16>
+                                                  : gated_delta_token_kernel<T, TOKEN_ROWS>,
+                                   dim3((unsigned)(entries * a.groups)), block, bytes, stream, 1, b, t.cols, t.groups);
+            }
+            const size_t bytes = ((size_t)2 * D + V + (size_t)t.groups * t.cols) * sizeof(float);
+            rc = kipp_launch(t.rows <= 8 ? ssd_token_kernel<T, 8> : t.rows <= 16 ? ssd_token_kernel<T, 16> : ssd_token_kernel<T, TOKEN_ROWS>, dim3((unsigned)(entries * a.heads)),
+                             block, bytes, stream, 1, b, conv_out, o_raw, t.cols, t.groups);
+            if (rc) return rc;
+            scanned = true;
+        }
+    }
+    const int channels = a.channels;
+    if (scanned) {
+    } else if constexpr (CONV) {
         const bool by_fours = scan_by_fours(b) && ((uintptr_t)conv_out & 15) == 0 && ((uintptr_t)scratch & 15) == 0;
         // the state space layer's scan reads the convolved rows themselves; decays and step sizes lie where the
         // records would
@@ -1135,12 +1338,12 @@ int launch_scan(const ScanArgs& a, int entries, int tokens, float* scratch, cuda
         const long long parts = (long long)tokens * b.norm_groups;
         if (parts > 0x7fffffffLL) return KIPP_ERR_ARG;
         const int per_part = a.heads * a.v_dim / b.norm_groups;
-        rc = kipp_launch(ssd_finish_kernel<T>, dim3((unsigned)parts), dim3(per_part >= 128 ? 128 : (per_part + 31) / 32 * 32), 0,
-                         stream, 1, b, (const float*)conv_out, (const float*)o_raw);
+        rc = kipp_launch(ssd_finish_kernel<T>, dim3((unsigned)parts), dim3(one_token ? 256 : per_part >= 128 ? 128 : (per_part + 31) / 32 * 32), 0,
+                         stream, 1, b, (const float*)conv_out, (const float*)o_raw, one_token && b.taps > 1 ? 1 : 0);
     } else {
         rc = kipp_launch(recurrent_finish_kernel<T, DELTA>, wgrid, dim3(128), 0, stream, 1, b, (const float*)o_raw, tokens);
     }
-    if (rc || !CONV || b.taps <= 1) return rc;
+    if (rc || !CONV || b.taps <= 1 || one_token) return rc;
     return kipp_launch(ssd_conv_keep_kernel<T>, dim3((unsigned)entries, (unsigned)((channels + 255) / 256)), dim3(256), 0, stream,
                        1, b);
 }
