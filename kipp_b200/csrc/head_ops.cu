@@ -290,9 +290,9 @@ head_matvec_kernel(T* __restrict__ C, const T* __restrict__ A, const T* __restri
 }
 
 // In bfloat16: the same product on the tensor cores (mma.sync m16n8k16), all heads in one launch.  A block of 4 warps takes 64 tokens x 64 features of one head; K is walked in steps of 32
-// through shared memory (16-byte asynchronous copies, zeros beyond M, N and K); a warp owns 16
+// through four stages of shared memory (16-byte asynchronous copies, zeros beyond M, N and K); a warp owns 16
 // tokens x 64 features.  The sum over k runs in the same order for every token.
-constexpr int HM = 64, HN = 64, HK = 32, HLD = HK + 8;
+constexpr int HM = 64, HN = 64, HK = 32, HLD = HK + 8, H_STAGES = 4;
 __device__ __forceinline__ void mma_bf16_16816(float* c, const uint32_t* a, uint32_t b0, uint32_t b1) {
     asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
                  : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
@@ -302,8 +302,8 @@ __global__ void __launch_bounds__(128)
 head_matmul_mma_kernel(bf16* __restrict__ C, const bf16* __restrict__ A, const bf16* __restrict__ W, int M, int N, int K,
                        long long lda, long long a_head, long long w_head, long long ldc, long long c_head,
                        const bf16* __restrict__ gate, long long ld_gate) {
-    __shared__ __align__(16) bf16 As[HM * HLD];
-    __shared__ __align__(16) bf16 Ws[HN * HLD];
+    __shared__ __align__(16) bf16 A_stage[H_STAGES][HM * HLD];
+    __shared__ __align__(16) bf16 W_stage[H_STAGES][HN * HLD];
     pdl_launch_dependents();
     pdl_wait();
     const int h = blockIdx.z;
@@ -315,19 +315,28 @@ head_matmul_mma_kernel(bf16* __restrict__ C, const bf16* __restrict__ A, const b
     float acc[HN / 8][4];
 #pragma unroll
     for (int j = 0; j < HN / 8; ++j) acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.f;
-    for (int k0 = 0; k0 < K; k0 += HK) {
-        __syncthreads();                                            // the step before has read its tiles
-        // 64 rows x 4 chunks of 8 elements for each operand: 256 chunks, two per thread and operand
+    // 64 rows x 4 chunks of 8 elements for each operand: 256 chunks, two per thread and operand
+    auto fetch = [&](int k0, int stage) {
+#pragma unroll
         for (int i = tid; i < HM * (HK / 8); i += 128) {
             const int r = i >> 2, c = (i & 3) * 8;
             const bool ka = k0 + c < K;
             const bool oa = ka && m0 + r < M, ow = ka && n0 + r < N;
-            cp_async16(smem_address(As + r * HLD + c), oa ? A + (size_t)(m0 + r) * lda + k0 + c : A, oa ? 16 : 0);
-            cp_async16(smem_address(Ws + r * HLD + c), ow ? W + (size_t)(n0 + r) * K + k0 + c : W, ow ? 16 : 0);
+            cp_async16(smem_address(A_stage[stage] + r * HLD + c), oa ? A + (size_t)(m0 + r) * lda + k0 + c : A, oa ? 16 : 0);
+            cp_async16(smem_address(W_stage[stage] + r * HLD + c), ow ? W + (size_t)(n0 + r) * K + k0 + c : W, ow ? 16 : 0);
         }
+    };
+#pragma unroll
+    for (int s = 0; s < H_STAGES - 1; ++s) {
+        if (s * HK < K) fetch(s * HK, s);
         cp_async_commit();
-        cp_async_wait<0>();
-        __syncthreads();
+    }
+    for (int k0 = 0, s = 0; k0 < K; k0 += HK, s = (s + 1) % H_STAGES) {
+        cp_async_wait<H_STAGES - 2>();
+        __syncthreads();                                            // this step's tiles are there, those of the step before are read
+        if (k0 + (H_STAGES - 1) * HK < K) fetch(k0 + (H_STAGES - 1) * HK, (s + H_STAGES - 1) % H_STAGES);
+        cp_async_commit();
+        const bf16 *As = A_stage[s], *Ws = W_stage[s];
 #pragma unroll
         for (int ks = 0; ks < HK; ks += 16) {
             const bf16* ar = As + (warp * 16 + gid) * HLD + ks + tig * 2;
