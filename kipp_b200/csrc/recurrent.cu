@@ -41,9 +41,10 @@
 // Everything that enters the recurrence is formed in float32 from the
 // projections (which arrive in the compute type); the state never leaves float32.
 //
-// (The state space layer's convolution is a kernel of its own before them, and the inputs its slot keeps
-// are written by one after them.)
-// Three kernels per step.  (1) prepare: a warp per (token, head) forms the token's vectors in
+// Convolutions are a kernel of their own before the scan (conv_run_kernel: a thread walks a run of tokens
+// of one channel with its weights in registers), and the inputs a slot keeps are written after it.
+//
+// The general form is three kernels per step.  (1) prepare: a warp per (token, head) forms the token's vectors in
 // float32 (q/r, k, and for the delta rule w, a * u, u) in a workspace; fully parallel over the
 // step's tokens.  (2) scan: a block per (entry, head, slice of 32 value columns) -- the columns
 // of S evolve independently -- walks the entry's tokens in order; a thread owns one column and
@@ -53,6 +54,13 @@
 // is a batch of one.  (3) finish: a warp per (token, head) divides by the root mean square,
 // applies weight, gate and scale and stores in the compute type.  The order of every sum depends
 // on the sizes only.
+//
+// Two kinds have scans of their own for the sizes that divide by four: ssd_scan_kernel (straight from the
+// convolved rows, no records) and gated_delta_scan_kernel.  There a thread works on pairs of float32 and the
+// shuffles of one token's sums travel while the next token is worked on.  For steps of one token per request
+// ssd_token_kernel and gated_delta_token_kernel do the convolution, the state and the output in one launch.
+// A scan of many tokens starts when the kernel before it has left the GPU (kipp_launch_spread): blocks that
+// were placed early share few multiprocessors, and a scan lasts as long as its most crowded one.
 #include "common.cuh"
 #include <math.h>
 #include <algorithm>
